@@ -222,3 +222,32 @@ class NizoraxConfig(ModelConfig):
             return list(range(n))
         a, b, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
         return list(range(a)) + list(range(a, b)) * times + list(range(b, n))
+
+
+class NomanexConfig(ModelConfig):
+    """Nomanex (`"architecture": "Nomanex"`): `vocab`, `width`, `norm.eps`, `residual_mult`, `embedding.bigram` (`{"buckets",
+    "mul_prev", "mul_cur"}` or absent: the table of hashed token pairs), and a list `layers`, each entry with `type` ("gla" or
+    "latent_attention"), the mixer's sizes and constants under `mixer`, and `mlp` (`{"kind": "dense", "ff", "limit"}`,
+    `{"kind": "moe", "expert": {"ff"}, "router": {"experts", "top", "groups": {"count", "keep"}}}` or null).  An entry with
+    `weights_of` uses that layer's weights with caches of its own."""
+
+    KNOWN_KEYS = ("architecture", "vocab", "width", "norm", "residual_mult", "embedding", "layers", "torch_dtype", "dtype",
+                  "eos_token_id", "bos_token_id", "max_positions")
+
+    @property
+    def vocab_size(self) -> int:
+        return int(self.raw["vocab"])
+
+    @property
+    def hidden_size(self) -> int:
+        return int(self.raw["width"])
+
+    @property
+    def num_hidden_layers(self) -> int:
+        return len(self.raw["layers"])
+
+    def weights_layer(self, i: int) -> int:
+        """The layer whose tensors layer i uses."""
+        while self.raw["layers"][i].get("weights_of") is not None:
+            i = int(self.raw["layers"][i]["weights_of"])
+        return i

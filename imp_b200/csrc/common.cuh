@@ -171,7 +171,28 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_float<__nv_bfloat16>(f
 __device__ __forceinline__ float gelu_tanh_f(float z) {
     return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
-__device__ __forceinline__ float gate_act_f(float g, int act) { return act == 0 ? g / (1.f + expf(-g)) : gelu_tanh_f(g); }
+// The activation of a feed-forward: how a gate and an up value become one (kinds 0 to 2), or what happens to a plain value
+// (kind 3; 0 elsewhere: nothing).
+//   0  silu(g) * u        1  gelu(g) * u, tanh form
+//   2  both clipped: g <- min(g, limit), u <- min(max(u, -limit), limit);  g * sigmoid(1.702 g) * (u + 1)
+//   3  max(v, 0)^2 (products without a gate)
+enum : int { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_CLIPPED = 2, ACT_RELU2 = 3 };
+struct GateAct {
+    int kind;
+    float limit;
+    __host__ __device__ GateAct(int k = 0, float l = 0.f) : kind(k), limit(l) {}
+};
+__device__ __forceinline__ float gated_f(float g, float u, const GateAct& a) {
+    if (a.kind == ACT_SILU) return g / (1.f + expf(-g)) * u;
+    if (a.kind == ACT_GELU_TANH) return gelu_tanh_f(g) * u;
+    g = fminf(g, a.limit);
+    u = fminf(fmaxf(u, -a.limit), a.limit);
+    return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+}
+__device__ __forceinline__ float relu2_f(float v) {
+    const float r = fmaxf(v, 0.f);
+    return r * r;
+}
 
 __device__ __forceinline__ float load_as_float(const void* p, int dtype, int64_t i) {
     return dtype == IMP_F32 ? reinterpret_cast<const float*>(p)[i]

@@ -41,6 +41,88 @@ IMP_API int imp_embedding(float* out, const void* table, const int* ids, int n_t
     IMP_RETURN_LAUNCH();
 }
 
+// out[t, :] = table[id, :] * scale + bigram[row, :], row = (prev * mul_prev + id * mul_cur) mod buckets, prev the token before in
+// the sequence; a sequence's first token (position 0) reads row `buckets`, the table's last.  The token before a portion is in the
+// sequence's state, prev_state[slot]; the CTA of the portion's first token reads it and then leaves the portion's last token there.
+// A CTA per token, four columns a thread where the rows allow it (VEC).
+template <typename TW, int VEC>
+__global__ void bigram_embedding_kernel(float* __restrict__ out, const TW* __restrict__ table, const TW* __restrict__ bigram,
+                                        const int* __restrict__ ids, const int* __restrict__ positions, const int* __restrict__ seq_of_token,
+                                        const int* __restrict__ q_start, const int* __restrict__ slots, int* __restrict__ prev_state, int n_seqs, int d,
+                                        int vocab, int buckets, int64_t mul_prev, int64_t mul_cur, float scale, int* status) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int t = blockIdx.x;
+    const int id = ids[t], seq = seq_of_token[t], pos = positions[t];
+    float* o = out + (int64_t)t * d;
+    bool bad = id < 0 || id >= vocab || seq < 0 || seq >= n_seqs;
+    int prev = 0;
+    if (!bad) {
+        const bool first = q_start[seq] == t;
+        prev = first ? prev_state[slots[seq]] : ids[t - 1];
+        if (first) {
+            __syncthreads();
+            if (threadIdx.x == 0) prev_state[slots[seq]] = ids[q_start[seq + 1] - 1];
+        }
+        if (pos > 0 && (prev < 0 || prev >= vocab)) bad = true;
+    }
+    if (bad) {
+        if (threadIdx.x == 0) imp_report(status, seq < 0 || seq >= n_seqs ? IMP_BAD_SEQUENCE : IMP_BAD_TOKEN_ID);
+        for (int i = threadIdx.x; i < d; i += blockDim.x) o[i] = 0.f;
+        return;
+    }
+    const int64_t row = pos == 0 ? buckets : ((int64_t)prev * mul_prev + (int64_t)id * mul_cur) % buckets;
+    const TW *a = table + (int64_t)id * d, *b = bigram + row * d;
+    for (int i = threadIdx.x * VEC; i < d; i += blockDim.x * VEC) {
+        if constexpr (VEC == 1) {
+            o[i] = fmaf(to_float(a[i]), scale, to_float(b[i]));
+        } else {
+            float v[4];
+            if constexpr (sizeof(TW) == 4) {
+                const float4 x = *reinterpret_cast<const float4*>(a + i), y = *reinterpret_cast<const float4*>(b + i);
+                v[0] = fmaf(x.x, scale, y.x), v[1] = fmaf(x.y, scale, y.y), v[2] = fmaf(x.z, scale, y.z), v[3] = fmaf(x.w, scale, y.w);
+            } else {
+                const uint2 ux = *reinterpret_cast<const uint2*>(a + i), uy = *reinterpret_cast<const uint2*>(b + i);
+                const __nv_bfloat16 *x = reinterpret_cast<const __nv_bfloat16*>(&ux), *y = reinterpret_cast<const __nv_bfloat16*>(&uy);
+#pragma unroll
+                for (int k = 0; k < 4; ++k) v[k] = fmaf(to_float(x[k]), scale, to_float(y[k]));
+            }
+            *reinterpret_cast<float4*>(o + i) = make_float4(v[0], v[1], v[2], v[3]);
+        }
+    }
+}
+
+// bigram: [buckets + 1, d] of the table's type.  prev_state: one word per slot.  mul_prev, mul_cur in [0, buckets).
+IMP_API int imp_bigram_embedding(float* out, const void* table, const void* bigram, const int* ids, const int* positions, const int* seq_of_token,
+                                 const int* q_start, const int* slots, int* prev_state, int n_tokens, int n_seqs, int d, int vocab, int buckets,
+                                 int64_t mul_prev, int64_t mul_cur, int table_dtype, float scale, int* status, void* stream) {
+    if (n_tokens == 0) return 0;
+    IMP_CHECK_ARG(out && table && bigram && ids && positions && seq_of_token && q_start && slots && prev_state && d > 0 && vocab > 0,
+                  "imp_bigram_embedding: bad argument");
+    IMP_CHECK_ARG(buckets > 0 && mul_prev >= 0 && mul_prev < buckets && mul_cur >= 0 && mul_cur < buckets,
+                  "imp_bigram_embedding: the multipliers must be reduced modulo the %d buckets", buckets);
+    cudaStream_t s = (cudaStream_t)stream;
+    const bool vec = d % 4 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)table % 16 == 0 && (uintptr_t)bigram % 16 == 0;
+    const dim3 grid(n_tokens), block(d >= 1024 ? 256 : 128);
+    cudaError_t e;
+#define BIGRAM(TW, VEC)                                                                                                                            \
+    e = imp_launch(bigram_embedding_kernel<TW, VEC>, grid, block, 0, s, out, (const TW*)table, (const TW*)bigram, ids, positions, seq_of_token, q_start, \
+                   slots, prev_state, n_seqs, d, vocab, buckets, mul_prev, mul_cur, scale, status)
+    if (table_dtype == IMP_F32) {
+        if (vec) BIGRAM(float, 4);
+        else BIGRAM(float, 1);
+    } else {
+        if (vec) BIGRAM(__nv_bfloat16, 4);
+        else BIGRAM(__nv_bfloat16, 1);
+    }
+#undef BIGRAM
+    if (e != cudaSuccess) {
+        imp_set_error("imp_bigram_embedding: %s", cudaGetErrorString(e));
+        return (int)e;
+    }
+    return 0;
+}
+
 // ------------------------------------------------------------------- swiglu
 // out[t, f] = silu(gate) * up; the activation is computed in 32-bit.  Layout of gu[t, 2F]:
 // block == 0: gate columns 0..F-1, then up columns F..2F-1;

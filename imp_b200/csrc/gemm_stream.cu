@@ -57,7 +57,7 @@ template <int NT, typename TO, bool SWIGLU, int STAGES, int RG>
 __global__ void __launch_bounds__(GS_WARPS * 32 * RG) gemm_stream_kernel(TO* __restrict__ C, int64_t ldc,
                                                                     const __nv_bfloat16* __restrict__ A, int64_t lda,
                                                                     const __nv_bfloat16* __restrict__ W, int64_t ldw,
-                                                                    int M, int N, int K, int gate_act) {
+                                                                    int M, int N, int K, GateAct gate_act) {
     IMP_TL_BEGIN(5)
     extern __shared__ __align__(128) unsigned char gs_smem[];
     constexpr int STAGE_BYTES = gs_stage_bytes(NT, RG);
@@ -178,7 +178,7 @@ __global__ void __launch_bounds__(GS_WARPS * 32 * RG) gemm_stream_kernel(TO* __r
                 const int col = (c_tile * RG + rg) * 8 + (l >> 2);
                 const int tok = 8 * nt + 2 * (l & 3) + c;
                 if (n0 + (l >> 2) + 8 < N && tok < M)
-                    C[(int64_t)tok * ldc + col] = from_float<TO>(gate_act_f(gate, gate_act) * up);
+                    C[(int64_t)tok * ldc + col] = from_float<TO>(gated_f(gate, up, gate_act));
             }
         } else {
             // 16 rows x 8*NT tokens = NT*128 sums; thread i takes register slot i / 32 of lane i % 32.
@@ -203,7 +203,7 @@ __global__ void __launch_bounds__(GS_WARPS * 32 * RG) gemm_stream_kernel(TO* __r
 
 template <int NT, typename TO, bool SWIGLU, int STAGES, int RG>
 static cudaError_t launch_stream_st(TO* C, int64_t ldc, const __nv_bfloat16* A, int64_t lda, const __nv_bfloat16* W,
-                                    int64_t ldw, int M, int N, int K, cudaStream_t s, int gate_act = 0) {
+                                    int64_t ldw, int M, int N, int K, cudaStream_t s, GateAct gate_act = GateAct()) {
     static bool attr_set = false;   // once per instantiation (one device per process)
     if (!attr_set) {
         cudaError_t e = cudaFuncSetAttribute(gemm_stream_kernel<NT, TO, SWIGLU, STAGES, RG>,
@@ -234,7 +234,7 @@ static int gs_env_stages() {
 
 template <int NT, typename TO, bool SWIGLU>
 static cudaError_t launch_stream_nt(TO* C, int64_t ldc, const __nv_bfloat16* A, int64_t lda, const __nv_bfloat16* W,
-                                    int64_t ldw, int M, int N, int K, cudaStream_t s, int gate_act = 0) {
+                                    int64_t ldw, int M, int N, int K, cudaStream_t s, GateAct gate_act = GateAct()) {
     int stages = gs_env_stages();
     // Up to 8 tokens: two row groups per CTA where 32-row tiles still give about one CTA per SM or more.
     // With at least one such tile per SM, four stages of 21 KiB (two CTAs per SM); with 96/148 of that
@@ -259,7 +259,7 @@ static cudaError_t launch_stream_nt(TO* C, int64_t ldc, const __nv_bfloat16* A, 
 
 template <typename TO, bool SWIGLU>
 static int launch_stream(TO* C, int64_t ldc, const __nv_bfloat16* A, int64_t lda, const __nv_bfloat16* W, int64_t ldw,
-                         int M, int N, int K, cudaStream_t s, int gate_act = 0) {
+                         int M, int N, int K, cudaStream_t s, GateAct gate_act = GateAct()) {
     const cudaError_t e = (M <= 8) ? launch_stream_nt<1, TO, SWIGLU>(C, ldc, A, lda, W, ldw, M, N, K, s, gate_act)
                                    : launch_stream_nt<2, TO, SWIGLU>(C, ldc, A, lda, W, ldw, M, N, K, s, gate_act);
     if (e != cudaSuccess) {
@@ -288,21 +288,22 @@ IMP_API int imp_gemm_bf16_stream(void* C, int64_t ldc, int out_dtype, const void
 
 // C[M, N/2] = silu(gate) * up where W[N, K] holds gate and up rows interleaved in blocks of 8
 // (rows 16j..16j+7 = gate rows 8j..8j+7, rows 16j+8..16j+15 = up rows 8j..8j+7); bfloat16 output.
-// imp_gemm_bf16_stream_gated: the same with the gate's activation chosen (0 silu, 1 the tanh form of gelu).
+// imp_gemm_bf16_stream_gated: the same with the gate's activation chosen (0 silu, 1 the tanh form of gelu, 2 clipped to
+// `limit`, see GateAct).
 IMP_API int imp_gemm_bf16_stream_gated(void* C, int64_t ldc, const void* A, int64_t lda, const void* W, int64_t ldw,
-                                       int M, int N, int K, int act, void* stream) {
+                                       int M, int N, int K, int act, float limit, void* stream) {
     if (M == 0 || N == 0) return 0;
-    IMP_CHECK_ARG(act == 0 || act == 1, "imp_gemm_bf16_stream_gated: unknown activation %d", act);
+    IMP_CHECK_ARG(act >= ACT_SILU && act <= ACT_CLIPPED, "imp_gemm_bf16_stream_gated: unknown activation %d", act);
     IMP_CHECK_ARG(C && A && W && M > 0 && N > 0 && K > 0, "imp_gemm_bf16_stream_swiglu: bad argument");
     IMP_CHECK_ARG(M <= 16, "imp_gemm_bf16_stream_swiglu: M %d exceeds 16", M);
     IMP_CHECK_ARG(N % 16 == 0, "imp_gemm_bf16_stream_swiglu: %d interleaved rows are not a multiple of 16", N);
     IMP_CHECK_ARG(ldc >= N / 2 && lda >= K && ldw >= K, "imp_gemm_bf16_stream_swiglu: leading dimension too small");
     if (K % 8 || lda % 8 || ldw % 8 || (uintptr_t)A % 16 || (uintptr_t)W % 16) return IMP_ERR_UNSUPPORTED;
     return launch_stream<__nv_bfloat16, true>((__nv_bfloat16*)C, ldc, (const __nv_bfloat16*)A, lda,
-                                              (const __nv_bfloat16*)W, ldw, M, N, K, (cudaStream_t)stream, act);
+                                              (const __nv_bfloat16*)W, ldw, M, N, K, (cudaStream_t)stream, GateAct(act, limit));
 }
 
 IMP_API int imp_gemm_bf16_stream_swiglu(void* C, int64_t ldc, const void* A, int64_t lda, const void* W, int64_t ldw,
                                         int M, int N, int K, void* stream) {
-    return imp_gemm_bf16_stream_gated(C, ldc, A, lda, W, ldw, M, N, K, 0, stream);
+    return imp_gemm_bf16_stream_gated(C, ldc, A, lda, W, ldw, M, N, K, 0, 0.f, stream);
 }

@@ -34,13 +34,32 @@ constexpr int TC_STAGE_BYTES = TC_A_BYTES + TC_B_BYTES;
 constexpr int TC_SMEM_BYTES = TC_STAGES * TC_STAGE_BYTES + 1024 /* alignment slack */ + 256 /* barriers */;
 constexpr int TC_TMEM_COLS = 256;
 
-// TC_OUT_GEGLU_BF16 is a value of the entry points only: the gated epilogue with the other activation (a kernel parameter).
-enum TcEpilogue : int { TC_OUT_BF16 = 0, TC_OUT_F32 = 1, TC_OUT_SWIGLU_BF16 = 2, TC_OUT_QKV_ROPE = 3, TC_OUT_GEGLU_BF16 = 4 };
+// Values of the entry points only, the activation being a kernel parameter: TC_OUT_GEGLU_BF16 and TC_OUT_CLIPGLU_BF16 are the
+// gated epilogue with other activations, TC_OUT_RELU2_BF16 is the plain one with the squared relu.
+enum TcEpilogue : int { TC_OUT_BF16 = 0, TC_OUT_F32 = 1, TC_OUT_SWIGLU_BF16 = 2, TC_OUT_QKV_ROPE = 3, TC_OUT_GEGLU_BF16 = 4,
+                        TC_OUT_CLIPGLU_BF16 = 5, TC_OUT_RELU2_BF16 = 6 };
+// The kernels' own epilogue and activation of an entry point's epilogue.
+static GateAct split_epilogue(int* epilogue, float limit) {
+    switch (*epilogue) {
+        case TC_OUT_GEGLU_BF16: *epilogue = TC_OUT_SWIGLU_BF16; return GateAct(ACT_GELU_TANH);
+        case TC_OUT_CLIPGLU_BF16: *epilogue = TC_OUT_SWIGLU_BF16; return GateAct(ACT_CLIPPED, limit);
+        case TC_OUT_RELU2_BF16: *epilogue = TC_OUT_BF16; return GateAct(ACT_RELU2);
+        default: return GateAct();
+    }
+}
+
+// The activation of a product without a gate, on 32 accumulator columns.
+template <int EPI> __device__ __forceinline__ void plain_act(float (&v)[32], const GateAct& act) {
+    if (EPI == TC_OUT_BF16 && act.kind == ACT_RELU2) {
+#pragma unroll
+        for (int i = 0; i < 32; ++i) v[i] = relu2_f(v[i]);
+    }
+}
 
 // Store 32 consecutive accumulator columns of one row (converted as the epilogue asks).
 template <int EPI>
 __device__ __forceinline__ void tc_store32(void* __restrict__ Cv, int64_t ldc, int row, int col0, int M, int N,
-                                           const float (&v)[32], int gate_act = 0) {
+                                           const float (&v)[32], GateAct gate_act = GateAct()) {
     if (row >= M || col0 >= N) return;
     if (EPI == TC_OUT_F32) {
         float* dst = reinterpret_cast<float*>(Cv) + (int64_t)row * ldc + col0;
@@ -77,7 +96,7 @@ __device__ __forceinline__ void tc_store32(void* __restrict__ Cv, int64_t ldc, i
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
                 const float gate = v[16 * j + i], up = v[16 * j + 8 + i];
-                o[8 * j + i] = __float2bfloat16_rn(gate_act_f(gate, gate_act) * up);
+                o[8 * j + i] = __float2bfloat16_rn(gated_f(gate, up, gate_act));
             }
         if (col0 + 32 <= N && (ldc % 8) == 0) {
             reinterpret_cast<uint4*>(dst)[0] = *reinterpret_cast<uint4*>(&o[0]);
@@ -92,7 +111,7 @@ __device__ __forceinline__ void tc_store32(void* __restrict__ Cv, int64_t ldc, i
 template <int EPI>
 __global__ void __launch_bounds__(128, 1) gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a,
                                                          const __grid_constant__ CUtensorMap map_w, void* __restrict__ Cv,
-                                                         int64_t ldc, int M, int N, int K, int* status, int gate_act) {
+                                                         int64_t ldc, int M, int N, int K, int* status, GateAct gate_act) {
     pdl_wait();
     pdl_launch_dependents();
     extern __shared__ unsigned char tc_smem_raw[];
@@ -176,6 +195,7 @@ __global__ void __launch_bounds__(128, 1) gemm_tc_kernel(const __grid_constant__
         for (int c = 0; c < TC_BN / 32; ++c) {
             float v[32];
             tc_ld32(lane_base + (uint32_t)(c * 32), v);
+            plain_act<EPI>(v, gate_act);
             tc_store32<EPI>(Cv, ldc, row, n0 + c * 32, M, N, v, gate_act);
         }
     }
@@ -201,7 +221,7 @@ template <int EPI>
 __global__ void __launch_bounds__(TCP_THREADS, 1) gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a,
                                                                             const __grid_constant__ CUtensorMap map_w,
                                                                             void* __restrict__ Cv, int64_t ldc, int M, int N,
-                                                                            int K, int* status, int gate_act) {
+                                                                            int K, int* status, GateAct gate_act) {
     pdl_wait();
     pdl_launch_dependents();
     extern __shared__ unsigned char tc_smem_raw[];
@@ -303,6 +323,7 @@ __global__ void __launch_bounds__(TCP_THREADS, 1) gemm_tc_persistent_kernel(cons
             for (int c = 0; c < TC_BN / 32; ++c) {
                 float v[32];
                 tc_ld32(taddr + (uint32_t)(c * 32), v);
+                plain_act<EPI>(v, gate_act);
                 tc_store32<EPI>(Cv, ldc, row, n0 + c * 32, M, N, v, gate_act);
             }
             tc_fence_before_sync();
@@ -579,7 +600,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TCP_THREADS, 1)
     gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                         void* __restrict__ Cv, int64_t ldc, int M, int N, int K, int* status,
                         const __grid_constant__ QkvRopeArgs qkv, int splits, int kb_per_split, int64_t split_stride,
-                        const __grid_constant__ CUtensorMap map_c, int tma_store, int gate_act) {
+                        const __grid_constant__ CUtensorMap map_c, int tma_store, GateAct gate_act) {
     // tma_store (bfloat16 and SwiGLU epilogues): C goes out through shared memory and TMA stores described by map_c
     // (boxes of 128 rows x 64 columns, clipped at the matrix edges) instead of 16-byte stores from every thread.
     // splits > 1 (32-bit output only): the K range is cut into `splits` parts, each (tile, part) is a unit of work of its
@@ -737,6 +758,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TCP_THREADS, 1)
                         for (int cc = 0; cc < 2; ++cc) {
                             float v[32];
                             tc_ld32(taddr + (uint32_t)((2 * j + cc) * 32), v);
+                            plain_act<EPI>(v, gate_act);
 #pragma unroll
                             for (int i = 0; i < 4; ++i) q[4 * cc + i] = tc2_pack8(v + 8 * i);
                         }
@@ -751,7 +773,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TCP_THREADS, 1)
 #pragma unroll
                                 for (int i = 0; i < 8; ++i) {
                                     const float gate = v[16 * h + i], up = v[16 * h + 8 + i];
-                                    o[8 * h + i] = gate_act_f(gate, gate_act) * up;
+                                    o[8 * h + i] = gated_f(gate, up, gate_act);
                                 }
                             q[2 * cc] = tc2_pack8(o);
                             q[2 * cc + 1] = tc2_pack8(o + 8);
@@ -772,6 +794,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TCP_THREADS, 1)
                 for (int c = 0; c < TC2_BN / 32; ++c) {
                     float v[32];
                     tc_ld32(taddr + (uint32_t)(c * 32), v);
+                    plain_act<EPI>(v, gate_act);
                     tc_store32<EPI == TC_OUT_QKV_ROPE ? TC_OUT_BF16 : EPI>(Cz, ldc, row, n0 + c * 32, M, N, v, gate_act);
                 }
             }
@@ -841,7 +864,7 @@ __global__ void __launch_bounds__(128, 1) gemm_tc_swap_kernel(const __grid_const
                                                               const __grid_constant__ CUtensorMap map_x, void* __restrict__ Cv,
                                                               int64_t ldc, int64_t split_stride, int M, int N, int K,
                                                               int kb_per_split, int tile_rows, int* status,
-                                                              uint32_t wait_limit, int skip_kb, int gate_act) {
+                                                              uint32_t wait_limit, int skip_kb, GateAct gate_act) {
     constexpr int TCS_STAGES = tcs_rows_stages<BN, WROWS>();
     static_assert(tcs_rows_stage_bytes<BN, WROWS>() >= TCS_W_BYTES && tcs_rows_stage_bytes<BN, WROWS>() % 1024 == 0, "a stage spans what the MMA reads");
     IMP_TL_BEGIN(10 + EPI)
@@ -957,7 +980,7 @@ __global__ void __launch_bounds__(128, 1) gemm_tc_swap_kernel(const __grid_const
                     const float up = __shfl_xor_sync(0xffffffffu, v[i], 8);   // lane r + 8 holds the matching up row
                     const int tok = c * 32 + i;
                     if (is_gate && tok < M && col + 8 < N && r < tile_rows)
-                        base[(int64_t)tok * ldc + ocol] = __float2bfloat16_rn(gate_act_f(v[i], gate_act) * up);
+                        base[(int64_t)tok * ldc + ocol] = __float2bfloat16_rn(gated_f(v[i], up, gate_act));
                 }
             } else if (col < N && r < tile_rows) {
                 if (EPI == TC_OUT_F32) {
@@ -969,6 +992,7 @@ __global__ void __launch_bounds__(128, 1) gemm_tc_swap_kernel(const __grid_const
                     }
                 } else {
                     __nv_bfloat16* base = reinterpret_cast<__nv_bfloat16*>(Cv);
+                    plain_act<EPI>(v, gate_act);
 #pragma unroll
                     for (int i = 0; i < 32; ++i) {
                         const int tok = c * 32 + i;
@@ -1069,7 +1093,7 @@ static int make_map(CUtensorMap* map, const void* base, int rows, int K, int64_t
 
 template <int EPI>
 static int launch_tc(void* C, int64_t ldc, const CUtensorMap& ma, const CUtensorMap& mw, const CUtensorMap& mw128, int M,
-                     int N, int K, int* status, cudaStream_t s, int gate_act = 0) {
+                     int N, int K, int* status, cudaStream_t s, GateAct gate_act = GateAct()) {
     static bool attr_set = false;
     if (!attr_set) {
         cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize, TC_SMEM_BYTES);
@@ -1127,12 +1151,12 @@ static int launch_tc(void* C, int64_t ldc, const CUtensorMap& ma, const CUtensor
 // gate and up rows of W interleaved in runs of 8; 4 = the same with the tanh form of gelu on the gate.
 // Returns IMP_ERR_UNSUPPORTED when the operands do not meet the alignment rules of the tensor copies
 // (bases on 16-byte boundaries, row strides multiples of 8 elements): the caller uses another kernel.
-IMP_API int imp_gemm_bf16_tc(void* C, int64_t ldc, int epilogue, const void* A, int64_t lda, const void* W, int64_t ldw,
-                             int M, int N, int K, int* status, void* stream) {
+// 5 = the gated form with both values clipped to `limit` (ACT_CLIPPED), 6 = bfloat16 C[M,N] = max(A W^T, 0)^2.
+IMP_API int imp_gemm_bf16_tc_act(void* C, int64_t ldc, int epilogue, float limit, const void* A, int64_t lda, const void* W, int64_t ldw,
+                                 int M, int N, int K, int* status, void* stream) {
     if (M == 0 || N == 0) return 0;
     IMP_CHECK_ARG(C && A && W && M > 0 && N > 0 && K > 0, "imp_gemm_bf16_tc: bad argument");
-    const int gate_act = epilogue == TC_OUT_GEGLU_BF16 ? 1 : 0;
-    if (gate_act) epilogue = TC_OUT_SWIGLU_BF16;
+    const GateAct gate_act = split_epilogue(&epilogue, limit);
     IMP_CHECK_ARG(epilogue >= 0 && epilogue <= 2, "imp_gemm_bf16_tc: unknown epilogue %d", epilogue);
     IMP_CHECK_ARG(lda >= K && ldw >= K && ldc >= (epilogue == 2 ? N / 2 : N), "imp_gemm_bf16_tc: leading dimension too small");
     if (epilogue == 2) IMP_CHECK_ARG(N % 16 == 0, "imp_gemm_bf16_tc: %d interleaved rows are not a multiple of 16", N);
@@ -1143,9 +1167,15 @@ IMP_API int imp_gemm_bf16_tc(void* C, int64_t ldc, int epilogue, const void* A, 
     cudaStream_t s = (cudaStream_t)stream;
     CUtensorMap mw128;   // the W tile in halves of 128 rows, for CTA pairs
     if (int rc = make_map(&mw128, W, N, K, ldw, 128)) return rc;
-    if (epilogue == TC_OUT_BF16) return launch_tc<TC_OUT_BF16>(C, ldc, ma, mw, mw128, M, N, K, status, s);
+    if (epilogue == TC_OUT_BF16) return launch_tc<TC_OUT_BF16>(C, ldc, ma, mw, mw128, M, N, K, status, s, gate_act);
     if (epilogue == TC_OUT_F32) return launch_tc<TC_OUT_F32>(C, ldc, ma, mw, mw128, M, N, K, status, s);
     return launch_tc<TC_OUT_SWIGLU_BF16>(C, ldc, ma, mw, mw128, M, N, K, status, s, gate_act);
+}
+
+IMP_API int imp_gemm_bf16_tc(void* C, int64_t ldc, int epilogue, const void* A, int64_t lda, const void* W, int64_t ldw, int M, int N,
+                             int K, int* status, void* stream) {
+    IMP_CHECK_ARG(epilogue != TC_OUT_CLIPGLU_BF16, "imp_gemm_bf16_tc: the clipped gate needs a limit (imp_gemm_bf16_tc_act)");
+    return imp_gemm_bf16_tc_act(C, ldc, epilogue, 0.f, A, lda, W, ldw, M, N, K, status, stream);
 }
 
 // ---- many rows, few tiles: the K range in parts ------------------------------------------------------
@@ -1234,7 +1264,8 @@ static int tcs_tile_rows(int M, int N, int splits) {
 }
 
 static int tcs_splits(int M, int N, int K, int epilogue) {
-    if (epilogue == TC_OUT_SWIGLU_BF16 || epilogue == TC_OUT_GEGLU_BF16) return 1;
+    // the gated epilogues and the squared relu need the whole sum
+    if (epilogue != TC_OUT_BF16 && epilogue != TC_OUT_F32) return 1;
     const int slots = tcs_slots(M);                      // resident CTAs
     const int tiles = (N + 127) / 128;
     const int total_kb = (K + TC_BK - 1) / TC_BK;
@@ -1252,7 +1283,7 @@ IMP_API int64_t imp_gemm_bf16_tc_swap_scratch_floats(int M, int N, int K, int ep
 
 template <int BN, int EPI, int WROWS = 128>
 static int launch_tcs(void* C, int64_t ldc, int64_t split_stride, const CUtensorMap& mw, const CUtensorMap& mx, int M, int N,
-                      int K, int splits, int kb_per_split, int tile_rows, int* status, cudaStream_t s, int gate_act = 0) {
+                      int K, int splits, int kb_per_split, int tile_rows, int* status, cudaStream_t s, GateAct gate_act = GateAct()) {
     static bool attr_set = false;
     if (!attr_set) {
         cudaError_t e = cudaFuncSetAttribute(gemm_tc_swap_kernel<BN, EPI, WROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -1269,18 +1300,17 @@ static int launch_tcs(void* C, int64_t ldc, int64_t split_stride, const CUtensor
 
 // C = A[M,K] * W[N,K]^T for 1 <= M <= 128 with the weights on the M side of the MMA.
 // epilogue as for imp_gemm_bf16_tc.  `scratch` must hold imp_gemm_bf16_tc_swap_scratch_floats() floats.
-static int gemm_bf16_tc_swap_impl(void* C, int64_t ldc, int epilogue, const void* A, int64_t lda, const void* W, int64_t ldw,
+static int gemm_bf16_tc_swap_impl(void* C, int64_t ldc, int epilogue, float limit, const void* A, int64_t lda, const void* W, int64_t ldw,
                                   int M, int N, int K, float* scratch, int* status, void* stream, bool partials_only) {
     if (M == 0 || N == 0) return 0;
     IMP_CHECK_ARG((C || partials_only) && A && W && M > 0 && N > 0 && K > 0, "imp_gemm_bf16_tc_swap: bad argument");
     IMP_CHECK_ARG(M <= 128, "imp_gemm_bf16_tc_swap: M %d exceeds 128", M);
-    const int gate_act = epilogue == TC_OUT_GEGLU_BF16 ? 1 : 0;
-    if (gate_act) epilogue = TC_OUT_SWIGLU_BF16;
+    const int splits = tcs_splits(M, N, K, epilogue);
+    const GateAct gate_act = split_epilogue(&epilogue, limit);
     IMP_CHECK_ARG(epilogue >= 0 && epilogue <= 2, "imp_gemm_bf16_tc_swap: unknown epilogue %d", epilogue);
     if (epilogue == 2) IMP_CHECK_ARG(N % 16 == 0, "imp_gemm_bf16_tc_swap: %d interleaved rows are not a multiple of 16", N);
     IMP_CHECK_ARG(lda >= K && ldw >= K && ldc >= (epilogue == 2 ? N / 2 : N), "imp_gemm_bf16_tc_swap: leading dimension too small");
     if (K % 8 || lda % 8 || ldw % 8 || (uintptr_t)A % 16 || (uintptr_t)W % 16) return IMP_ERR_UNSUPPORTED;
-    const int splits = tcs_splits(M, N, K, epilogue);
     IMP_CHECK_ARG(splits == 1 || scratch, "imp_gemm_bf16_tc_swap: %d splits of K need scratch memory", splits);
     const int total_kb = (K + TC_BK - 1) / TC_BK;
     const int kb_per_split = (total_kb + splits - 1) / splits;
@@ -1312,9 +1342,9 @@ static int gemm_bf16_tc_swap_impl(void* C, int64_t ldc, int epilogue, const void
                            (const float*)scratch, split_stride, M, N, splits);
         if (e != cudaSuccess) { imp_set_error("gemm_tc_swap: %s", cudaGetErrorString(e)); return (int)e; }
     } else if (epilogue == TC_OUT_BF16) {
-        rc = BN == 32 ? launch_tcs<32, TC_OUT_BF16>(C, ldc, 0, mw, mx, M, N, K, 1, kb_per_split, tile_rows, status, s)
-           : BN == 64 ? launch_tcs<64, TC_OUT_BF16>(C, ldc, 0, mw, mx, M, N, K, 1, kb_per_split, tile_rows, status, s)
-                      : launch_tcs<128, TC_OUT_BF16>(C, ldc, 0, mw, mx, M, N, K, 1, kb_per_split, tile_rows, status, s);
+        rc = BN == 32 ? launch_tcs<32, TC_OUT_BF16>(C, ldc, 0, mw, mx, M, N, K, 1, kb_per_split, tile_rows, status, s, gate_act)
+           : BN == 64 ? launch_tcs<64, TC_OUT_BF16>(C, ldc, 0, mw, mx, M, N, K, 1, kb_per_split, tile_rows, status, s, gate_act)
+                      : launch_tcs<128, TC_OUT_BF16>(C, ldc, 0, mw, mx, M, N, K, 1, kb_per_split, tile_rows, status, s, gate_act);
     } else if (epilogue == TC_OUT_F32) {
         rc = BN == 32 ? launch_tcs<32, TC_OUT_F32>(C, ldc, 0, mw, mx, M, N, K, 1, kb_per_split, tile_rows, status, s)
            : BN == 64 ? launch_tcs<64, TC_OUT_F32>(C, ldc, 0, mw, mx, M, N, K, 1, kb_per_split, tile_rows, status, s)
@@ -1350,7 +1380,12 @@ IMP_API int imp_gemm_tc_test_hooks(unsigned wait_limit, int skip_kb) {
 
 IMP_API int imp_gemm_bf16_tc_swap(void* C, int64_t ldc, int epilogue, const void* A, int64_t lda, const void* W, int64_t ldw,
                                   int M, int N, int K, float* scratch, int* status, void* stream) {
-    return gemm_bf16_tc_swap_impl(C, ldc, epilogue, A, lda, W, ldw, M, N, K, scratch, status, stream, false);
+    IMP_CHECK_ARG(epilogue != TC_OUT_CLIPGLU_BF16, "imp_gemm_bf16_tc_swap: the clipped gate needs a limit (imp_gemm_bf16_tc_swap_act)");
+    return gemm_bf16_tc_swap_impl(C, ldc, epilogue, 0.f, A, lda, W, ldw, M, N, K, scratch, status, stream, false);
+}
+IMP_API int imp_gemm_bf16_tc_swap_act(void* C, int64_t ldc, int epilogue, float limit, const void* A, int64_t lda, const void* W, int64_t ldw,
+                                      int M, int N, int K, float* scratch, int* status, void* stream) {
+    return gemm_bf16_tc_swap_impl(C, ldc, epilogue, limit, A, lda, W, ldw, M, N, K, scratch, status, stream, false);
 }
 
 // How many partial results imp_gemm_bf16_tc_swap_partials leaves for this shape (1: it does not split, call the
@@ -1364,7 +1399,7 @@ IMP_API int imp_gemm_bf16_tc_swap_partials(float* scratch, const void* A, int64_
                                            int N, int K, int* status, void* stream) {
     IMP_CHECK_ARG(scratch, "imp_gemm_bf16_tc_swap_partials: no scratch memory");
     if (tcs_splits(M, N, K, TC_OUT_F32) < 2) return IMP_ERR_UNSUPPORTED;
-    return gemm_bf16_tc_swap_impl(nullptr, N, TC_OUT_F32, A, lda, W, ldw, M, N, K, scratch, status, stream, true);
+    return gemm_bf16_tc_swap_impl(nullptr, N, TC_OUT_F32, 0.f, A, lda, W, ldw, M, N, K, scratch, status, stream, true);
 }
 
 // C[M, N] (bfloat16 or float32, by `epilogue`) = the sum of the partial results, in split order.

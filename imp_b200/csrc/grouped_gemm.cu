@@ -7,7 +7,8 @@
 //              launch does not depend on the routing): routed experts.  Row r of the list reads A row a_rows[r]
 //              (null: r) and writes C row r.  The grid covers the most tiles any routing can make
 //              (rows / BM + groups); a CTA finds its group by walking seg, and leaves if there is no tile for it.
-// Optionally two weight matrices per group and the epilogue silu(A Wg^T) * (A Wu^T).
+// Epilogues on the 32-bit sums: none; silu(A Wg^T) * (A Wu^T) with two weight matrices per group; max(A W^T, 0)^2; or A W^T
+// times sigmoid of a gate that stands beside C (row r, column c_group_cols * g + n of `gate`).
 //
 // bfloat16: mma.sync m16n8k16 with 32-bit accumulation, 64 x 64 x 64 tiles through a cp.async ring of three or four stages,
 // fragments by ldmatrix, four warps.  (Tiles of 128 x 64 and 128 x 128 measured no faster for many rows a group and slower
@@ -20,6 +21,7 @@
 namespace {
 
 constexpr int GG_BM = 64, GG_BN = 64;
+enum : int { GG_PLAIN = 0, GG_SWIGLU = 1, GG_RELU2 = 2, GG_SIGMOID_GATE = 3 };   // the kernels' epilogues
 
 struct GroupedArgs {
     const void* A;
@@ -34,6 +36,8 @@ struct GroupedArgs {
     const int* seg;
     int M, N, K, G;
     int vec;   // rows of A and W start on 16 bytes and K is a multiple of 8 (bfloat16) / 4 (float32)
+    const void* gate;   // GG_SIGMOID_GATE: rows gate_ld apart, in the activations' type
+    int64_t gate_ld;
     int il;    // the gated epilogue's two matrices are one, gate and up rows alternating in runs of 8 (W2 unused)
 };
 
@@ -66,6 +70,17 @@ __device__ __forceinline__ bool find_tile(const GroupedArgs& p, int& g, int& row
 }
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+
+// The epilogue of a product with one weight matrix: row lr of C, column n of the group.
+template <int EPI, typename T>
+__device__ __forceinline__ float plain_epilogue(const GroupedArgs& p, float v, int64_t lr, int g, int n) {
+    if (EPI == GG_RELU2) return relu2_f(v);
+    if (EPI == GG_SIGMOID_GATE) {
+        const float z = to_float(reinterpret_cast<const T*>(p.gate)[lr * p.gate_ld + p.c_group_cols * g + n]);
+        return v / (1.f + expf(-z));
+    }
+    return v;
+}
 
 // --------------------------------------------------------------------------------------- bfloat16
 constexpr int GB_BK = 64, GB_LD = GB_BK + 8;   // a row of a block is a whole 128-byte line; padded rows: ldmatrix hits 32 different banks
@@ -114,10 +129,11 @@ template <bool SWIGLU, int BM> struct GroupedTile {
     static constexpr size_t SMEM = STAGES * STAGE_ELEMS * 2;
 };
 
-template <bool SWIGLU, int BM>
+template <int EPI, int BM>
 __global__ void __launch_bounds__(128) grouped_gemm_bf16_kernel(const GroupedArgs p) {
     pdl_wait();
     pdl_launch_dependents();
+    constexpr bool SWIGLU = EPI == GG_SWIGLU;
     using Tile = GroupedTile<SWIGLU, BM>;
     constexpr int GB_STAGES = Tile::STAGES;
     constexpr int WM = BM == 64 ? 32 : 16, WN = BM == 64 ? 32 : 16, MI = WM / 16, NJ = WN / 16;
@@ -220,6 +236,7 @@ __global__ void __launch_bounds__(128) grouped_gemm_bf16_kernel(const GroupedArg
                     if (n >= p.N) continue;
                     float v = acc[i][j][half * 2 + e];
                     if (SWIGLU) v = silu_f(v) * acu[i][j][half * 2 + e];   // the activation on the 32-bit sums
+                    else v = plain_epilogue<EPI, __nv_bfloat16>(p, v, lr, g, n);
                     crow[n] = __float2bfloat16_rn(v);
                 }
         }
@@ -228,8 +245,9 @@ __global__ void __launch_bounds__(128) grouped_gemm_bf16_kernel(const GroupedArg
 // ---------------------------------------------------------------------------------------- float32
 constexpr int GF_BK = 16;
 
-template <bool SWIGLU>
+template <int EPI>
 __global__ void __launch_bounds__(256) grouped_gemm_f32_kernel(const GroupedArgs p) {
+    constexpr bool SWIGLU = EPI == GG_SWIGLU;
     pdl_wait();
     pdl_launch_dependents();
     int g, row0, row_end;
@@ -313,7 +331,7 @@ __global__ void __launch_bounds__(256) grouped_gemm_f32_kernel(const GroupedArgs
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int gn = n0 + tn + j;
-            if (gn < p.N) C[(int64_t)lr * p.ldc + gn] = SWIGLU ? silu_f(acc[i][j]) * acu[i][j] : acc[i][j];
+            if (gn < p.N) C[(int64_t)lr * p.ldc + gn] = SWIGLU ? silu_f(acc[i][j]) * acu[i][j] : plain_epilogue<EPI, float>(p, acc[i][j], lr, g, gn);
         }
     }
 }
@@ -323,18 +341,22 @@ __global__ void __launch_bounds__(256) grouped_gemm_f32_kernel(const GroupedArgs
 // A: activations (dtype), rows lda apart.  W (and W2 with swiglu == 1): [G][N, K], groups w_group_stride elements apart,
 // rows ldw apart; swiglu == 2: W is [G][2N, K] with gate and up rows alternating in runs of 8 (W2 unused, N a multiple
 // of 8).  C: rows ldc apart.  seg == null: uniform groups of M rows each; else the list has M rows in all.
-IMP_API int imp_grouped_gemm(void* C, int64_t ldc, int64_t c_group_cols, const void* A, int64_t lda, int64_t a_group_cols,
-                             const int* a_rows, const void* W, const void* W2, int64_t w_group_stride, int64_t ldw, const int* seg,
-                             int M, int N, int K, int G, int swiglu, int dtype, void* stream) {
+// `epi` (0 where swiglu is set): 0 none, 2 max(., 0)^2, 3 times sigmoid(gate), gate's rows gate_ld apart and its columns C's own.
+IMP_API int imp_grouped_gemm_ex(void* C, int64_t ldc, int64_t c_group_cols, const void* A, int64_t lda, int64_t a_group_cols,
+                                const int* a_rows, const void* W, const void* W2, int64_t w_group_stride, int64_t ldw, const int* seg,
+                                int M, int N, int K, int G, int swiglu, int epi, const void* gate, int64_t gate_ld, int dtype, void* stream) {
     if (M == 0 || N == 0 || G == 0) return 0;
     IMP_CHECK_ARG(C && A && W && M > 0 && N > 0 && K > 0 && G > 0, "imp_grouped_gemm: bad argument");
     IMP_CHECK_ARG(swiglu != 1 || W2, "imp_grouped_gemm: the gated epilogue needs a second weight");
     IMP_CHECK_ARG(swiglu != 2 || N % 8 == 0, "imp_grouped_gemm: interleaved gate and up rows come in runs of 8");
+    IMP_CHECK_ARG(epi == GG_PLAIN || (!swiglu && (epi == GG_RELU2 || (epi == GG_SIGMOID_GATE && gate))), "imp_grouped_gemm: unknown epilogue %d, or no gate", epi);
+    if (swiglu) epi = GG_SWIGLU;
     GroupedArgs p;
     p.A = A, p.lda = lda, p.a_rows = a_rows, p.a_group_cols = a_group_cols;
     p.W = W, p.W2 = W2, p.w_group_stride = w_group_stride, p.ldw = ldw;
     p.C = C, p.ldc = ldc, p.c_group_cols = c_group_cols, p.seg = seg;
     p.M = M, p.N = N, p.K = K, p.G = G;
+    p.gate = gate, p.gate_ld = gate_ld;
     p.il = swiglu == 2 ? 1 : 0;
     const int el = dtype == IMP_F32 ? 4 : 2, per16 = 16 / el;
     auto aligned = [&](const void* q) { return q == nullptr || (uintptr_t)q % 16 == 0; };
@@ -343,35 +365,45 @@ IMP_API int imp_grouped_gemm(void* C, int64_t ldc, int64_t c_group_cols, const v
                 ? 1
                 : 0;
     cudaStream_t s = (cudaStream_t)stream;
-    cudaError_t e;
+    cudaError_t e = cudaSuccess;
     // few rows a group (a decode step's experts, its per-head products): 16-row tiles
     const int bm = (dtype != IMP_F32 && (seg ? M / G : M) < 16) ? 16 : GG_BM;
     const int row_tiles = seg ? (M + bm - 1) / bm + G : (M + bm - 1) / bm;
     IMP_CHECK_ARG(row_tiles <= 65535 && G <= 65535, "imp_grouped_gemm: too many row tiles or groups for one launch");
     const dim3 grid((N + GG_BN - 1) / GG_BN, row_tiles, seg ? 1 : G);
-    if (dtype == IMP_F32) {
-        e = swiglu ? imp_launch(grouped_gemm_f32_kernel<true>, grid, dim3(256), 0, s, p) : imp_launch(grouped_gemm_f32_kernel<false>, grid, dim3(256), 0, s, p);
-    } else {
-        static bool raised = false;
-        if (!raised) {
-            cudaFuncSetAttribute(grouped_gemm_bf16_kernel<true, 64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GroupedTile<true, 64>::SMEM);
-            cudaFuncSetAttribute(grouped_gemm_bf16_kernel<false, 64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GroupedTile<false, 64>::SMEM);
-            cudaFuncSetAttribute(grouped_gemm_bf16_kernel<true, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GroupedTile<true, 16>::SMEM);
-            cudaFuncSetAttribute(grouped_gemm_bf16_kernel<false, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GroupedTile<false, 16>::SMEM);
-            raised = true;
-        }
-        if (bm == 16)
-            e = swiglu ? imp_launch(grouped_gemm_bf16_kernel<true, 16>, grid, dim3(128), GroupedTile<true, 16>::SMEM, s, p)
-                       : imp_launch(grouped_gemm_bf16_kernel<false, 16>, grid, dim3(128), GroupedTile<false, 16>::SMEM, s, p);
-        else
-            e = swiglu ? imp_launch(grouped_gemm_bf16_kernel<true, 64>, grid, dim3(128), GroupedTile<true, 64>::SMEM, s, p)
-                       : imp_launch(grouped_gemm_bf16_kernel<false, 64>, grid, dim3(128), GroupedTile<false, 64>::SMEM, s, p);
+#define GG_BF16(EPI, BM)                                                                                                                  \
+    do {                                                                                                                                  \
+        constexpr size_t smem = GroupedTile<EPI == GG_SWIGLU, BM>::SMEM;                                                                  \
+        static bool raised = false;                                                                                                       \
+        if (!raised) raised = cudaFuncSetAttribute(grouped_gemm_bf16_kernel<EPI, BM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) == cudaSuccess; \
+        e = imp_launch(grouped_gemm_bf16_kernel<EPI, BM>, grid, dim3(128), smem, s, p);                                                   \
+    } while (0)
+#define GG_RUN(EPI)                                                                                          \
+    do {                                                                                                     \
+        if (dtype == IMP_F32) e = imp_launch(grouped_gemm_f32_kernel<EPI>, grid, dim3(256), 0, s, p);        \
+        else if (bm == 16) GG_BF16(EPI, 16);                                                                 \
+        else GG_BF16(EPI, 64);                                                                               \
+    } while (0)
+    switch (epi) {
+        case GG_SWIGLU: GG_RUN(GG_SWIGLU); break;
+        case GG_RELU2: GG_RUN(GG_RELU2); break;
+        case GG_SIGMOID_GATE: GG_RUN(GG_SIGMOID_GATE); break;
+        default: GG_RUN(GG_PLAIN); break;
     }
+#undef GG_RUN
+#undef GG_BF16
     if (e != cudaSuccess) {
         imp_set_error("imp_grouped_gemm: %s", cudaGetErrorString(e));
         return (int)e;
     }
     return 0;
+}
+
+IMP_API int imp_grouped_gemm(void* C, int64_t ldc, int64_t c_group_cols, const void* A, int64_t lda, int64_t a_group_cols,
+                             const int* a_rows, const void* W, const void* W2, int64_t w_group_stride, int64_t ldw, const int* seg,
+                             int M, int N, int K, int G, int swiglu, int dtype, void* stream) {
+    return imp_grouped_gemm_ex(C, ldc, c_group_cols, A, lda, a_group_cols, a_rows, W, W2, w_group_stride, ldw, seg, M, N, K, G, swiglu, 0, nullptr, 0,
+                               dtype, stream);
 }
 
 // dst[g][c][r] = src[g][r][c]: per-group transposes of small weight matrices, at load time.

@@ -1119,6 +1119,261 @@ ModelPlan nizorax_plan(const NizoraxConfig& cfg) {
     return plan;
 }
 
+// ------------------------------------------------------------------------------------ Nomanex
+NomanexConfig NomanexConfig::from_json(const Json& d, const std::string& where) {
+    NomanexConfig c;
+    c.architecture = d.get_string("architecture", "Nomanex");
+    c.vocab_size = positive("vocab", require_int(d, "vocab", where), where);
+    c.hidden_size = positive("width", require_int(d, "width", where), where);
+    c.max_position_embeddings = positive("max_positions", d.get_int("max_positions", 1 << 16), where);
+    c.torch_dtype = d.get_string("torch_dtype", d.get_string("dtype", "bfloat16"));
+    if (c.torch_dtype != "bfloat16" && c.torch_dtype != "float32")
+        bad(where + ": torch_dtype '" + c.torch_dtype + "' is not supported (bfloat16 or float32)");
+    if (const Json* eos = d.find("eos_token_id")) {
+        if (eos->is_array()) {
+            for (const auto& e : eos->items())
+                if (e.is_int()) c.eos_token_ids.push_back((int)e.as_int());
+        } else if (eos->is_int()) {
+            c.eos_token_ids.push_back((int)eos->as_int());
+        }
+    }
+    c.bos_token_id = d.get_int("bos_token_id", -1);
+    c.raw = d;
+    c.norm_eps = require_float(require_object(d, "norm", where), "eps", where + ": norm");
+    if (!(c.norm_eps > 0)) bad(where + ": norm.eps must be positive");
+    c.residual_mult = d.get_double("residual_mult", 1.0);
+    auto optional_object = [&](const Json& in, const char* key, const std::string& w) -> const Json* {
+        const Json* v = in.find(key);
+        if (!v || v->is_null()) return nullptr;
+        if (!v->is_object()) bad(w + ": '" + key + "' must be an object or null");
+        return v;
+    };
+    if (const Json* e = optional_object(d, "embedding", where))
+        if (const Json* b = optional_object(*e, "bigram", where + ": embedding")) {
+            const std::string bw = where + ": embedding.bigram";
+            c.has_bigram = true;
+            c.buckets = positive("buckets", require_int(*b, "buckets", bw), bw);
+            c.mul_prev = require_int(*b, "mul_prev", bw);
+            c.mul_cur = require_int(*b, "mul_cur", bw);
+        }
+    const Json& layers = require(d, "layers", where);
+    if (!layers.is_array() || layers.size() == 0) bad(where + ": 'layers' must be a non-empty list");
+    const int64_t n_layers = (int64_t)layers.size();
+    int i = 0;
+    for (const Json& lj : layers.items()) {
+        const std::string lw = where + ": layers[" + std::to_string(i) + "]";
+        if (!lj.is_object()) bad(lw + " must be an object");
+        Layer l;
+        l.type = lj.get_string("type", "");
+        if (const Json* w = lj.find("weights_of"))
+            if (!w->is_null()) {
+                l.weights_of = require_int(lj, "weights_of", lw);
+                if (l.weights_of < 0 || l.weights_of >= n_layers || l.weights_of == i)
+                    bad(lw + ": weights_of " + std::to_string(l.weights_of) + " must name another of the " + std::to_string(n_layers) + " layers");
+                c.layers.push_back(l);
+                ++i;
+                continue;       // everything else is that layer's
+            }
+        const Json& m = require_object(lj, "mixer", lw);
+        const std::string mw = lw + ".mixer";
+        l.heads = positive("heads", require_int(m, "heads", mw), mw);
+        l.dim = positive("dim", require_int(m, "dim", mw), mw);
+        l.vdim = positive("vdim", m.get_int("vdim", l.dim), mw);
+        if (l.type == "gla") {
+            l.tau = require_float(m, "tau", mw);
+            if (!(l.tau > 0)) bad(mw + ": tau must be positive");
+            l.decay_rank = m.get_int("decay_rank", 0);
+        } else if (l.type == "latent_attention") {
+            l.rot_dim = positive("rot_dim", require_int(m, "rot_dim", mw), mw);
+            l.kv_rank = positive("kv_rank", require_int(m, "kv_rank", mw), mw);
+            l.scale = m.find("scale") ? require_float(m, "scale", mw) : 1.0 / std::sqrt((double)(l.dim + l.rot_dim));
+            if (!(l.scale > 0)) bad(mw + ": scale must be positive");
+            if (const Json* mask = optional_object(m, "mask", mw)) l.window = positive("size", require_int(*mask, "size", mw + ".mask"), mw + ".mask");
+            const Json& rot = require_object(m, "rot", mw);
+            const std::string rw = mw + ".rot";
+            l.rot_base = require_float(rot, "base", rw);
+            l.rot_dims = positive("dims", rot.get_int("dims", l.rot_dim), rw);
+            if (!(l.rot_base > 0)) bad(rw + ": base must be positive");
+            if (l.rot_dims % 2 || l.rot_dims > l.rot_dim) bad(rw + ": dims " + std::to_string(l.rot_dims) + " must be even and at most rot_dim " + std::to_string(l.rot_dim));
+        } else {
+            bad(lw + ": unknown layer type '" + l.type + "' (known: gla, latent_attention)");
+        }
+        if (const Json* f = optional_object(lj, "mlp", lw)) {
+            const std::string fw = lw + ".mlp";
+            l.mlp = f->get_string("kind", "");
+            if (l.mlp == "dense") {
+                l.ff = positive("ff", require_int(*f, "ff", fw), fw);
+                l.limit = require_float(*f, "limit", fw);
+                if (!(l.limit > 0)) bad(fw + ": limit must be positive");
+            } else if (l.mlp == "moe") {
+                l.expert_ff = positive("ff", require_int(require_object(*f, "expert", fw), "ff", fw + ".expert"), fw + ".expert");
+                const Json& r = require_object(*f, "router", fw);
+                const std::string rw = fw + ".router";
+                l.experts = positive("experts", require_int(r, "experts", rw), rw);
+                l.top = positive("top", require_int(r, "top", rw), rw);
+                if (l.top > l.experts) bad(rw + ": top " + std::to_string(l.top) + " exceeds the " + std::to_string(l.experts) + " experts");
+                if (const Json* g = optional_object(r, "groups", rw)) {
+                    l.groups = positive("count", require_int(*g, "count", rw + ".groups"), rw + ".groups");
+                    l.keep = positive("keep", require_int(*g, "keep", rw + ".groups"), rw + ".groups");
+                    if (l.experts % l.groups || l.keep > l.groups || l.top > l.keep * (l.experts / l.groups))
+                        bad(rw + ".groups: count must divide the experts, keep be at most count, and the kept groups hold `top` experts");
+                }
+            } else {
+                bad(fw + ": unknown kind '" + l.mlp + "' (known: dense, moe)");
+            }
+        }
+        c.layers.push_back(l);
+        ++i;
+    }
+    c.num_hidden_layers = n_layers;
+    for (int j = 0; j < (int)n_layers; ++j) {
+        const Layer& own = c.layers[(size_t)c.weights_layer(j)];   // refuses a circle
+        Layer& l = c.layers[(size_t)j];
+        if (l.weights_of >= 0 && !l.type.empty() && l.type != own.type)
+            bad(where + ": layers[" + std::to_string(j) + "]: type '" + l.type + "' is not that of the layer whose weights it uses ('" + own.type + "')");
+    }
+    return c;
+}
+
+int NomanexConfig::weights_layer(int i) const {
+    int at = i;
+    for (size_t n = 0; n <= layers.size(); ++n) {
+        const int64_t next = layers[(size_t)at].weights_of;
+        if (next < 0) return at;
+        at = (int)next;
+    }
+    bad("config.json: layers[" + std::to_string(i) + "]: weights_of leads in a circle");
+    return -1;
+}
+
+std::vector<int> NomanexConfig::owners() const {
+    std::vector<int> o;
+    for (int i = 0; i < (int)layers.size(); ++i)
+        if (layers[(size_t)i].weights_of < 0) o.push_back(i);
+    return o;
+}
+
+Json NomanexConfig::to_json() const {
+    Json j = raw.is_object() ? raw : Json::object();
+    j["architecture"] = architecture;
+    j["vocab"] = vocab_size;
+    j["width"] = hidden_size;
+    j["torch_dtype"] = torch_dtype;
+    j.erase("dtype");
+    return j;
+}
+
+// Layer i's tensors are 'l<i>.norm1' (with '.b' and '.alpha'), 'l<i>.mix.*' and 'l<i>.mlp.*'.  The plan holds the layers that own
+// tensors; a layer that uses another's weights is that layer once more in the run order, which gives it caches of its own.
+ModelPlan nomanex_plan(const NomanexConfig& cfg) {
+    const int64_t d = cfg.hidden_size;
+    ModelPlan plan;
+    plan.architecture = cfg.architecture;
+    plan.hidden_size = d;
+    plan.vocab_size = cfg.vocab_size;
+    plan.max_positions = cfg.max_position_embeddings;
+    auto norm = [&](const std::string& tensor) {
+        PartSpec n;
+        n.kind = "dynamic_tanh";
+        n.params["size"] = d;
+        n.tensors = {{"weight", tensor}, {"bias", tensor + ".b"}, {"alpha", tensor + ".alpha"}};
+        return n;
+    };
+    const std::vector<int> owners = cfg.owners();
+    std::map<int, int> place;   // config layer -> plan layer
+    for (int i : owners) {
+        const NomanexConfig::Layer& l = cfg.layers[(size_t)i];
+        place[i] = (int)plan.layers.size();
+        const std::string p = "l" + std::to_string(i) + ".", a = p + "mix.", f = p + "mlp.";
+        PartSpec mixer;
+        mixer.params["hidden_size"] = d;
+        mixer.params["num_heads"] = l.heads;
+        mixer.params["value_dim"] = l.vdim;
+        mixer.params["norm_eps"] = cfg.norm_eps;
+        if (l.type == "gla") {
+            mixer.kind = "gated_linear_attention";
+            mixer.params["key_dim"] = l.dim;
+            mixer.params["tau"] = l.tau;
+            if (l.decay_rank > 0) mixer.params["decay_rank"] = l.decay_rank;
+            mixer.tensors = {{"q_proj", a + "q"}, {"k_proj", a + "k"}, {"v_proj", a + "v"}, {"gate_proj", a + "g"}, {"decay_down", a + "a1"},
+                             {"decay_up", a + "a2"}, {"decay_bias", a + "a2.b"}, {"out_norm", a + "norm"}, {"o_proj", a + "o"}};
+        } else {
+            mixer.kind = "latent_attention";
+            mixer.params["head_dim"] = l.dim;
+            mixer.params["rot_dim"] = l.rot_dim;
+            mixer.params["rot_dims"] = l.rot_dims;
+            mixer.params["rot_base"] = l.rot_base;
+            mixer.params["rot_pairing"] = "neighbours";
+            mixer.params["kv_rank"] = l.kv_rank;
+            mixer.params["q_rank"] = (int64_t)0;
+            mixer.params["scale"] = l.scale;
+            mixer.params["window"] = l.window;
+            mixer.params["out_gate"] = true;
+            mixer.params["pad_cache"] = true;
+            mixer.params["max_positions"] = cfg.max_position_embeddings;
+            mixer.tensors = {{"q_proj", a + "q"}, {"kv_down", a + "dkv"}, {"kv_norm", a + "dkv.norm"}, {"k_up", a + "uk"}, {"v_up", a + "uv"},
+                             {"gate_proj", a + "g"}, {"o_proj", a + "o"}};
+        }
+        LayerSpec layer;
+        layer.block = "parallel";
+        layer.block_params["residual_mult"] = cfg.residual_mult;
+        layer.block_params["has_ffn"] = !l.mlp.empty();
+        layer.parts = {{"norm", norm(p + "norm1")}, {"mixer", mixer}};
+        if (!l.mlp.empty()) {
+            PartSpec ffn;
+            ffn.params["hidden_size"] = d;
+            if (l.mlp == "dense") {
+                ffn.kind = "gated_mlp";
+                ffn.params["intermediate_size"] = l.ff;
+                ffn.params["activation"] = "clipped";
+                ffn.params["limit"] = l.limit;
+                ffn.tensors = {{"gate_proj", f + "gate"}, {"up_proj", f + "up"}, {"down_proj", f + "down"}};
+            } else {
+                ffn.kind = "routed_experts";
+                ffn.params["num_experts"] = l.experts;
+                ffn.params["top_k"] = l.top;
+                ffn.params["expert_size"] = l.expert_ff;
+                ffn.params["expert"] = "relu2";
+                ffn.params["router_bias"] = false;
+                ffn.params["scores"] = "softmax_all";
+                ffn.params["num_groups"] = l.groups;
+                ffn.params["keep_groups"] = l.keep;
+                ffn.params["group_score"] = "max";
+                ffn.tensors = {{"router", f + "router"}};
+                for (int64_t e = 0; e < l.experts; ++e) {
+                    const std::string n = std::to_string(e), t = f + "e" + n + ".";
+                    ffn.tensors.emplace_back("up_" + n, t + "up");
+                    ffn.tensors.emplace_back("down_" + n, t + "down");
+                }
+            }
+            layer.parts.emplace_back("feed_forward", ffn);
+        }
+        plan.layers.push_back(layer);
+    }
+    if (owners.size() != cfg.layers.size()) {
+        plan.has_order = true;
+        for (int i = 0; i < (int)cfg.layers.size(); ++i) plan.order.push_back(place.at(cfg.weights_layer(i)));
+    }
+    plan.embedding.params["vocab_size"] = cfg.vocab_size;
+    plan.embedding.params["hidden_size"] = d;
+    if (cfg.has_bigram) {
+        plan.embedding.kind = "bigram_embedding";
+        plan.embedding.params["buckets"] = cfg.buckets;
+        plan.embedding.params["mul_prev"] = cfg.mul_prev;
+        plan.embedding.params["mul_cur"] = cfg.mul_cur;
+        plan.embedding.tensors = {{"weight", "embed"}, {"bigram", "bigram"}};
+    } else {
+        plan.embedding.kind = "token_embedding";
+        plan.embedding.tensors = {{"weight", "embed"}};
+    }
+    plan.final_norm = norm("final.norm");
+    plan.head.kind = "linear_head";
+    plan.head.params["vocab_size"] = cfg.vocab_size;
+    plan.head.params["hidden_size"] = d;
+    plan.head.tensors = {{"weight", "head"}};
+    return plan;
+}
+
 // ------------------------------------------------------------------------------------ registry
 namespace {
 std::mutex g_arch_mutex;
@@ -1164,6 +1419,13 @@ void ensure_builtin_archs() {
         };
         nz.plan = [](const Json& d) { return nizorax_plan(NizoraxConfig::from_json(d, "config.json")); };
         archs()[nz.name] = nz;
+        Architecture nm;
+        nm.name = "Nomanex";
+        nm.parse_config = [](const Json& d, const std::string& where) -> std::shared_ptr<ModelConfig> {
+            return std::make_shared<NomanexConfig>(NomanexConfig::from_json(d, where));
+        };
+        nm.plan = [](const Json& d) { return nomanex_plan(NomanexConfig::from_json(d, "config.json")); };
+        archs()[nm.name] = nm;
     });
 }
 }  // namespace

@@ -186,6 +186,42 @@ struct NizoraxConfig : ModelConfig {
 
 ModelPlan nizorax_plan(const NizoraxConfig& cfg);
 
+// Nomanex ("architecture": "Nomanex"): a parallel decoder, x <- x + m (mixer(h) + ff(h)) with one norm h = tanh(alpha x) w + b a
+// layer.  A layer's mixer is gated linear attention (a decay per key channel) or latent attention over a sliding window (gated
+// heads, a rotation of neighbouring pairs, no query latent); its feed-forward is dense with a clipped gate, a mixture of experts
+// without gates (softmax scores over all experts, groups), or absent.  A layer with `weights_of` uses another layer's weights with
+// caches of its own.  The embedding may add a row of a table of hashed token pairs.  The keys are this family's own.
+struct NomanexConfig : ModelConfig {
+    struct Layer {
+        std::string type;                         // "gla" | "latent_attention"
+        int64_t heads = 0, dim = 0, vdim = 0;
+        // gla
+        double tau = 1.0;
+        int64_t decay_rank = 0;                   // 0 = the checkpoint's tensor decides
+        // latent attention
+        int64_t rot_dim = 0, kv_rank = 0, rot_dims = 0, window = 0;   // window 0: none
+        double scale = 0, rot_base = 10000.0;
+        // feed-forward
+        std::string mlp;                          // "" (none) | "dense" | "moe"
+        int64_t ff = 0;                           // dense
+        double limit = 0;
+        int64_t experts = 0, top = 0, expert_ff = 0, groups = 0, keep = 0;   // moe; groups 0: none
+        int64_t weights_of = -1;                  // the layer whose weights this one uses; -1: its own
+    };
+    std::vector<Layer> layers;
+    double norm_eps = 1e-6, residual_mult = 1.0;
+    bool has_bigram = false;
+    int64_t buckets = 0, mul_prev = 0, mul_cur = 0;
+
+    static NomanexConfig from_json(const Json& d, const std::string& where);
+    Json to_json() const override;
+    // The layer whose tensors layer i uses, and the layers that own tensors, in order.
+    int weights_layer(int i) const;
+    std::vector<int> owners() const;
+};
+
+ModelPlan nomanex_plan(const NomanexConfig& cfg);
+
 // ------------------------------------------------------------------------------------ registry
 struct Architecture {
     std::string name;

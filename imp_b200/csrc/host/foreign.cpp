@@ -125,8 +125,8 @@ struct ForeignBlock : Block, Foreign {
 struct ForeignEmbedding : Embedding, Foreign {
     int64_t hidden = 0;
     bool graph_safe() const override { return false; }
-    Tensor forward(Step& st) override {
-        ImpCall c = base_call(st, nullptr);
+    Tensor forward(Step& st, LayerCache* cache) override {
+        ImpCall c = base_call(st, cache);
         c.h = st.rt->empty(st.T(), hidden, F32, true);
         run(c);
         return c.h;

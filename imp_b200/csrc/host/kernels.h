@@ -14,6 +14,9 @@ int imp_device_sm_count(void);
 
 int imp_embedding(float* out, const void* table, const int* ids, int n_tokens, int d, int vocab, int table_dtype,
                   float scale, int* status, void* stream);
+int imp_bigram_embedding(float* out, const void* table, const void* bigram, const int* ids, const int* positions, const int* seq_of_token,
+                         const int* q_start, const int* slots, int* prev_state, int n_tokens, int n_seqs, int d, int vocab, int buckets,
+                         int64_t mul_prev, int64_t mul_cur, int table_dtype, float scale, int* status, void* stream);
 int imp_swiglu(void* out, const void* gate_up, int n_tokens, int F, int block, int dtype, void* stream);
 int imp_cast(void* dst, int dst_dtype, const void* src, int src_dtype, int64_t n, void* stream);
 int imp_random_fill(void* out, int dtype, int64_t n, uint64_t tensor_seed, int mode, float std, float norm_std,
@@ -74,12 +77,16 @@ int imp_gemm_bf16_stream(void* C, int64_t ldc, int out_dtype, const void* A, int
 int imp_gemm_bf16_stream_swiglu(void* C, int64_t ldc, const void* A, int64_t lda, const void* W, int64_t ldw, int M, int N,
                                 int K, void* stream);
 int imp_gemm_bf16_stream_gated(void* C, int64_t ldc, const void* A, int64_t lda, const void* W, int64_t ldw, int M, int N,
-                               int K, int act, void* stream);
+                               int K, int act, float limit, void* stream);
 int imp_gemm_bf16_tc_splits(int M, int N, int K);
 int imp_gemm_bf16_tc_partials(float* scratch, const void* A, int64_t lda, const void* W, int64_t ldw, int M, int N, int K, int* status,
                               void* stream);
 int imp_gemm_bf16_tc(void* C, int64_t ldc, int epilogue, const void* A, int64_t lda, const void* W, int64_t ldw, int M,
                      int N, int K, int* status, void* stream);
+int imp_gemm_bf16_tc_act(void* C, int64_t ldc, int epilogue, float limit, const void* A, int64_t lda, const void* W, int64_t ldw, int M,
+                         int N, int K, int* status, void* stream);
+int imp_gemm_bf16_tc_swap_act(void* C, int64_t ldc, int epilogue, float limit, const void* A, int64_t lda, const void* W, int64_t ldw,
+                              int M, int N, int K, float* scratch, int* status, void* stream);
 int64_t imp_gemm_bf16_tc_swap_scratch_floats(int M, int N, int K, int epilogue);
 int imp_gemm_bf16_tc_swap(void* C, int64_t ldc, int epilogue, const void* A, int64_t lda, const void* W, int64_t ldw, int M,
                           int N, int K, float* scratch, int* status, void* stream);
@@ -108,6 +115,11 @@ int imp_typical_filter(float* logits, int64_t ld, int n_rows, int V, const float
 int imp_sample_mirostat(const float* logits, int64_t ld, int n_rows, int V, const int* active, const float* temperature,
                         const float* mu, const float* uniform, int* out, float* surprise, void* stream);
 
+// a norm without statistics behind the sum of two branches (dynamic_tanh.cu)
+int imp_add_dyt(float* h, float mult, const void* t1, const float* parts1, int n_splits1, const void* y1, const int* row1, const float* wts1,
+                int top1, const void* t2, const float* parts2, int n_splits2, const void* y2, const int* row2, const float* wts2, int top2,
+                const float* alpha, const void* w, const void* b, void* out, const int* rows, int n_stream, int n_out, int d, int act_dtype,
+                int w_dtype, void* stream);
 // layer norm with the residual sum, and streams whose branches carry a factor per column (layernorm.cu)
 int imp_add_layernorm(float* h, const void* branch, const float* col_scale, const void* w, void* out, const int* rows,
                       int n_out_rows, int d, float eps, int act_dtype, int w_dtype, int write_h, void* stream);
@@ -139,6 +151,10 @@ int imp_gdrc_prepare(const void* proj, int64_t ld, const float* conv_w, int taps
                      const int* q_start, const int* slots, int n_tokens, int n_seqs, int G, int D, int H, int Dv, const float* dpre,
                      const float* a_log, const float* dt_bias, float unit_eps, float* q, float* kw, float* w, float* v, float* scal,
                      int act_dtype, int* status, void* stream);
+int imp_gla_prepare(const void* proj, int64_t ld, int n_tokens, int H, int D, int Dv, int R, const float* w2t, const float* bias, float tau,
+                    float q_scale, float* q, float* kw, float* w, float* v, float* scal, int act_dtype, void* stream);
+int imp_gla_decode(const void* proj, int64_t ld, int n_tokens, int H, int D, int Dv, int R, const float* w2t, const float* bias, float tau,
+                   float q_scale, const float* out_w, float eps, float* state, const int* slots, void* y, int act_dtype, void* stream);
 int imp_gdr_output_ex(void* y, const float* o, const void* gate, int64_t gate_ld, const float* w, int w_head_stride, int gate_act,
                       float eps, int n_tokens, int H, int Dv, int act_dtype, void* stream);
 // attention with normalised, partly rotated, scaled and gated heads; blocks of two mixers (qkv_prepare.cu)
@@ -157,7 +173,7 @@ int imp_diff_combine(void* y, const void* attn, int64_t ld, int n_tokens, int G,
 int imp_head_gate(void* y, int64_t y_ld, const void* g, int64_t g_ld, int n_tokens, int H, int Dv, int dtype, void* stream);
 int imp_rms_pair_mean(void* out, const void* a, const float* wa, float ca, const void* b, const float* wb, float cb, int n_rows, int d,
                       float eps, int dtype, void* stream);
-int imp_gated_act(void* out, const void* gate_up, int n_tokens, int F, int block, int act, int dtype, void* stream);
+int imp_gated_act(void* out, const void* gate_up, int n_tokens, int F, int block, int act, float limit, int dtype, void* stream);
 int imp_act_rows(void* out, const void* x, int64_t ld, int n_tokens, int n, int act, int dtype, void* stream);
 int imp_gather_head_cols(void* dst, const void* src, int n_tokens, int H, int ds, int n, int dtype, void* stream);
 // a short causal convolution added to its input; a normalised polynomial as activation (short_conv.cu)
@@ -168,6 +184,9 @@ int imp_polynorm(void* out, const void* z, int64_t ld, int n_tokens, int n, cons
 int imp_grouped_gemm(void* C, int64_t ldc, int64_t c_group_cols, const void* A, int64_t lda, int64_t a_group_cols,
                      const int* a_rows, const void* W, const void* W2, int64_t w_group_stride, int64_t ldw, const int* seg,
                      int M, int N, int K, int G, int swiglu, int dtype, void* stream);
+int imp_grouped_gemm_ex(void* C, int64_t ldc, int64_t c_group_cols, const void* A, int64_t lda, int64_t a_group_cols,
+                        const int* a_rows, const void* W, const void* W2, int64_t w_group_stride, int64_t ldw, const int* seg,
+                        int M, int N, int K, int G, int swiglu, int epi, const void* gate, int64_t gate_ld, int dtype, void* stream);
 int imp_transpose_groups(void* dst, const void* src, int G, int R, int Cn, int dtype, void* stream);
 // latent attention (latent_attention.cu)
 int imp_latent_prepare(const void* proj, int64_t ld, int n_tokens, int q_rank, int kv_rank, int rot, const float* wq,
@@ -175,6 +194,11 @@ int imp_latent_prepare(const void* proj, int64_t ld, int n_tokens, int q_rank, i
                        int rot_dims, int max_pos, const int* positions, const int* seq_of_token, const int* block_table,
                        int bt_stride, int n_seqs, void* pages, int page_size, int num_pages, int act_dtype, int* status,
                        void* stream);
+int imp_latent_prepare_ex(const void* proj, int64_t ld, int n_tokens, int q_rank, int kv_rank, int rot, const float* wq, const float* wkv,
+                          float eps, void* cq, int64_t cq_ld, const float* cos_tab, const float* sin_tab, int rot_dims, int pairing,
+                          int max_pos, const int* positions, const int* seq_of_token, const int* block_table, int bt_stride, int n_seqs,
+                          void* pages, int page_len, int page_size, int num_pages, const void* q, int64_t q_ld, int q_head, void* q_out,
+                          int64_t q_out_ld, int H, int act_dtype, int* status, void* stream);
 int imp_latent_query_rope(const void* q, int64_t q_ld, int n_tokens, int H, int D, int rot, void* out, int64_t out_ld, int kv_rank,
                           const float* cos_tab, const float* sin_tab, int rot_dims, int max_pos, const int* positions,
                           int act_dtype, int* status, void* stream);
@@ -193,12 +217,16 @@ int imp_wkv_output(void* y, const float* o, const void* g, int64_t ldg, const fl
 int imp_moe_route(const void* x, int64_t ldx, int n_tokens, int d, const float* wr, const float* br, int E, int top, const float* wg,
                   int* idx, float* wts, float* gate, int act_dtype, void* stream);
 int imp_moe_route_ex(const void* x, int64_t ldx, int n_tokens, int d, const float* wr, const float* br, int E, int top, const float* wg,
-                     int* idx, float* wts, float* gate, int score_mode, int n_groups, int keep, float weight_scale, int act_dtype, void* stream);
+                     int* idx, float* wts, float* gate, int score_mode, int n_groups, int keep, int group_top, float weight_scale, int act_dtype,
+                     void* stream);
 int imp_moe_sort(const int* idx, int n_tokens, int top, int E, int* seg, int* row_token, int* pair_row, void* stream);
 int imp_gather_rows(void* dst, const void* src, int64_t ld, const int* idx, int n_rows, int d, int dtype, void* stream);
 int imp_moe_combine(void* out, const void* y, const int* pair_row, const float* wts, int n_tokens, int top, const void* shared,
                     const float* gate, int d, int act_dtype, void* stream);
 }
 
+// Epilogues of the products over groups (imp_grouped_gemm_ex).
+enum { GROUPED_PLAIN = 0, GROUPED_RELU2 = 2, GROUPED_SIGMOID_GATE = 3 };
 // Epilogues of the tcgen05 products.
-enum { TC_OUT_BF16 = 0, TC_OUT_F32 = 1, TC_OUT_SWIGLU = 2, TC_OUT_GEGLU = 4 };   // 2 / 4: act(gate) * up, act silu / gelu (tanh form)
+enum { TC_OUT_BF16 = 0, TC_OUT_F32 = 1, TC_OUT_SWIGLU = 2, TC_OUT_GEGLU = 4, TC_OUT_CLIPGLU = 5, TC_OUT_RELU2 = 6 };
+// 2 / 4: act(gate) * up, act silu / gelu (tanh form); 5: gate and up clipped to a limit; 6: max(., 0)^2, no gate

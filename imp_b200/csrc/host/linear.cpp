@@ -57,13 +57,14 @@ void swiglu(Runtime& rt, Tensor out, const Tensor& gate_up, int interleave) {
     check_launch(imp_swiglu(out.data, gate_up.data, (int)rows(out), (int)cols(out), interleave, out.dtype, rt.stream), "swiglu");
 }
 
-void gated_act(Runtime& rt, Tensor out, const Tensor& gate_up, int interleave, int act) {
-    if (act == 0) return swiglu(rt, out, gate_up, interleave);
+void gated_act(Runtime& rt, Tensor out, const Tensor& gate_up, int interleave, GatedAct act) {
+    if (act.kind == 0) return swiglu(rt, out, gate_up, interleave);
     need(cols(gate_up) == 2 * cols(out) && rows(gate_up) == rows(out) && gate_up.dtype == out.dtype && contiguous(out) &&
              contiguous(gate_up),
          "gated_act: gate_up must be [T, 2F] beside out [T, F], both dense");
     ++rt.launches;
-    check_launch(imp_gated_act(out.data, gate_up.data, (int)rows(out), (int)cols(out), interleave, act, out.dtype, rt.stream), "gated_act");
+    check_launch(imp_gated_act(out.data, gate_up.data, (int)rows(out), (int)cols(out), interleave, act.kind, act.limit, out.dtype, rt.stream),
+                 "gated_act");
 }
 
 void embedding(Runtime& rt, Tensor out, const Tensor& table, const int32_t* ids, int n, float scale) {
@@ -104,9 +105,9 @@ static void gemm_stream(Runtime& rt, Tensor out, const Tensor& a, const Tensor& 
     check_launch(rc, "gemm_bf16_stream");
 }
 
-static bool gemm_tc(Runtime& rt, Tensor out, const Tensor& a, const Tensor& w, int epilogue = -1) {
+static bool gemm_tc(Runtime& rt, Tensor out, const Tensor& a, const Tensor& w, int epilogue = -1, float limit = 0.f) {
     if (epilogue < 0) epilogue = out.dtype == F32 ? TC_OUT_F32 : TC_OUT_BF16;
-    if (epilogue != TC_OUT_SWIGLU && epilogue != TC_OUT_GEGLU) {
+    if (epilogue == TC_OUT_BF16 || epilogue == TC_OUT_F32) {
         // few 256 x 256 tiles for the device's CTA pairs (a portion of a prompt): the K range in parts, then their sum
         const int M = (int)rows(a), N = (int)rows(w), K = (int)cols(a);
         const int n_splits = imp_gemm_bf16_tc_splits(M, N, K);
@@ -123,7 +124,7 @@ static bool gemm_tc(Runtime& rt, Tensor out, const Tensor& a, const Tensor& w, i
             rt.arena->restore(mark);
         }
     }
-    const int rc = imp_gemm_bf16_tc(out.data, out.stride0, epilogue, a.data, a.stride0, w.data, w.stride0, (int)rows(a),
+    const int rc = imp_gemm_bf16_tc_act(out.data, out.stride0, epilogue, limit, a.data, a.stride0, w.data, w.stride0, (int)rows(a),
                                     (int)rows(w), (int)cols(a), rt.status, rt.stream);
     if (rc == -2) return false;
     ++rt.launches;
@@ -131,12 +132,12 @@ static bool gemm_tc(Runtime& rt, Tensor out, const Tensor& a, const Tensor& w, i
     return true;
 }
 
-static bool gemm_tc_swap(Runtime& rt, Tensor out, const Tensor& a, const Tensor& w, int epilogue = -1) {
+static bool gemm_tc_swap(Runtime& rt, Tensor out, const Tensor& a, const Tensor& w, int epilogue = -1, float limit = 0.f) {
     if (epilogue < 0) epilogue = out.dtype == F32 ? TC_OUT_F32 : TC_OUT_BF16;
     const int M = (int)rows(a), N = (int)rows(w), K = (int)cols(a);
     const int64_t n_scratch = imp_gemm_bf16_tc_swap_scratch_floats(M, N, K, epilogue);
     float* scratch = n_scratch > 0 ? (float*)rt.arena->alloc((size_t)n_scratch * 4) : nullptr;
-    const int rc = imp_gemm_bf16_tc_swap(out.data, out.stride0, epilogue, a.data, a.stride0, w.data, w.stride0, M, N, K, scratch,
+    const int rc = imp_gemm_bf16_tc_swap_act(out.data, out.stride0, epilogue, limit, a.data, a.stride0, w.data, w.stride0, M, N, K, scratch,
                                          rt.status, rt.stream);
     if (rc == -2) return false;
     rt.launches += n_scratch > 0 ? 2 : 1;
@@ -159,13 +160,23 @@ static bool gemm_tc_swap_partials(Runtime& rt, Tensor out, const Tensor& a, cons
     return true;
 }
 
-Tensor summed(Runtime& rt, const Branch& b) {
-    if (b.split()) {
-        const int epi = b.t.dtype == F32 ? TC_OUT_F32 : TC_OUT_BF16;
+// A summand's tensor, its unsummed parts or its routed rows added up into it.
+static void sum_term(Runtime& rt, const Tensor& t, const float* parts, int n_splits, const RoutedRows& r) {
+    if (parts) {
+        const int epi = t.dtype == F32 ? TC_OUT_F32 : TC_OUT_BF16;
         ++rt.launches;
-        check_launch(imp_gemm_bf16_tc_swap_sum(b.t.data, b.t.stride0, epi, b.parts, (int)rows(b.t), (int)cols(b.t), b.n_splits, rt.stream),
-                     "gemm_bf16_tc_swap_sum");
+        check_launch(imp_gemm_bf16_tc_swap_sum(t.data, t.stride0, epi, parts, (int)rows(t), (int)cols(t), n_splits, rt.stream), "gemm_bf16_tc_swap_sum");
     }
+    if (r.y) {
+        need(contiguous(t), "summed: routed rows are added into a dense tensor");
+        ++rt.launches;
+        check_launch(imp_moe_combine(t.data, r.y, r.pair_row, r.wts, (int)rows(t), r.top, nullptr, nullptr, (int)cols(t), t.dtype == F32 ? 0 : 1, rt.stream),
+                     "moe_combine");
+    }
+}
+
+Tensor summed(Runtime& rt, const Branch& b) {
+    sum_term(rt, b.t, b.parts, b.n_splits, b.rows);
     if (b.own_norm.weight && !b.empty()) {
         need(contiguous(b.t), "summed: a branch with a norm of its own must be dense");
         ++rt.launches;
@@ -176,6 +187,14 @@ Tensor summed(Runtime& rt, const Branch& b) {
     if (b.col_scale && !b.empty()) {
         ++rt.launches;
         check_launch(imp_scale_columns(b.t.data, b.t.stride0, (int)rows(b.t), (int)cols(b.t), b.col_scale, b.t.dtype, rt.stream), "scale_columns");
+    }
+    if (!b.second.empty()) sum_term(rt, b.second.t, b.second.parts, b.second.n_splits, b.second.rows);
+    if (!b.empty() && (b.mult != 1.f || !b.second.empty())) {
+        need(contiguous(b.t) && (b.second.empty() || contiguous(b.second.t)), "summed: the two summands of a branch must be dense");
+        ++rt.launches;
+        check_launch(imp_scaled_sum(b.t.data, b.t.data, b.mult, b.second.empty() ? nullptr : b.second.t.data, b.mult, nullptr, 0.f, (int)rows(b.t),
+                                    (int)cols(b.t), b.t.dtype, rt.stream),
+                     "scaled_sum");
     }
     return b.t;
 }
@@ -237,17 +256,17 @@ Branch linear(Runtime& rt, Tensor out, const Tensor& x, const Tensor& w, bool ma
     return Branch::of(out);
 }
 
-void linear_gated(Runtime& rt, Tensor out, const Tensor& x, const Tensor& w, int act) {
+void linear_gated(Runtime& rt, Tensor out, const Tensor& x, const Tensor& w, GatedAct act) {
     const int64_t M = M_of(x), F = cols(out);
     if (M == 0) return;
-    need(act == 0 || act == 1, "linear_gated: unknown activation");
-    const int epi = act == 0 ? TC_OUT_SWIGLU : TC_OUT_GEGLU;
+    need(act.kind >= 0 && act.kind <= 2, "linear_gated: unknown activation");
+    const int epi = act.kind == 0 ? TC_OUT_SWIGLU : act.kind == 1 ? TC_OUT_GEGLU : TC_OUT_CLIPGLU;
     const bool bf16 = x.dtype == BF16 && w.dtype == BF16 && out.dtype == BF16;
     const bool lib = use_library_gemm();
-    if (bf16 && M > stream_m_max() && M <= SMALL_M_MAX && !lib && gemm_tc_swap(rt, out, x, w, epi)) return;
+    if (bf16 && M > stream_m_max() && M <= SMALL_M_MAX && !lib && gemm_tc_swap(rt, out, x, w, epi, act.limit)) return;
     if (bf16 && M <= SMALL_M_MAX) {
         const int rc = imp_gemm_bf16_stream_gated(out.data, out.stride0, x.data, x.stride0, w.data, w.stride0, (int)M, (int)(2 * F),
-                                                  (int)cols(x), act, rt.stream);
+                                                  (int)cols(x), act.kind, act.limit, rt.stream);
         if (rc != -2) {
             ++rt.launches;
             check_launch(rc, "gemm_bf16_stream_gated");
@@ -255,12 +274,25 @@ void linear_gated(Runtime& rt, Tensor out, const Tensor& x, const Tensor& w, int
         }
     }
     if (bf16 && !lib) {
-        if (M <= TC_SWAP_MAX_M && gemm_tc_swap(rt, out, x, w, epi)) return;
-        if (gemm_tc(rt, out, x, w, epi)) return;
+        if (M <= TC_SWAP_MAX_M && gemm_tc_swap(rt, out, x, w, epi, act.limit)) return;
+        if (gemm_tc(rt, out, x, w, epi, act.limit)) return;
     }
     Tensor gu = rt.empty(M, 2 * F, x.dtype);
     linear(rt, gu, x, w);
     gated_act(rt, out, gu, SWIGLU_INTERLEAVE, act);
+}
+
+void linear_relu2(Runtime& rt, Tensor out, const Tensor& x, const Tensor& w) {
+    const int64_t M = M_of(x);
+    if (M == 0) return;
+    need(contiguous(out), "linear_relu2: the output must be dense");
+    if (x.dtype == BF16 && w.dtype == BF16 && out.dtype == BF16 && !use_library_gemm() && M > stream_m_max()) {
+        if (M <= TC_SWAP_MAX_M && gemm_tc_swap(rt, out, x, w, TC_OUT_RELU2)) return;
+        if (M > TC_SWAP_MAX_M && gemm_tc(rt, out, x, w, TC_OUT_RELU2)) return;
+    }
+    linear(rt, out, x, w);
+    ++rt.launches;
+    check_launch(imp_act_rows(out.data, out.data, out.stride0, (int)M, (int)cols(out), 2, out.dtype, rt.stream), "act_rows");
 }
 
 void linear_swiglu(Runtime& rt, Tensor out, const Tensor& x, const Tensor& w) { linear_gated(rt, out, x, w, 0); }
@@ -275,7 +307,7 @@ void add_rmsnorm(Runtime& rt, Tensor h, const Branch& branch, const Tensor& weig
     need(rows_idx ? n_out == n_rows : n_out == rows(h), "add_rmsnorm: out has the wrong number of rows");
     const int write_h = rows_idx ? 0 : 1;
     const void* plain = nullptr;
-    if (branch.col_scale) {
+    if (branch.col_scale || branch.own_norm.weight || branch.compound()) {
         plain = summed(rt, branch).data;     // this norm adds plain tensors: the factor per column is applied first
     } else if (branch.split()) {
         need(rows(branch.t) == rows(h) && cols(branch.t) == d && branch.t.dtype == out.dtype, "add_rmsnorm: branch shape or type");

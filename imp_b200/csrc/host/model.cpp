@@ -82,7 +82,45 @@ void Diagnostics::dump_stream(Step& st, int run, const Tensor& h, const Branch& 
     std::vector<float> hs(n);
     IMP_CUDA(cudaMemcpyAsync(hs.data(), h.data, n * 4, cudaMemcpyDeviceToHost, st.rt->stream));
     IMP_CUDA(cudaStreamSynchronize(st.rt->stream));
-    if (!pending.empty() && !pending.split()) {
+    if (!pending.empty() && (pending.compound() || pending.second.parts)) {
+        // two summands with a factor: worked out in 32-bit beside the tensors, which stay as the next norm expects them
+        auto add_term = [&](const Tensor& t, const float* parts, int n_splits, const RoutedRows& r) {
+            if (!t.data) return;
+            const size_t el = elem_size(t.dtype), T = n / d;
+            auto widen1 = [&](const std::vector<char>& bytes, size_t i) {
+                float v;
+                if (t.dtype == F32) {
+                    v = ((const float*)bytes.data())[i];
+                } else {
+                    const uint32_t bits = (uint32_t)((const uint16_t*)bytes.data())[i] << 16;
+                    memcpy(&v, &bits, 4);
+                }
+                return v;
+            };
+            auto fetch = [&](const void* src, size_t bytes) {
+                std::vector<char> out(bytes);
+                IMP_CUDA(cudaMemcpyAsync(out.data(), src, bytes, cudaMemcpyDeviceToHost, st.rt->stream));
+                IMP_CUDA(cudaStreamSynchronize(st.rt->stream));
+                return out;
+            };
+            if (parts) {
+                const std::vector<char> p = fetch(parts, (size_t)n_splits * n * 4);
+                for (int s = 0; s < n_splits; ++s)
+                    for (size_t i = 0; i < n; ++i) hs[i] += pending.mult * ((const float*)p.data())[(size_t)s * n + i];
+            } else if (r.y) {
+                const size_t P = T * (size_t)r.top;
+                const std::vector<char> y = fetch(r.y, P * d * el), row = fetch(r.pair_row, P * 4), w = fetch(r.wts, P * 4);
+                for (size_t q = 0; q < P; ++q)
+                    for (size_t c = 0; c < d; ++c)
+                        hs[q / (size_t)r.top * d + c] += pending.mult * ((const float*)w.data())[q] * widen1(y, (size_t)((const int32_t*)row.data())[q] * d + c);
+            } else {
+                const std::vector<char> v = fetch(t.data, n * el);
+                for (size_t i = 0; i < n; ++i) hs[i] += pending.mult * widen1(v, i);
+            }
+        };
+        add_term(pending.t, pending.parts, pending.n_splits, pending.rows);
+        add_term(pending.second.t, pending.second.parts, pending.second.n_splits, pending.second.rows);
+    } else if (!pending.empty() && !pending.split()) {
         std::vector<char> raw(n * elem_size(pending.t.dtype));
         std::vector<float> scale(d, 1.f);
         IMP_CUDA(cudaMemcpyAsync(raw.data(), pending.t.data, raw.size(), cudaMemcpyDeviceToHost, st.rt->stream));
@@ -334,6 +372,12 @@ void DeviceModel::finish_build() {
         const bool next_takes = j + 1 < order_.size() ? blocks_[(size_t)order_[j + 1]]->takes_column_scale() : final_norm_->takes_column_scale();
         scale_ok[(size_t)order_[j]] = scale_ok[(size_t)order_[j]] && next_takes;
     }
+    // For one of two summands with a constant factor.
+    std::vector<bool> pair_ok(blocks_.size(), true);
+    for (size_t j = 0; j < order_.size(); ++j) {
+        const bool next_takes = j + 1 < order_.size() ? blocks_[(size_t)order_[j + 1]]->takes_branch_pair() : final_norm_->takes_branch_pair();
+        pair_ok[(size_t)order_[j]] = pair_ok[(size_t)order_[j]] && next_takes;
+    }
     // And for one that carries a norm of its own.
     std::vector<bool> norm_ok(blocks_.size(), true);
     for (size_t j = 0; j < order_.size(); ++j) {
@@ -343,6 +387,7 @@ void DeviceModel::finish_build() {
     for (size_t i = 0; i < blocks_.size(); ++i) {
         blocks_[i]->norm_pending = norm_ok[i];
         blocks_[i]->scale_pending = scale_ok[i];
+        blocks_[i]->pair_pending = pair_ok[i];
         keep_embedding_ = keep_embedding_ || blocks_[i]->wants_embedding();
     }
     // Cache needs: one entry per mixer of every run position (one entry, possibly empty, for a position with a
@@ -374,6 +419,16 @@ void DeviceModel::finish_build() {
             cache_specs_.push_back(CacheSpec());
             cache_position_.push_back(it->second);
             cache_count_.push_back(1);
+        }
+    }
+    // An embedding that owns state has the last entry.
+    const PartClass& ec = part_class("embedding", plan_.embedding.kind);
+    if (ec.cache_spec) {
+        const CacheSpec es = ec.cache_spec(plan_.embedding.params);
+        if (es.kind == CacheSpec::Paged) fail(IMP_ERROR_UNSUPPORTED, "an embedding may own state, not a paged cache");
+        if (es.kind == CacheSpec::State) {
+            embedding_cache_position_ = (int)cache_specs_.size();
+            cache_specs_.push_back(es);
         }
     }
     cache_first_.clear();
@@ -422,6 +477,12 @@ void DeviceModel::attach_cache(CacheManager* cache) {
         own += owns ? cache_count_[j] : 1;
     }
     (void)own;
+    if (embedding_cache_position_ >= 0) {
+        embedding_cache_ = LayerCache();
+        embedding_cache_.view = cache->layer_view(embedding_cache_position_, rt_->dtype);
+        embedding_cache_.view.writes = 1;
+        embedding_cache_.group = cache->layer_ref()[(size_t)embedding_cache_position_].group;
+    }
 }
 
 Tensor DeviceModel::forward(Step& st) {
@@ -433,7 +494,7 @@ Tensor DeviceModel::forward(Step& st) {
     st.diag = diag_.get();
     st.layer = -1;
     if (diag_) diag_->begin(st);
-    Tensor h = embedding_->forward(st);
+    Tensor h = embedding_->forward(st, embedding_cache_position_ >= 0 ? &embedding_cache_ : nullptr);
     stage(st, "embedding", h);
     st.embedding_out = Tensor{};
     if (keep_embedding_) {

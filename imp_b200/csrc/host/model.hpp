@@ -87,6 +87,8 @@ private:
     std::vector<int> order_, cache_position_, cache_count_, cache_first_;
     std::vector<CacheSpec> cache_specs_;
     std::vector<LayerCache> layer_caches_;
+    int embedding_cache_position_ = -1;          // the embedding's entry among cache_specs_, if it owns state
+    LayerCache embedding_cache_;
     std::vector<TilingSpec> tilings_;
     bool graph_safe_ = true, keep_embedding_ = false;
     CacheManager* cache_ = nullptr;

@@ -28,9 +28,17 @@ Tensor cat_rows(Runtime& rt, WeightStore& store, const std::vector<Tensor>& part
 Tensor to_float32(Runtime& rt, WeightStore& store, const Tensor& t);   // a 32-bit copy of a small weight
 
 void swiglu(Runtime& rt, Tensor out, const Tensor& gate_up, int interleave);
-// The same with the activation chosen: act 0 silu, 1 gelu (tanh form).
-void gated_act(Runtime& rt, Tensor out, const Tensor& gate_up, int interleave, int act);
-void linear_gated(Runtime& rt, Tensor out, const Tensor& x, const Tensor& w_interleaved, int act);
+// The same with the activation chosen: 0 silu(g) u, 1 gelu(g) u (tanh form), 2 both clipped to `limit`:
+// g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit), u' = min(max(u, -limit), limit).
+struct GatedAct {
+    int kind;
+    float limit;
+    GatedAct(int k, float l = 0.f) : kind(k), limit(l) {}
+};
+void gated_act(Runtime& rt, Tensor out, const Tensor& gate_up, int interleave, GatedAct act);
+void linear_gated(Runtime& rt, Tensor out, const Tensor& x, const Tensor& w_interleaved, GatedAct act);
+// out = max(x w^T, 0)^2, in the product's epilogue where that kernel runs.
+void linear_relu2(Runtime& rt, Tensor out, const Tensor& x, const Tensor& w);
 void cast(Runtime& rt, Tensor dst, const Tensor& src);
 
 // The tensor a branch stands for (runs the summing kernel if its parts are still apart).

@@ -240,25 +240,33 @@ void Mixer::call(Step& st, ImpCall& c) {
     copy_out(st, summed(st, b), c.out);
 }
 void FeedForward::call(Step& st, ImpCall& c) {
-    const bool keep = defer_out;
+    const bool keep = defer_out, keep_rows = defer_rows;
     defer_out = false;
+    defer_rows = false;
     Branch b = forward(st, c.x);
     defer_out = keep;
+    defer_rows = keep_rows;
     copy_out(st, summed(st, b), c.out);
 }
 void Block::call(Step& st, ImpCall& c) {
     LayerCache lc;
     if (c.cache) lc.view = *c.cache;
-    const bool keep = defer_pending, keep_scale = scale_pending;
+    const bool keep = defer_pending, keep_scale = scale_pending, keep_pair = pair_pending;
     defer_pending = false;
     scale_pending = false;
+    pair_pending = false;
     Branch b = forward(st, c.h, branch_of(c.branch), c.cache ? &lc : nullptr);
     defer_pending = keep;
     scale_pending = keep_scale;
+    pair_pending = keep_pair;
     c.has_out = b.empty() ? 0 : 1;
     if (!b.empty()) copy_out(st, summed(st, b), c.out);
 }
-void Embedding::call(Step& st, ImpCall& c) { copy_out(st, forward(st), c.h); }
+void Embedding::call(Step& st, ImpCall& c) {
+    LayerCache lc;
+    if (c.cache) lc.view = *c.cache;
+    copy_out(st, forward(st, c.cache ? &lc : nullptr), c.h);
+}
 void Head::call(Step& st, ImpCall& c) { copy_out(st, forward(st, c.x), c.out); }
 
 }  // namespace imp

@@ -14,7 +14,7 @@
 //   feed_forward  forward(step, x) -> branch output [T, hidden].
 //   block         part_slots(params) (class level): the parts it arranges, by slot name;
 //                 forward(step, h, pending, cache) -> the branch it leaves pending.
-//   embedding     forward(step) -> [T, hidden] float32 stream.
+//   embedding     forward(step, cache) -> [T, hidden] float32 stream; with a cache_spec (class level) it owns state, too.
 //   head          forward(step, x_rows) -> [R, vocab] float32 logits.
 //
 // Unsummed branch outputs.  A matrix product of few rows is cut over the contraction and leaves
@@ -134,14 +134,35 @@ struct BranchNorm {
     float eps = 0.f;
     int dtype = F32;                // of weight and bias
 };
+// Rows of routed experts that nobody has added up yet: row t of the branch is sum_k wts[t, k] * y[pair_row[t, k]].
+struct RoutedRows {
+    const void* y = nullptr;        // dense [T * top, cols], in the branch tensor's type; null: the branch is not of this form
+    const int* pair_row = nullptr;  // [T, top]
+    const float* wts = nullptr;     // [T, top]
+    int top = 0;
+};
+// One more summand of a branch: a tensor, its unsummed parts, or rows of routed experts (`t` then is where the sum belongs).
+struct BranchTerm {
+    Tensor t{};
+    float* parts = nullptr;
+    int n_splits = 0;
+    RoutedRows rows{};
+    bool empty() const { return t.data == nullptr; }
+};
 struct Branch {
     Tensor t{};
     float* parts = nullptr;
     int n_splits = 0;
     const float* col_scale = nullptr;   // float32 [cols], or null
     BranchNorm own_norm{};
+    RoutedRows rows{};                  // of `t`; only towards whoever asked for it (FeedForward::defer_rows)
+    // A branch of two sublayers side by side and with a constant factor stands for mult * (this + second): towards a norm that
+    // says takes_branch_pair(); summed() works it out for everyone else.
+    float mult = 1.f;
+    BranchTerm second{};
     bool empty() const { return t.data == nullptr; }
     bool split() const { return parts != nullptr; }
+    bool compound() const { return rows.y || mult != 1.f || !second.empty(); }
     static Branch of(const Tensor& t) { Branch b; b.t = t; return b; }
 };
 
@@ -159,6 +180,7 @@ struct Norm : Part {
     virtual bool takes_split_sum() const { return false; }
     virtual bool takes_column_scale() const { return false; }   // multiplies a branch's col_scale in while adding
     virtual bool takes_normed_branch() const { return false; }  // applies a branch's own_norm while adding
+    virtual bool takes_branch_pair() const { return false; }    // adds a branch's two summands, times its constant, itself
     // This norm as the own norm of a branch (a layer norm's weight, bias and eps); false: it cannot ride with a branch.
     virtual bool as_branch_norm(BranchNorm* out) const { (void)out; return false; }
     virtual Tensor add_norm(Step& st, Tensor h, const Branch& branch, const int32_t* rows = nullptr, int n_rows = 0) = 0;
@@ -195,6 +217,7 @@ struct Mixer : Part {
 struct FeedForward : Part {
     const char* category() const override { return "feed_forward"; }
     bool defer_out = false;
+    bool defer_rows = false;                             // may return rows of routed experts that are not added up (Branch::rows)
     virtual Branch forward(Step& st, Tensor x) = 0;
     void call(Step& st, ImpCall& c) override;
 };
@@ -207,6 +230,8 @@ struct Block : Part {
     virtual bool takes_column_scale() const { return false; }   // the pending it is given may carry a col_scale
     bool norm_pending = false;                           // set by the model: the pending it returns may carry a norm of its own
     virtual bool takes_normed_branch() const { return false; }  // the pending it is given may carry a norm of its own
+    bool pair_pending = false;                           // set by the model: the pending it returns may have two summands and a factor
+    virtual bool takes_branch_pair() const { return false; }    // the pending it is given may have two summands and a factor
     virtual bool wants_embedding() const { return false; }      // reads Step::embedding_out
     virtual Mixer* mixer() const { return nullptr; }     // the part that owns this layer's cache, if any
     // A block with several mixers names them in the order of its mixer slots; each owns a cache, and forward()
@@ -222,7 +247,7 @@ struct Block : Part {
 
 struct Embedding : Part {
     const char* category() const override { return "embedding"; }
-    virtual Tensor forward(Step& st) = 0;
+    virtual Tensor forward(Step& st, LayerCache* cache) = 0;   // cache: its state, null where its class declares none
     void call(Step& st, ImpCall& c) override;
 };
 
@@ -268,7 +293,7 @@ struct BuildArgs {
 
 struct PartClass {
     std::function<TensorSpecs(const Json& params)> tensor_specs;      // may be empty: no tensors
-    std::function<CacheSpec(const Json& params)> cache_spec;          // mixers
+    std::function<CacheSpec(const Json& params)> cache_spec;          // mixers, and embeddings that own state
     std::function<std::vector<Slot>(const Json& params)> part_slots;  // blocks
     std::function<Part*(BuildArgs&)> create;
 };
@@ -282,6 +307,7 @@ void ensure_builtin_parts();   // registers the library's own kinds once
 void register_mixer_parts();    // parts_mixers.cpp: the kinds beyond plain attention (called by ensure_builtin_parts)
 void register_recurrent_parts();   // parts_recurrent.cpp: retention, the delta rules over the general scan, attention with gated heads, the post-norm block
 void register_sandwich_parts();    // parts_sandwich.cpp: the block with a norm before and after each sublayer, the short convolution on a sublayer's input, differential attention, the polynomial feed-forward
+void register_parallel_parts();   // parts_parallel.cpp: the norm without statistics, the embedding with a table of token pairs, the block whose sublayers share one norm
 void register_routed_parts();   // parts_routed.cpp: layer norm, latent attention, wkv, routed experts, blocks with scaled branches
 
 // Builds parts and owns them.  Parts without tensors are shared between equal specs.

@@ -206,11 +206,12 @@ struct GQAAttention : Mixer {
 // ------------------------------------------------------------------------------- feed-forward
 // down( act(x Wg^T) * (x Wu^T) ), activation in 32-bit (src/graph/executor_forward.cu:933-951,
 // 1124-1140; src/compute/activation.cu:67-87).  params: hidden_size, intermediate_size, activation ("silu", the default,
-// or "gelu_tanh": 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))).  Registered as "swiglu" and as "gated_mlp".
+// "gelu_tanh": 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))), or "clipped": with `limit`, g = min(gate, limit) and
+// u = min(max(up, -limit), limit) become g sigmoid(1.702 g) (u + 1)).  Registered as "swiglu" and as "gated_mlp".
 struct SwiGLU : FeedForward {
     int64_t f;
     bool interleaved;
-    int act = 0;   // 0 silu, 1 gelu (tanh form)
+    GatedAct act{0};
     Tensor w_gu, w_down;
     static TensorSpecs specs(const Json& p) {
         const int64_t d = need_int(p, "hidden_size", "swiglu"), f = need_int(p, "intermediate_size", "swiglu");
@@ -223,8 +224,14 @@ struct SwiGLU : FeedForward {
     explicit SwiGLU(BuildArgs& a) {
         f = need_int(a.params, "intermediate_size", "swiglu");
         const std::string an = a.params.get_string("activation", "silu");
-        if (an != "silu" && an != "gelu_tanh") fail(IMP_ERROR_INVALID_MODEL, "gated feed-forward: unknown activation '" + an + "' (known: silu, gelu_tanh)");
-        act = an == "silu" ? 0 : 1;
+        if (an != "silu" && an != "gelu_tanh" && an != "clipped")
+            fail(IMP_ERROR_INVALID_MODEL, "gated feed-forward: unknown activation '" + an + "' (known: silu, gelu_tanh, clipped)");
+        act = GatedAct(an == "silu" ? 0 : an == "gelu_tanh" ? 1 : 2);
+        if (act.kind == 2) {
+            const Json* l = a.params.find("limit");
+            if (!l || !l->is_number() || !(l->as_double() > 0)) fail(IMP_ERROR_INVALID_MODEL, "gated feed-forward: the clipped activation needs a positive 'limit'");
+            act.limit = (float)l->as_double();
+        }
         Runtime& rt = *a.rt;
         Tensor gate = a.tensor("gate_proj"), up = a.tensor("up_proj");
         // Gate and up rows alternate in runs of 8 so that one kernel can produce the activation from the fused
@@ -297,7 +304,7 @@ struct TokenEmbedding : Embedding {
         s.emplace_back("weight", TensorSpec{{need_int(p, "vocab_size", "token_embedding"), need_int(p, "hidden_size", "token_embedding")}});
         return s;
     }
-    Tensor forward(Step& st) override {
+    Tensor forward(Step& st, LayerCache*) override {
         Tensor out = st.rt->empty(st.T(), cols(weight), F32, /*step=*/true);
         embedding(*st.rt, out, weight, st.view.token_ids, st.T(), scale);
         return out;
@@ -361,6 +368,7 @@ void ensure_builtin_parts() {
         register_routed_parts();
         register_sandwich_parts();
         register_recurrent_parts();
+        register_parallel_parts();
     });
 }
 

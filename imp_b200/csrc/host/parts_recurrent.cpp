@@ -1,5 +1,5 @@
-// Part kinds: three recurrent mixers over the general scan of csrc/delta_rule.cu (retention, the generalised delta
-// rule, the delta rule with a decay per key channel), softmax attention whose heads are normalised, rotated in part,
+// Part kinds: four recurrent mixers over the general scan of csrc/delta_rule.cu (retention, gated linear attention, the generalised
+// delta rule, the delta rule with a decay per key channel), softmax attention whose heads are normalised, rotated in part,
 // scaled, masked by chunks and gated, and a post-norm block (the normalised sum is the stream) that holds one mixer
 // or two side by side.  Every size and constant is a parameter; no kind knows which model it is in.
 #include <cmath>
@@ -166,6 +166,104 @@ struct Retention : Mixer {
             check_launch(imp_lsr_output_row(y.data, b.o, gate.data, gate.stride0, wn, gate_act, eps, (int)T, H * Dv, rt.dtype, rt.stream), "lsr_output_row");
         else
             check_launch(imp_gdr_output_ex(y.data, b.o, gate.data, gate.stride0, wn, wn ? Dv : 0, gate_act, eps, (int)T, H, Dv, rt.dtype, rt.stream), "gdr_output");
+        return linear(rt, rt.empty(T, rows(w_o)), y, w_o, defer_out);
+    }
+};
+
+// ------------------------------------------------------------------------------------ gated linear attention
+// q = query_scale W_q x, k = W_k x (H heads of D), v = W_v x (H heads of Dv); a decay per head and key channel,
+// alpha = sigmoid(W_a2 (W_a1 x) + b_a)^(1/tau);
+//   S <- diag(alpha) S + k v^T;  o = S^T q;  y = o / rms(o) per head * w_norm [Dv] * silu(W_g x);  out = W_o y.
+// Portions run prepare, scan (the general scan with a decay per channel and nothing removed) and output kernels; a step of single
+// tokens is one kernel from the projections to y (csrc/delta_rule.cu).
+// State per request: S (H heads of D x Dv, float32), zero at the start.
+// params: hidden_size, num_heads, key_dim, value_dim, tau, query_scale (default key_dim^-1/2), norm_eps, decay_rank (0 or absent: the
+//         rows of the checkpoint's W_a1).
+struct GatedLinearAttention : Mixer {
+    int H, D, Dv, rank;
+    float eps, tau, q_scale;
+    Tensor w_in, w_o, w2t, a_bias, out_norm;   // the last three float32
+
+    struct Sizes {
+        int64_t d, H, D, Dv;
+    };
+    static Sizes sizes(const Json& p) {
+        const char* me = "gated_linear_attention";
+        Sizes s{need_int(p, "hidden_size", me), need_int(p, "num_heads", me), need_int(p, "key_dim", me), need_int(p, "value_dim", me)};
+        if (s.H <= 0 || s.D <= 0 || s.D > 256 || s.Dv <= 0) fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": key_dim must lie in (0, 256], heads and value_dim be positive");
+        return s;
+    }
+    static TensorSpecs specs(const Json& p) {
+        const Sizes z = sizes(p);
+        const int64_t r = p.get_int("decay_rank", 0);
+        TensorSpecs s;
+        s.emplace_back("q_proj", TensorSpec{{z.H * z.D, z.d}});
+        s.emplace_back("k_proj", TensorSpec{{z.H * z.D, z.d}});
+        s.emplace_back("v_proj", TensorSpec{{z.H * z.Dv, z.d}});
+        s.emplace_back("gate_proj", TensorSpec{{z.H * z.Dv, z.d}});
+        s.emplace_back("decay_down", TensorSpec{{r > 0 ? r : -1, z.d}});
+        s.emplace_back("decay_up", TensorSpec{{z.H * z.D, r > 0 ? r : -1}});
+        s.emplace_back("decay_bias", TensorSpec{{z.H * z.D}, "vector", "normal"});
+        s.emplace_back("out_norm", TensorSpec{{z.Dv}, "norm", "one_plus_normal"});
+        s.emplace_back("o_proj", TensorSpec{{z.d, z.H * z.Dv}});
+        return s;
+    }
+    static CacheSpec cache(const Json& p) {
+        const Sizes z = sizes(p);
+        return scan_state(z.H, z.D, z.Dv);
+    }
+    explicit GatedLinearAttention(BuildArgs& a) {
+        const char* me = "gated_linear_attention";
+        const Sizes z = sizes(a.params);
+        H = (int)z.H, D = (int)z.D, Dv = (int)z.Dv;
+        eps = (float)a.params.get_double("norm_eps", 1e-6);
+        tau = (float)need_double(a.params, "tau", me);
+        if (!(tau > 0)) fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": tau must be positive");
+        q_scale = (float)a.params.get_double("query_scale", 1.0 / std::sqrt((double)D));
+        Runtime& rt = *a.rt;
+        const Tensor w_1 = a.tensor("decay_down"), w_2 = a.tensor("decay_up");
+        rank = (int)rows(w_1);
+        if (rows(w_1) != cols(w_2)) fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": the two decay matrices do not share their inner size");
+        w_in = cat_rows_padded(rt, *a.store, {a.tensor("q_proj"), a.tensor("k_proj"), a.tensor("v_proj"), a.tensor("gate_proj"), w_1});
+        w_o = a.tensor("o_proj");
+        // W_a2 transposed and in 32-bit: its product is made by the kernels that use the decay
+        const Tensor w_2f = to_float32(rt, *a.store, w_2);
+        w2t = a.store->alloc(F32, {rank, z.H * z.D});
+        check_launch(imp_transpose_groups(w2t.data, w_2f.data, 1, (int)(z.H * z.D), rank, 0, rt.stream), "transpose_groups");
+        a_bias = to_float32(rt, *a.store, a.tensor("decay_bias"));
+        out_norm = to_float32(rt, *a.store, a.tensor("out_norm"));
+        IMP_CUDA(cudaStreamSynchronize(rt.stream));
+        a.store->release(w_2f.data);
+        for (const char* n : {"q_proj", "k_proj", "v_proj", "gate_proj", "decay_down", "decay_up", "decay_bias", "out_norm"}) a.drop(n);
+    }
+    Branch forward(Step& st, Tensor x, LayerCache* cache) override {
+        Runtime& rt = *st.rt;
+        if (!cache || cache->view.kind != 2 || cache->view.n_states < 1) fail(IMP_ERROR_INTERNAL, "gated_linear_attention runs against a state cache");
+        const int64_t T = rows(x);
+        float* S = (float*)cache->view.states[0].data;
+        Tensor proj = rt.empty(T, rows(w_in));
+        linear(rt, proj, x, w_in);
+        Tensor y = rt.empty(T, (int64_t)H * Dv);
+        int rc = -2;
+        if (st.decode_only())
+            rc = imp_gla_decode(proj.data, proj.stride0, (int)T, H, D, Dv, rank, (const float*)w2t.data, (const float*)a_bias.data, tau, q_scale,
+                                (const float*)out_norm.data, eps, S, st.view.state_slots, y.data, rt.dtype, rt.stream);
+        if (rc == -2) {
+            ScanBuffers b(rt, T, H, D, Dv, true, false);
+            rt.launches += 3;
+            check_launch(imp_gla_prepare(proj.data, proj.stride0, (int)T, H, D, Dv, rank, (const float*)w2t.data, (const float*)a_bias.data, tau, q_scale,
+                                         b.q, b.kw, b.w, b.v, b.scal, rt.dtype, rt.stream),
+                         "gla_prepare");
+            check_launch(imp_lsr_scan(3, b.kw, b.q, b.w, nullptr, nullptr, b.v, b.scal, nullptr, S, b.o, st.view.q_start, st.view.state_slots, st.B(), D,
+                                      H, Dv, rt.stream),
+                         "lsr_scan");
+            const Tensor gate = col_slice(proj, (int64_t)2 * H * D + (int64_t)H * Dv, (int64_t)H * Dv);
+            check_launch(imp_gdr_output_ex(y.data, b.o, gate.data, gate.stride0, (const float*)out_norm.data, 0, 0, eps, (int)T, H, Dv, rt.dtype, rt.stream),
+                         "gdr_output");
+        } else {
+            ++rt.launches;
+            check_launch(rc, "gla_decode");
+        }
         return linear(rt, rt.empty(T, rows(w_o)), y, w_o, defer_out);
     }
 };
@@ -664,6 +762,9 @@ void register_recurrent_parts() {
     PartClass ret = class_of<Retention>(&Retention::specs);
     ret.cache_spec = &Retention::cache;
     register_part_class("mixer", "retention", ret, true);
+    PartClass gla = class_of<GatedLinearAttention>(&GatedLinearAttention::specs);
+    gla.cache_spec = &GatedLinearAttention::cache;
+    register_part_class("mixer", "gated_linear_attention", gla, true);
     PartClass gd = class_of<GeneralDelta>(&GeneralDelta::specs);
     gd.cache_spec = &GeneralDelta::cache;
     register_part_class("mixer", "general_delta", gd, true);

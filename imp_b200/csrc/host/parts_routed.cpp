@@ -127,23 +127,35 @@ struct LayerNorm : Norm {
 // output are not used), and W_uv maps each head's latent-space result to its values.  Per token the cache holds
 // C + R numbers whatever the number of heads.
 //
+// Options: no query latent (`q_rank` 0: q = W_q x, a tensor `q_proj`); a sliding window (`window`: the last so many keys, 0 all);
+// the rotation's pairing (`rot_pairing`: "halves" i, i + rot_dims/2 | "neighbours" 2i, 2i + 1); the heads' values multiplied by
+// sigmoid(W_g x) before W_o (`out_gate`: a tensor `gate_proj`); the cached vector padded with zeros to a multiple of 16 where the
+// tensor-core kernels then take it (`pad_cache`).  Without a query latent all of x's projections are one product.
+//
 // params: hidden_size, num_heads, head_dim (plain), rot_dim, value_dim, kv_rank, q_rank, scale, norm_eps, rot_base,
-//         rot_dims (entries of the rotated part that are rotated: even, at most rot_dim), max_positions.
+//         rot_dims (entries of the rotated part that are rotated: even, at most rot_dim), max_positions, window, rot_pairing,
+//         out_gate, pad_cache.
 struct LatentAttention : Mixer {
-    int H, D, R, Dv, C, Q, rot_dims;
+    int H, D, R, Dv, C, Q, L, rot_dims, pairing = 0;   // L: the length of a cached vector
+    bool gated = false;
     float eps;
     AttentionGeometry g;
+    int64_t gate_col = 0;
     Tensor w_down, w_uq, w_ukT, w_uv, w_o, n_q, n_kv;
     Position* position = nullptr;
 
     struct Sizes {
-        int64_t d, H, D, R, Dv, C, Q;
+        int64_t d, H, D, R, Dv, C, Q, L;
     };
     static Sizes sizes(const Json& p) {
         const char* me = "latent_attention";
         Sizes s{need_int(p, "hidden_size", me), need_int(p, "num_heads", me), need_int(p, "head_dim", me), need_int(p, "rot_dim", me),
-                need_int(p, "value_dim", me), need_int(p, "kv_rank", me), need_int(p, "q_rank", me)};
-        if (s.H <= 0 || s.D <= 0 || s.R <= 0 || s.Dv <= 0 || s.C <= 0 || s.Q <= 0) fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": every size must be positive");
+                need_int(p, "value_dim", me), need_int(p, "kv_rank", me), need_int(p, "q_rank", me), 0};
+        s.L = s.C + s.R;
+        if (p.get_bool("pad_cache", false) && s.L <= 256) s.L = (s.L + 15) / 16 * 16;
+        if (s.H <= 0 || s.D <= 0 || s.R <= 0 || s.Dv <= 0 || s.C <= 0 || s.Q < 0) fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": every size must be positive");
+        if (s.Q > 0 && (s.L != s.C + s.R || p.get_string("rot_pairing", "halves") != "halves"))
+            fail(IMP_ERROR_UNSUPPORTED, std::string(me) + ": a query latent goes with rotated halves and an unpadded cache");
         if (s.C + s.R > 1024)
             fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": kv_rank + rot_dim = " + std::to_string(s.C + s.R) + " exceeds the attention kernels' 1024 (tensor cores up to 256)");
         return s;
@@ -151,19 +163,24 @@ struct LatentAttention : Mixer {
     static TensorSpecs specs(const Json& p) {
         const Sizes z = sizes(p);
         TensorSpecs s;
-        s.emplace_back("q_down", TensorSpec{{z.Q, z.d}});
-        s.emplace_back("q_norm", TensorSpec{{z.Q}, "norm", "one_plus_normal"});
-        s.emplace_back("q_up", TensorSpec{{z.H * (z.D + z.R), z.Q}});
+        if (z.Q > 0) {
+            s.emplace_back("q_down", TensorSpec{{z.Q, z.d}});
+            s.emplace_back("q_norm", TensorSpec{{z.Q}, "norm", "one_plus_normal"});
+            s.emplace_back("q_up", TensorSpec{{z.H * (z.D + z.R), z.Q}});
+        } else {
+            s.emplace_back("q_proj", TensorSpec{{z.H * (z.D + z.R), z.d}});
+        }
         s.emplace_back("kv_down", TensorSpec{{z.C + z.R, z.d}});
         s.emplace_back("kv_norm", TensorSpec{{z.C}, "norm", "one_plus_normal"});
         s.emplace_back("k_up", TensorSpec{{z.H * z.D, z.C}});
         s.emplace_back("v_up", TensorSpec{{z.H * z.Dv, z.C}});
+        if (p.get_bool("out_gate", false)) s.emplace_back("gate_proj", TensorSpec{{z.H * z.Dv, z.d}});
         s.emplace_back("o_proj", TensorSpec{{z.d, z.H * z.Dv}});
         return s;
     }
     static CacheSpec cache(const Json& p) {
         const Sizes z = sizes(p);
-        CacheSpec s = CacheSpec::paged(1, (int)(z.C + z.R), 0);
+        CacheSpec s = CacheSpec::paged(1, (int)z.L, (int)p.get_int("window", 0));
         s.keys_only = true;
         return s;
     }
@@ -171,32 +188,48 @@ struct LatentAttention : Mixer {
     explicit LatentAttention(BuildArgs& a) {
         const char* me = "latent_attention";
         const Sizes z = sizes(a.params);
-        H = (int)z.H, D = (int)z.D, R = (int)z.R, Dv = (int)z.Dv, C = (int)z.C, Q = (int)z.Q;
+        H = (int)z.H, D = (int)z.D, R = (int)z.R, Dv = (int)z.Dv, C = (int)z.C, Q = (int)z.Q, L = (int)z.L;
+        gated = a.params.get_bool("out_gate", false);
+        const std::string pr = a.params.get_string("rot_pairing", "halves");
+        if (pr != "neighbours" && pr != "halves") fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": unknown rot_pairing '" + pr + "' (known: neighbours, halves)");
+        pairing = pr == "neighbours" ? 1 : 0;
         rot_dims = (int)a.params.get_int("rot_dims", R);
         if (rot_dims < 2 || rot_dims % 2 || rot_dims > R)
             fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": rot_dims " + std::to_string(rot_dims) + " must be even and within rot_dim " + std::to_string(R));
         eps = (float)a.params.get_double("norm_eps", 1e-6);
-        g.hq = H, g.hkv = 1, g.dh = C + R, g.window = 0;
+        g.hq = H, g.hkv = 1, g.dh = L, g.window = (int)a.params.get_int("window", 0);
+        if (g.window < 0) fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": 'window' must not be negative");
         g.scale = (float)need_double(a.params, "scale", me);
         Runtime& rt = *a.rt;
-        // one product for both down-projections; its rows are padded to a multiple of 8
-        std::vector<Tensor> in = {a.tensor("q_down"), a.tensor("kv_down")};
-        const int64_t n = z.Q + z.C + z.R, pad = (8 - n % 8) % 8;
-        Tensor zeros{};
-        if (pad) {
-            zeros = a.store->alloc(in[0].dtype, {pad, z.d});
+        // one product for everything that reads x: [query latent or q | latent and rotated key part | gate], the gate starting on a
+        // multiple of 8 columns and the rows padded to one
+        std::vector<Tensor> in = {a.tensor(Q > 0 ? "q_down" : "q_proj"), a.tensor("kv_down")}, pads;
+        int64_t n = (Q > 0 ? z.Q : z.H * (z.D + z.R)) + z.C + z.R;
+        auto pad_to8 = [&] {
+            const int64_t pad = (8 - n % 8) % 8;
+            if (!pad) return;
+            Tensor zeros = a.store->alloc(in[0].dtype, {pad, z.d});
             IMP_CUDA(cudaMemsetAsync(zeros.data, 0, (size_t)numel(zeros) * elem_size(zeros.dtype), rt.stream));
             in.push_back(zeros);
+            pads.push_back(zeros);
+            n += pad;
+        };
+        pad_to8();
+        if (gated) {
+            gate_col = n;
+            in.push_back(a.tensor("gate_proj"));
+            n += z.H * z.Dv;
+            pad_to8();
         }
         w_down = cat_rows(rt, *a.store, in);
-        w_uq = a.tensor("q_up");
+        if (Q > 0) w_uq = a.tensor("q_up");
         w_uv = a.tensor("v_up");
         w_o = a.tensor("o_proj");
         // W_uk [H][D, C] -> [H][C, D]: the latent-space query is a product with W_uk's transpose
         const Tensor uk = a.tensor("k_up");
         w_ukT = a.store->alloc(uk.dtype, {z.H * z.C, z.D});
         check_launch(imp_transpose_groups(w_ukT.data, uk.data, H, D, C, uk.dtype == F32 ? 0 : 1, rt.stream), "transpose_groups");
-        n_q = to_float32(rt, *a.store, a.tensor("q_norm"));
+        if (Q > 0) n_q = to_float32(rt, *a.store, a.tensor("q_norm"));
         n_kv = to_float32(rt, *a.store, a.tensor("kv_norm"));
         Json pos = Json::object(), pp = Json::object();
         pos["kind"] = "rotary";
@@ -207,8 +240,8 @@ struct LatentAttention : Mixer {
         pos["params"] = pp;
         position = part_cast<Position>(a.factory->shared("position", pos), "a position encoding");
         IMP_CUDA(cudaStreamSynchronize(rt.stream));
-        if (pad) a.store->release(zeros.data);
-        for (const char* nme : {"q_down", "kv_down", "k_up", "q_norm", "kv_norm"}) a.drop(nme);
+        for (const Tensor& t : pads) a.store->release(t.data);
+        for (const char* nme : {"q_down", "q_proj", "kv_down", "gate_proj", "k_up", "q_norm", "kv_norm"}) a.drop(nme);
     }
 
     std::vector<TilingSpec> tilings() const override { return attention_tilings(); }
@@ -223,32 +256,55 @@ struct LatentAttention : Mixer {
         const int dt = rt.dtype == F32 ? 0 : 1;
         Tensor proj = rt.empty(T, rows(w_down));
         linear(rt, proj, x, w_down);
-        Tensor cq = rt.empty(T, Q);
-        ++rt.launches;
-        check_launch(imp_latent_prepare(proj.data, proj.stride0, (int)T, Q, C, R, (const float*)n_q.data, (const float*)n_kv.data, eps, cq.data,
-                                        cq.stride0, rot.cos, rot.sin, rot.rot_dim, rot.max_pos, st.view.positions, st.view.seq_of_token,
-                                        cv.block_table, cv.bt_stride, st.B(), cv.writes ? cv.k_pages : nullptr, cv.page_size, cv.num_pages, dt,
-                                        rt.status, rt.stream),
-                     "latent_prepare");
-        Tensor q = rt.empty(T, (int64_t)H * (D + R));
-        linear(rt, q, cq, w_uq);
-        const int64_t L = C + R;
-        Tensor q_lat = rt.empty(T, H * L);
-        rt.launches += 2;
+        const int64_t q_cols = Q > 0 ? Q : (int64_t)H * (D + R);
+        Tensor cq{}, q;
+        if (Q > 0) {
+            // the norms first: the query's product reads the normalised latent
+            cq = rt.empty(T, Q);
+            prepare(st, proj, Q, cq, Tensor{}, Tensor{}, rot, cv);
+            q = rt.empty(T, (int64_t)H * (D + R));
+            linear(rt, q, cq, w_uq);
+        } else {
+            q = col_slice(proj, 0, q_cols);
+        }
+        Tensor q_lat = rt.empty(T, (int64_t)H * L);
+        rt.launches += 1;
         check_launch(imp_grouped_gemm(q_lat.data, q_lat.stride0, L, q.data, q.stride0, D + R, nullptr, w_ukT.data, nullptr, (int64_t)C * D, D, nullptr,
                                       (int)T, C, D, H, 0, dt, rt.stream),
                      "grouped_gemm (latent query)");
-        check_launch(imp_latent_query_rope(q.data, q.stride0, (int)T, H, D, R, q_lat.data, q_lat.stride0, C, rot.cos, rot.sin, rot.rot_dim,
-                                           rot.max_pos, st.view.positions, dt, rt.status, rt.stream),
-                     "latent_query_rope");
-        Tensor attn = rt.empty(T, H * L);
+        if (Q > 0) {
+            ++rt.launches;
+            check_launch(imp_latent_query_rope(q.data, q.stride0, (int)T, H, D, R, q_lat.data, q_lat.stride0, C, rot.cos, rot.sin, rot.rot_dim,
+                                               rot.max_pos, st.view.positions, dt, rt.status, rt.stream),
+                         "latent_query_rope");
+        } else {
+            prepare(st, col_slice(proj, q_cols, C + R), 0, Tensor{}, q, q_lat, rot, cv);
+        }
+        Tensor attn = rt.empty(T, (int64_t)H * L);
         paged_attention(st, attn, q_lat, g, *cache, tiling_ids);
         Tensor o = rt.empty(T, (int64_t)H * Dv);
         ++rt.launches;
-        check_launch(imp_grouped_gemm(o.data, o.stride0, Dv, attn.data, attn.stride0, L, nullptr, w_uv.data, nullptr, (int64_t)Dv * C, C, nullptr,
-                                      (int)T, Dv, C, H, 0, dt, rt.stream),
+        const Tensor gate = gated ? col_slice(proj, gate_col, (int64_t)H * Dv) : Tensor{};
+        check_launch(imp_grouped_gemm_ex(o.data, o.stride0, Dv, attn.data, attn.stride0, L, nullptr, w_uv.data, nullptr, (int64_t)Dv * C, C, nullptr,
+                                         (int)T, Dv, C, H, 0, gated ? GROUPED_SIGMOID_GATE : GROUPED_PLAIN, gate.data, gate.stride0, dt, rt.stream),
                      "grouped_gemm (values)");
         return linear(rt, rt.empty(T, rows(w_o)), o, w_o, defer_out);
+    }
+    // Norms and rotations of `down` = [query latent (q_rank) | latent | rotated key part] and the cache write; with `q` also the
+    // rotated parts of the heads' queries, behind their latent-space queries in q_lat.
+    void prepare(Step& st, const Tensor& down, int q_rank, const Tensor& cq, const Tensor& q, const Tensor& q_lat, const Position::Rotary& rot,
+                 const ImpCacheView& cv) {
+        Runtime& rt = *st.rt;
+        const size_t el = elem_size(rt.dtype);
+        ++rt.launches;
+        check_launch(imp_latent_prepare_ex(down.data, down.stride0, (int)rows(down), q_rank, C, R, q_rank > 0 ? (const float*)n_q.data : nullptr,
+                                           (const float*)n_kv.data, eps, cq.data, cq.stride0, rot.cos, rot.sin, rot.rot_dim, pairing, rot.max_pos,
+                                           st.view.positions, st.view.seq_of_token, cv.block_table, cv.bt_stride, st.B(),
+                                           cv.writes ? cv.k_pages : nullptr, L, cv.page_size, cv.num_pages,
+                                           q.data ? (const char*)q.data + (size_t)D * el : nullptr, q.stride0, D + R,
+                                           q_lat.data ? (char*)q_lat.data + (size_t)C * el : nullptr, q_lat.stride0, H, rt.dtype == F32 ? 0 : 1,
+                                           rt.status, rt.stream),
+                     "latent_prepare");
     }
 };
 
@@ -354,7 +410,7 @@ struct Wkv : Mixer {
 };
 
 // --------------------------------------------------------------------------------------- routed experts
-// A mixture of gated feed-forward experts: router logits z = W_r x + b in 32-bit; the `top_k` experts with the largest
+// A mixture of feed-forward experts, gated by default: router logits z = W_r x + b in 32-bit; the `top_k` experts with the largest
 // logits are chosen, weighted by the softmax over the chosen logits; expert e is W_down_e (silu(W_gate_e x) * (W_up_e x)).
 // Optionally a shared expert of the same form runs for every token and is added times sigmoid(w_sg . x).
 // The experts' matrices are stacked at load; a step sorts its (token, choice) pairs by expert on the device and runs two
@@ -363,14 +419,17 @@ struct Wkv : Mixer {
 // Options: the router without a bias (`router_bias`: false); sigmoid scores, a chosen expert weighing its score times
 // `weight_scale`, not renormalised (`scores`: "sigmoid"; default "softmax" as above); experts in `num_groups` equal groups of
 // neighbours of which the `keep_groups` best (by the sum of a group's two largest scores) can be chosen from; a shared expert
-// that is added as it is (`shared_gate`: false).
+// that is added as it is (`shared_gate`: false); scores that are the softmax over all experts, a chosen expert weighing its score
+// (`scores`: "softmax_all"); a group counted by its largest score instead of the sum of two (`group_score`: "max", the default with
+// "softmax_all"; else "top2"); experts without a gate, W_down_e max(W_up_e x, 0)^2 (`expert`: "relu2"; default "swiglu"; no
+// shared expert then).  With `defer_rows` set, and no shared expert, the chosen experts' rows are handed on unsummed (Branch::rows).
 //
 // params: hidden_size, num_experts, top_k, expert_size, shared_size (0: no shared expert), router_bias, scores, weight_scale,
-//         num_groups, keep_groups, shared_gate.
+//         num_groups, keep_groups, group_score, shared_gate, expert.
 struct RoutedExperts : FeedForward {
     int64_t d, E, top, F, Fs;
-    bool has_bias = true, has_sgate = true;
-    int score_mode = 0, n_groups = 0, keep_groups = 0;
+    bool has_bias = true, has_sgate = true, gated_expert = true;
+    int score_mode = 0, n_groups = 0, keep_groups = 0, group_top = 2;
     float weight_scale = 1.f;
     Tensor w_gate, w_up, w_down;       // [E * F, d], [E * F, d], [E * d, F]; or w_gate [E * 2F, d], gate and up rows alternating in runs of 8
     bool interleaved = false;
@@ -378,6 +437,11 @@ struct RoutedExperts : FeedForward {
     Tensor s_gu, s_down;               // the shared expert
     bool s_interleaved = false;
 
+    static bool gated_kind(const Json& p) {
+        const std::string k = p.get_string("expert", "swiglu");
+        if (k != "swiglu" && k != "relu2") fail(IMP_ERROR_INVALID_MODEL, "routed_experts: unknown expert '" + k + "' (known: swiglu, relu2)");
+        return k == "swiglu";
+    }
     static TensorSpecs specs(const Json& p) {
         const char* me = "routed_experts";
         const int64_t d = need_int(p, "hidden_size", me), E = need_int(p, "num_experts", me), top = need_int(p, "top_k", me),
@@ -391,10 +455,16 @@ struct RoutedExperts : FeedForward {
             fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": " + std::to_string(ng) + " groups must divide the " + std::to_string(E) + " experts, and the " +
                                               std::to_string(keep) + " kept groups must hold the " + std::to_string(top) + " chosen experts");
         const std::string sc = p.get_string("scores", "softmax");
-        if (sc != "softmax" && sc != "sigmoid") fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": unknown scores '" + sc + "' (known: softmax, sigmoid)");
+        if (sc != "softmax" && sc != "sigmoid" && sc != "softmax_all")
+            fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": unknown scores '" + sc + "' (known: softmax, sigmoid, softmax_all)");
+        const std::string gsc = p.get_string("group_score", sc == "softmax_all" ? "max" : "top2");
+        if ((gsc != "max" && gsc != "top2") || (sc == "softmax_all" && gsc != "max"))
+            fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": unknown group_score '" + gsc + "' (known: top2, max; softmax_all goes with max)");
+        const bool gated = gated_kind(p);
+        if (!gated && Fs > 0) fail(IMP_ERROR_UNSUPPORTED, std::string(me) + ": experts without a gate go without a shared expert");
         for (int64_t e = 0; e < E; ++e) {
             const std::string n = std::to_string(e);
-            s.emplace_back("gate_" + n, TensorSpec{{F, d}});
+            if (gated) s.emplace_back("gate_" + n, TensorSpec{{F, d}});
             s.emplace_back("up_" + n, TensorSpec{{F, d}});
             s.emplace_back("down_" + n, TensorSpec{{d, F}});
         }
@@ -413,7 +483,10 @@ struct RoutedExperts : FeedForward {
         F = need_int(a.params, "expert_size", me), Fs = a.params.get_int("shared_size", 0);
         has_bias = a.params.get_bool("router_bias", true);
         has_sgate = a.params.get_bool("shared_gate", true);
-        score_mode = a.params.get_string("scores", "softmax") == "sigmoid" ? 1 : 0;
+        gated_expert = gated_kind(a.params);
+        const std::string sc = a.params.get_string("scores", "softmax");
+        score_mode = sc == "sigmoid" ? 1 : sc == "softmax_all" ? 2 : 0;
+        group_top = a.params.get_string("group_score", score_mode == 2 ? "max" : "top2") == "max" ? 1 : 2;
         weight_scale = (float)a.params.get_double("weight_scale", 1.0);
         n_groups = (int)a.params.get_int("num_groups", 0);
         keep_groups = (int)a.params.get_int("keep_groups", 0);
@@ -421,14 +494,16 @@ struct RoutedExperts : FeedForward {
         std::vector<Tensor> gs, us, ds;
         for (int64_t e = 0; e < E; ++e) {
             const std::string n = std::to_string(e);
-            gs.push_back(a.tensor("gate_" + n));
+            if (gated_expert) gs.push_back(a.tensor("gate_" + n));
             us.push_back(a.tensor("up_" + n));
             ds.push_back(a.tensor("down_" + n));
         }
         // bfloat16 and F a multiple of 8: every expert's gate and up rows alternate in runs of 8, the layout of the fused
         // gate-up product, so that an expert with many rows can go to that product (see forward)
-        interleaved = F % SWIGLU_INTERLEAVE == 0 && gs[0].dtype == BF16 && us[0].dtype == BF16;
-        if (interleaved) {
+        interleaved = gated_expert && F % SWIGLU_INTERLEAVE == 0 && gs[0].dtype == BF16 && us[0].dtype == BF16;
+        if (!gated_expert) {
+            w_up = cat_rows(rt, *a.store, us);
+        } else if (interleaved) {
             std::vector<Tensor> both;
             for (int64_t e = 0; e < E; ++e) both.push_back(interleave_gate_up(rt, *a.store, gs[(size_t)e], us[(size_t)e]));
             w_gate = cat_rows(rt, *a.store, both);
@@ -451,7 +526,7 @@ struct RoutedExperts : FeedForward {
         IMP_CUDA(cudaStreamSynchronize(rt.stream));
         for (int64_t e = 0; e < E; ++e) {
             const std::string n = std::to_string(e);
-            a.drop("gate_" + n);
+            if (gated_expert) a.drop("gate_" + n);
             a.drop("up_" + n);
             a.drop("down_" + n);
         }
@@ -476,7 +551,8 @@ struct RoutedExperts : FeedForward {
         rt.launches += 5;
         const bool gated = Fs > 0 && has_sgate;
         check_launch(imp_moe_route_ex(x.data, x.stride0, (int)T, (int)d, (const float*)router.data, has_bias ? (const float*)router_bias.data : nullptr, (int)E,
-                                      (int)top, gated ? (const float*)sg.data : nullptr, idx, wts, gate, score_mode, n_groups, keep_groups, weight_scale, dt,
+                                      (int)top, gated ? (const float*)sg.data : nullptr, idx, wts, gate, score_mode, n_groups, keep_groups, group_top,
+                                      weight_scale, dt,
                                       rt.stream),
                      "moe_route");
         check_launch(imp_moe_sort(idx, (int)T, (int)top, (int)E, seg, row_token, pair_row, rt.stream), "moe_sort");
@@ -490,7 +566,8 @@ struct RoutedExperts : FeedForward {
         cudaStreamCaptureStatus capturing = cudaStreamCaptureStatusNone;
         IMP_CUDA(cudaStreamIsCapturing(rt.stream, &capturing));
         static const double dense_work = [] { const std::string e = env_string("IMP_B200_MOE_DENSE_WORK", ""); return e.empty() ? 2147483648.0 : std::atof(e.c_str()); }();
-        if (interleaved && !st.decode_only() && capturing == cudaStreamCaptureStatusNone && dense_work > 0 &&
+        const bool tensor_cores = interleaved || (!gated_expert && w_up.dtype == BF16 && w_down.dtype == BF16 && F % 8 == 0 && d % 8 == 0);
+        if (tensor_cores && !st.decode_only() && capturing == cudaStreamCaptureStatusNone && dense_work > 0 &&
             (double)P / (double)E * (double)F * (double)d >= dense_work) {
             std::vector<int> hseg((size_t)E + 1);
             Tensor xs = rt.empty(P, d);
@@ -504,15 +581,22 @@ struct RoutedExperts : FeedForward {
                 Tensor xe = tensor2d((char*)xs.data + (size_t)(a0 * d) * el, rt.dtype, n, d);
                 Tensor ae = tensor2d((char*)act.data + (size_t)(a0 * F) * el, rt.dtype, n, F);
                 Tensor ye = tensor2d((char*)y.data + (size_t)(a0 * d) * el, rt.dtype, n, d);
-                Tensor wgu = tensor2d((char*)w_gate.data + (size_t)(e * 2 * F * d) * el, w_gate.dtype, 2 * F, d);
                 Tensor wd = tensor2d((char*)w_down.data + (size_t)(e * d * F) * el, w_down.dtype, d, F);
-                linear_swiglu(rt, ae, xe, wgu);
+                if (gated_expert)
+                    linear_swiglu(rt, ae, xe, tensor2d((char*)w_gate.data + (size_t)(e * 2 * F * d) * el, w_gate.dtype, 2 * F, d));
+                else
+                    linear_relu2(rt, ae, xe, tensor2d((char*)w_up.data + (size_t)(e * F * d) * el, w_up.dtype, F, d));
                 linear(rt, ye, ae, wd);
             }
         } else {
-            check_launch(imp_grouped_gemm(act.data, F, 0, x.data, x.stride0, 0, row_token, w_gate.data, interleaved ? nullptr : w_up.data,
-                                          (interleaved ? 2 : 1) * F * d, d, seg, (int)P, (int)F, (int)d, (int)E, interleaved ? 2 : 1, dt, rt.stream),
-                         "grouped_gemm (experts, gate and up)");
+            if (!gated_expert)
+                check_launch(imp_grouped_gemm_ex(act.data, F, 0, x.data, x.stride0, 0, row_token, w_up.data, nullptr, F * d, d, seg, (int)P, (int)F, (int)d,
+                                                 (int)E, 0, GROUPED_RELU2, nullptr, 0, dt, rt.stream),
+                             "grouped_gemm (experts, up)");
+            else
+                check_launch(imp_grouped_gemm(act.data, F, 0, x.data, x.stride0, 0, row_token, w_gate.data, interleaved ? nullptr : w_up.data,
+                                              (interleaved ? 2 : 1) * F * d, d, seg, (int)P, (int)F, (int)d, (int)E, interleaved ? 2 : 1, dt, rt.stream),
+                             "grouped_gemm (experts, gate and up)");
             check_launch(imp_grouped_gemm(y.data, d, 0, act.data, F, 0, nullptr, w_down.data, nullptr, d * F, F, seg, (int)P, (int)d, (int)F, (int)E, 0,
                                           dt, rt.stream),
                          "grouped_gemm (experts, down)");
@@ -531,6 +615,12 @@ struct RoutedExperts : FeedForward {
             linear(rt, shared, sa, s_down);
         }
         Tensor out = rt.empty(T, d);
+        if (defer_rows && Fs == 0) {
+            --rt.launches;
+            Branch b = Branch::of(out);
+            b.rows = RoutedRows{y.data, pair_row, wts, (int)top};
+            return b;
+        }
         check_launch(imp_moe_combine(out.data, y.data, pair_row, wts, (int)T, (int)top, Fs > 0 ? shared.data : nullptr, gated ? gate : nullptr, (int)d,
                                      dt, rt.stream),
                      "moe_combine");

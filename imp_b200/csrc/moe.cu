@@ -3,8 +3,9 @@
 //   z[t, e]   = x[t] . Wr[e] + b[e]                       32-bit
 //   chosen    = the `top` experts with the largest z (the lower index wins a tie)
 //   weight    = softmax over the chosen logits only; or, with sigmoid scores s = sigmoid(z): weight = s * weight_scale
+//               or, with softmax scores over all experts: weight = that softmax * weight_scale, not renormalised
 //   groups    = optionally the experts form n_groups equal groups of neighbours; a group's score is the sum of its two
-//               largest scores, and only the experts of the `keep` best groups can be chosen
+//               largest scores, or its largest one, and only the experts of the `keep` best groups can be chosen
 //   gate[t]   = sigmoid(x[t] . Wg)                         one number per token, for a shared expert (optional)
 //   out[t]    = sum_k weight[t, k] * y[place(t, k)] + gate[t] * shared[t]
 //
@@ -46,7 +47,7 @@ __global__ void __launch_bounds__(ROUTE_BLOCK) moe_route_kernel(const TA* __rest
                                                                const float* __restrict__ wr, const float* __restrict__ br, int E, int top,
                                                                const float* __restrict__ wg, int* __restrict__ idx, float* __restrict__ wts,
                                                                float* __restrict__ gate, int vec, int score_mode, int n_groups, int keep,
-                                                               float weight_scale) {
+                                                               int group_top, float weight_scale) {
     pdl_wait();
     pdl_launch_dependents();
     extern __shared__ __align__(16) float sm[];   // x [TPB][d4], then z [TPB][E], then the groups' scores [TPB][n_groups]
@@ -105,8 +106,20 @@ __global__ void __launch_bounds__(ROUTE_BLOCK) moe_route_kernel(const TA* __rest
         float* zt = z + tk * E;
         const int64_t t = t0 + tk;
         float chosen[ROUTE_MAX_TOP];
+        // softmax scores: the choice runs on the logits (same order); the weights need the largest and the sum over all experts
+        float z_max = 0.f, z_sum = 1.f;
+        if (score_mode == 2) {
+            float m = -INFINITY;
+            for (int e = lane; e < E; e += 32) m = fmaxf(m, zt[e]);
+            z_max = warp_max(m);
+            float sum = 0.f;
+            for (int e = lane; e < E; e += 32) sum += expf(zt[e] - z_max);
+            z_sum = warp_sum(sum);
+            __syncwarp();
+        }
         if (n_groups > 0) {
-            // a group's score: the sum of its two largest scores (of its one score where a group is one expert); then `keep`
+            // a group's score: the sum of its two largest scores (of its one score where a group is one expert),
+            // or with group_top 1 its largest one; then `keep`
             // rounds of arg-max over the groups, the lower index winning a tie; the experts of the other groups leave
             float* gt = gsc + tk * n_groups;
             const int per = E / n_groups;
@@ -117,7 +130,7 @@ __global__ void __launch_bounds__(ROUTE_BLOCK) moe_route_kernel(const TA* __rest
                     if (v > a) b = a, a = v;
                     else if (v > b) b = v;
                 }
-                gt[g] = per > 1 ? a + b : a;
+                gt[g] = per > 1 && group_top == 2 ? a + b : a;
             }
             __syncwarp();
             for (int k = 0; k < keep; ++k) {
@@ -162,6 +175,8 @@ __global__ void __launch_bounds__(ROUTE_BLOCK) moe_route_kernel(const TA* __rest
         }
         if (lane == 0 && score_mode == 1) {
             for (int k = 0; k < top; ++k) wts[t * top + k] = chosen[k] * weight_scale;   // the scores themselves, not renormalised
+        } else if (lane == 0 && score_mode == 2) {
+            for (int k = 0; k < top; ++k) wts[t * top + k] = expf(chosen[k] - z_max) / z_sum * weight_scale;
         } else if (lane == 0) {
             const float largest = chosen[0];   // the first chosen is the largest
             float sum = 0.f;
@@ -287,19 +302,19 @@ IMP_API int imp_gather_rows(void* dst, const void* src, int64_t ld, const int* i
 
 template <typename TA, int TPB>
 static cudaError_t launch_route(const void* x, int64_t ldx, int n_tokens, int d, const float* wr, const float* br, int E, int top, const float* wg,
-                                int* idx, float* wts, float* gate, int vec, int score_mode, int n_groups, int keep, float weight_scale, size_t smem,
+                                int* idx, float* wts, float* gate, int vec, int score_mode, int n_groups, int keep, int group_top, float weight_scale, size_t smem,
                                 cudaStream_t s) {
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(moe_route_kernel<TA, TPB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
     }
     return imp_launch(moe_route_kernel<TA, TPB>, dim3((n_tokens + TPB - 1) / TPB), dim3(ROUTE_BLOCK), smem, s, (const TA*)x, ldx, n_tokens, d, wr, br,
-                      E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, weight_scale);
+                      E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale);
 }
 
 template <typename TA>
 static cudaError_t route_by_size(const void* x, int64_t ldx, int n_tokens, int d, const float* wr, const float* br, int E, int top, const float* wg,
-                                 int* idx, float* wts, float* gate, int vec, int score_mode, int n_groups, int keep, float weight_scale,
+                                 int* idx, float* wts, float* gate, int vec, int score_mode, int n_groups, int keep, int group_top, float weight_scale,
                                  cudaStream_t s) {
     // more tokens a CTA where there are many (a row of the router is read once per CTA), one where there are few (more CTAs)
     int tpb = n_tokens >= 1024 ? 8 : n_tokens >= 256 ? 4 : n_tokens >= 64 ? 2 : 1;
@@ -308,31 +323,33 @@ static cudaError_t route_by_size(const void* x, int64_t ldx, int n_tokens, int d
     while (tpb > 1 && bytes(tpb) > 160 * 1024) tpb /= 2;
     if (bytes(tpb) > 200 * 1024) return cudaErrorInvalidValue;
     switch (tpb) {
-        case 8: return launch_route<TA, 8>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, weight_scale, bytes(8), s);
-        case 4: return launch_route<TA, 4>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, weight_scale, bytes(4), s);
-        case 2: return launch_route<TA, 2>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, weight_scale, bytes(2), s);
-        default: return launch_route<TA, 1>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, weight_scale, bytes(1), s);
+        case 8: return launch_route<TA, 8>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, bytes(8), s);
+        case 4: return launch_route<TA, 4>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, bytes(4), s);
+        case 2: return launch_route<TA, 2>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, bytes(2), s);
+        default: return launch_route<TA, 1>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, bytes(1), s);
     }
 }
 
 // x [T, d] (activation type, rows ldx apart); wr float32 [E, d], br float32 [E] or null; wg float32 [d] or null (then
 // gate is not written).  idx int32 [T, top], wts float32 [T, top], gate float32 [T].
 // score_mode 0: weights are the softmax over the chosen logits; 1: scores are sigmoid(z) and a weight is its score times
-// weight_scale.  n_groups > 0: only experts of the `keep` best of n_groups equal groups of neighbours can be chosen.
+// weight_scale; 2: scores are the softmax over all experts, a weight as in 1.
+// group_top: how many of its largest scores a group counts by (1 or 2).  n_groups > 0: only experts of the `keep` best of n_groups equal groups of neighbours can be chosen.
 IMP_API int imp_moe_route_ex(const void* x, int64_t ldx, int n_tokens, int d, const float* wr, const float* br, int E, int top, const float* wg,
-                             int* idx, float* wts, float* gate, int score_mode, int n_groups, int keep, float weight_scale, int act_dtype,
+                             int* idx, float* wts, float* gate, int score_mode, int n_groups, int keep, int group_top, float weight_scale, int act_dtype,
                              void* stream) {
     if (n_tokens == 0) return 0;
     IMP_CHECK_ARG(x && wr && idx && wts && d > 0 && (!wg || gate), "imp_moe_route: bad argument");
     IMP_CHECK_ARG(E > 0 && E <= ROUTE_MAX_E && top > 0 && top <= E && top <= ROUTE_MAX_TOP,
                   "imp_moe_route: %d experts (at most %d), %d chosen (at most %d and no more than there are)", E, ROUTE_MAX_E, top, ROUTE_MAX_TOP);
-    IMP_CHECK_ARG((score_mode == 0 || score_mode == 1) && n_groups >= 0 && (n_groups == 0 || (E % n_groups == 0 && keep > 0 && keep <= n_groups &&
+    IMP_CHECK_ARG(score_mode >= 0 && score_mode <= 2 && (group_top == 1 || group_top == 2) && n_groups >= 0 && (n_groups == 0 || (E % n_groups == 0 && keep > 0 && keep <= n_groups &&
                                                                                              top <= keep * (E / n_groups))),
                   "imp_moe_route: %d groups over %d experts, %d kept, %d chosen", n_groups, E, keep, top);
+    IMP_CHECK_ARG(score_mode != 2 || n_groups == 0 || group_top == 1, "imp_moe_route: with softmax scores over all experts groups count by their largest score");
     const int vec = (d % 4 == 0 && (uintptr_t)wr % 16 == 0 && (!wg || (uintptr_t)wg % 16 == 0)) ? 1 : 0;
     cudaStream_t s = (cudaStream_t)stream;
-    cudaError_t e = act_dtype == IMP_F32 ? route_by_size<float>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, weight_scale, s)
-                                         : route_by_size<__nv_bfloat16>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, weight_scale, s);
+    cudaError_t e = act_dtype == IMP_F32 ? route_by_size<float>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, s)
+                                         : route_by_size<__nv_bfloat16>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, s);
     if (e != cudaSuccess) {
         imp_set_error("imp_moe_route: %s (rows of %d values, %d experts)", cudaGetErrorString(e), d, E);
         return (int)e;
@@ -342,7 +359,7 @@ IMP_API int imp_moe_route_ex(const void* x, int64_t ldx, int n_tokens, int d, co
 
 IMP_API int imp_moe_route(const void* x, int64_t ldx, int n_tokens, int d, const float* wr, const float* br, int E, int top, const float* wg,
                           int* idx, float* wts, float* gate, int act_dtype, void* stream) {
-    return imp_moe_route_ex(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, 0, 0, 0, 1.f, act_dtype, stream);
+    return imp_moe_route_ex(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, 0, 0, 0, 2, 1.f, act_dtype, stream);
 }
 
 IMP_API int imp_moe_sort(const int* idx, int n_tokens, int top, int E, int* seg, int* row_token, int* pair_row, void* stream) {

@@ -165,10 +165,9 @@ __global__ void __launch_bounds__(256) rms_pair_mean_kernel(TA* __restrict__ out
     for (int i = threadIdx.x; i < d; i += blockDim.x) o[i] = from_float<TA>(fmaf(to_float(ar[i]) * ra, wa[i], to_float(br[i]) * rb * wb[i]));
 }
 
-// out[t, f] = act(gate) * up over rows [gate | up] (block == 0) or runs of `block` gate entries followed by their up entries.
-// act: 0 silu, 1 gelu (tanh form).
+// out[t, f] = the gated activation (GateAct, kinds 0 to 2) over rows [gate | up] (block == 0) or runs of `block` gate entries followed by their up entries.
 template <typename T>
-__global__ void gated_act_kernel(T* __restrict__ out, const T* __restrict__ gu, int64_t n_tokens, int F, int block, int act) {
+__global__ void gated_act_kernel(T* __restrict__ out, const T* __restrict__ gu, int64_t n_tokens, int F, int block, GateAct act) {
     pdl_wait();
     pdl_launch_dependents();
     const int64_t total = n_tokens * (int64_t)F;
@@ -179,12 +178,11 @@ __global__ void gated_act_kernel(T* __restrict__ out, const T* __restrict__ gu, 
         const int ui = block ? gi + block : F + f;
         const float g = to_float(gu[t * 2 * F + gi]);
         const float u = to_float(gu[t * 2 * F + ui]);
-        const float a = gate_act_f(g, act);
-        out[i] = from_float<T>(a * u);
+        out[i] = from_float<T>(gated_f(g, u, act));
     }
 }
 
-// out[t, j] = act(x[t, j]) for j < n: a dense copy of a slice of wider rows.  act: 0 identity, 1 tanh.
+// out[t, j] = act(x[t, j]) for j < n: a dense copy of a slice of wider rows.  act: 0 identity, 1 tanh, 2 max(v, 0)^2.
 template <typename T>
 __global__ void act_rows_kernel(T* __restrict__ out, const T* __restrict__ x, int64_t ld, int64_t n_tokens, int n, int act) {
     pdl_wait();
@@ -193,7 +191,7 @@ __global__ void act_rows_kernel(T* __restrict__ out, const T* __restrict__ x, in
     for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
         const int64_t t = i / n;
         const float v = to_float(x[t * ld + (i - t * n)]);
-        out[i] = from_float<T>(act == 1 ? tanhf(v) : v);
+        out[i] = from_float<T>(act == 1 ? tanhf(v) : act == 2 ? relu2_f(v) : v);
     }
 }
 
@@ -378,21 +376,21 @@ IMP_API int imp_rms_pair_mean(void* out, const void* a, const float* wa, float c
     IMP_RETURN_LAUNCH();
 }
 
-IMP_API int imp_gated_act(void* out, const void* gate_up, int n_tokens, int F, int block, int act, int dtype, void* stream) {
+IMP_API int imp_gated_act(void* out, const void* gate_up, int n_tokens, int F, int block, int act, float limit, int dtype, void* stream) {
     if (n_tokens == 0 || F == 0) return 0;
-    IMP_CHECK_ARG(out && gate_up && n_tokens > 0 && F > 0 && block >= 0 && (block == 0 || F % block == 0) && (act == 0 || act == 1),
+    IMP_CHECK_ARG(out && gate_up && n_tokens > 0 && F > 0 && block >= 0 && (block == 0 || F % block == 0) && act >= ACT_SILU && act <= ACT_CLIPPED,
                   "imp_gated_act: bad argument");
     cudaStream_t s = (cudaStream_t)stream;
     const int64_t total = (int64_t)n_tokens * F;
     const dim3 grid((unsigned)std::min<int64_t>((total + 255) / 256, 65535));
-    if (dtype == IMP_F32) imp_launch(gated_act_kernel<float>, grid, dim3(256), 0, s, (float*)out, (const float*)gate_up, (int64_t)n_tokens, F, block, act);
-    else imp_launch(gated_act_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, (int64_t)n_tokens, F, block, act);
+    if (dtype == IMP_F32) imp_launch(gated_act_kernel<float>, grid, dim3(256), 0, s, (float*)out, (const float*)gate_up, (int64_t)n_tokens, F, block, GateAct(act, limit));
+    else imp_launch(gated_act_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, (int64_t)n_tokens, F, block, GateAct(act, limit));
     IMP_RETURN_LAUNCH();
 }
 
 IMP_API int imp_act_rows(void* out, const void* x, int64_t ld, int n_tokens, int n, int act, int dtype, void* stream) {
     if (n_tokens == 0 || n == 0) return 0;
-    IMP_CHECK_ARG(out && x && n > 0 && ld >= n && (act == 0 || act == 1), "imp_act_rows: bad argument");
+    IMP_CHECK_ARG(out && x && n > 0 && ld >= n && act >= 0 && act <= 2, "imp_act_rows: bad argument");
     cudaStream_t s = (cudaStream_t)stream;
     const int64_t total = (int64_t)n_tokens * n;
     const dim3 grid((unsigned)std::min<int64_t>((total + 255) / 256, 65535));
