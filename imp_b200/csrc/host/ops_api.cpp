@@ -74,14 +74,25 @@ IMP_EXPORT int imp_op_linear_swiglu(const ImpTensor* out, const ImpTensor* x, co
     });
 }
 
-// The same with the gate's activation chosen: 0 silu, 1 the tanh form of gelu.
-IMP_EXPORT int imp_op_linear_gated(const ImpTensor* out, const ImpTensor* x, const ImpTensor* w_interleaved, int act, void* stream,
-                                   int32_t* status) {
+// The same with the activation chosen: 0 silu, 1 the tanh form of gelu, 2 both values clipped to `limit` (see GatedAct).
+IMP_EXPORT int imp_op_linear_gated(const ImpTensor* out, const ImpTensor* x, const ImpTensor* w_interleaved, int act, float limit,
+                                   void* stream, int32_t* status) {
     return guarded([&] {
         if (!out || !x || !w_interleaved) fail(IMP_ERROR_INVALID_ARG, "imp_op_linear_gated: null tensor");
         Runtime rt = runtime_for(stream, status);
         rt.dtype = x->dtype;
-        linear_gated(rt, *out, *x, *w_interleaved, act);
+        linear_gated(rt, *out, *x, *w_interleaved, GatedAct(act, limit));
+        g_fallbacks += rt.fallback_calls;
+    });
+}
+
+// out = max(x w^T, 0)^2.
+IMP_EXPORT int imp_op_linear_relu2(const ImpTensor* out, const ImpTensor* x, const ImpTensor* w, void* stream, int32_t* status) {
+    return guarded([&] {
+        if (!out || !x || !w) fail(IMP_ERROR_INVALID_ARG, "imp_op_linear_relu2: null tensor");
+        Runtime rt = runtime_for(stream, status);
+        rt.dtype = x->dtype;
+        linear_relu2(rt, *out, *x, *w);
         g_fallbacks += rt.fallback_calls;
     });
 }

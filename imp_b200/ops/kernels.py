@@ -114,15 +114,28 @@ def linear_swiglu(out: torch.Tensor, x: torch.Tensor, w_interleaved: torch.Tenso
     return out
 
 
-def linear_gated(out: torch.Tensor, x: torch.Tensor, w_interleaved: torch.Tensor, activation: str = "silu") -> torch.Tensor:
-    """out[M, F] = act(x Wg^T) * (x Wu^T), act "silu" or "gelu_tanh", with the activation in the product's epilogue
+def linear_gated(out: torch.Tensor, x: torch.Tensor, w_interleaved: torch.Tensor, activation: str = "silu",
+                 limit: float = 0.0) -> torch.Tensor:
+    """out[M, F] = act(x Wg^T) * (x Wu^T), act "silu" or "gelu_tanh", or "clipped": g sigmoid(1.702 g) (u + 1) with
+    g = min(x Wg^T, limit) and u = x Wu^T held within +-limit; with the activation in the product's epilogue
     where the library has such a kernel for the shape (csrc/host/linear.cpp `linear_gated`)."""
     _need_cuda(out, x, w_interleaved)
     if x.shape[0] == 0:
         return out
-    act = {"silu": 0, "gelu_tanh": 1}[activation]
+    act = {"silu": 0, "gelu_tanh": 1, "clipped": 2}[activation]
     o, a, w = _view(out), _view(x), _view(w_interleaved)
-    _op_check(L.load().imp_op_linear_gated(ctypes.byref(o), ctypes.byref(a), ctypes.byref(w), act, _stream(), None), "linear_gated")
+    _op_check(L.load().imp_op_linear_gated(ctypes.byref(o), ctypes.byref(a), ctypes.byref(w), act, float(limit), _stream(), None), "linear_gated")
+    return out
+
+
+def linear_relu2(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """out = max(x W^T, 0)^2, with the activation in the product's epilogue where the library has such a kernel for the
+    shape (csrc/host/linear.cpp `linear_relu2`)."""
+    _need_cuda(out, x, w)
+    if x.shape[0] == 0:
+        return out
+    o, a, ww = _view(out), _view(x), _view(w)
+    _op_check(L.load().imp_op_linear_relu2(ctypes.byref(o), ctypes.byref(a), ctypes.byref(ww), _stream(), None), "linear_relu2")
     return out
 
 

@@ -295,8 +295,11 @@ class PartHandle:
             c.cache = ctypes.cast(cache._ptr, ctypes.POINTER(capi.ImpCacheView))
         return as_torch(self._call(c, ctx).out, self.device)
 
-    def embed(self, ctx: Optional[StepContext] = None):
-        return as_torch(self._call(capi.ImpCall(), ctx).h, self.device)
+    def embed(self, ctx: Optional[StepContext] = None, cache: Optional[LayerCache] = None):
+        c = capi.ImpCall()
+        if cache is not None:
+            c.cache = ctypes.cast(cache._ptr, ctypes.POINTER(capi.ImpCacheView))
+        return as_torch(self._call(c, ctx).h, self.device)
 
     def block_forward(self, h, pending, ctx: Optional[StepContext] = None, cache: Optional[LayerCache] = None):
         c = capi.ImpCall()
