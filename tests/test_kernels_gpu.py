@@ -208,21 +208,37 @@ def test_linear_swiglu_fused(K, M, F, K_):
 
 @pytest.mark.parametrize("M", [1, 5, 11, 16, 40, 100, 130, 300, 1100])
 @pytest.mark.parametrize("F,K_", [(8, 64), (200, 96), (1536, 512), (24, 100)])
-@pytest.mark.parametrize("activation", ["silu", "gelu_tanh"])
+@pytest.mark.parametrize("activation", ["silu", "gelu_tanh", "clipped"])
 def test_linear_gated_fused(K, M, F, K_, activation):
-    """The gated product with either activation, over the row counts that choose each of its kernels."""
+    """The gated product with each activation, over the row counts that choose each of its kernels."""
     x = rnd(M, K_, dtype=torch.bfloat16, seed=33).to(DEV)
     wg = rnd(F, K_, dtype=torch.bfloat16, seed=34, scale=0.3).to(DEV)
     wu = rnd(F, K_, dtype=torch.bfloat16, seed=35, scale=0.3).to(DEV)
     w = K.interleave_gate_up(wg, wu)
-    out = K.linear_gated(torch.full((M, F), float("nan"), dtype=torch.bfloat16, device=DEV), x, w, activation)
+    out = K.linear_gated(torch.full((M, F), float("nan"), dtype=torch.bfloat16, device=DEV), x, w, activation, limit=1.3)
     g = x.double().cpu() @ wg.double().cpu().T
     u = x.double().cpu() @ wu.double().cpu().T
     if activation == "silu":
         a = g / (1 + torch.exp(-g))
+    elif activation == "clipped":
+        assert (g > 1.3).any() and (u.abs() > 1.3).any()
+        g, u = torch.clamp(g, max=1.3), torch.clamp(u, -1.3, 1.3) + 1
+        a = g * torch.sigmoid(1.702 * g)
     else:
         a = 0.5 * g * (1 + torch.tanh(math.sqrt(2 / math.pi) * (g + 0.044715 * g ** 3)))
     close(out, a * u, torch.bfloat16)
+
+
+@pytest.mark.parametrize("M", [1, 5, 16, 40, 100, 130, 300, 1100])
+@pytest.mark.parametrize("N,K_", [(8, 64), (264, 96), (1536, 4096), (24, 100)])
+@pytest.mark.parametrize("dtype", [torch.bfloat16, torch.float32])
+def test_linear_relu2(K, M, N, K_, dtype):
+    """The product with a squared relu behind it, over the row counts that choose each of its kernels."""
+    x = rnd(M, K_, dtype=dtype, seed=36).to(DEV)
+    w = rnd(N, K_, dtype=dtype, seed=37, scale=1.0 / math.sqrt(K_)).to(DEV)
+    out = K.linear_relu2(torch.full((M, N), float("nan"), dtype=dtype, device=DEV), x, w)
+    want = torch.relu(x.double().cpu() @ w.double().cpu().T) ** 2
+    close(out, want, dtype, scale=float(want.abs().max()))
 
 
 @pytest.mark.parametrize("M,N,K_", [(128, 256, 64), (1, 8, 8), (130, 264, 72), (300, 520, 200), (257, 1000, 4104),
