@@ -92,14 +92,14 @@ def to_imp(x) -> "capi.ImpTensor":
     code = {torch.float32: capi.ELEM_F32, torch.bfloat16: capi.ELEM_BF16, torch.int32: capi.ELEM_I32}.get(x.dtype)
     if code is None:
         raise TypeError(f"element type {x.dtype} cannot cross into the library (float32, bfloat16, int32)")
-    if not x.is_cuda or x.dim() > 4 or x.dim() == 0:
-        raise TypeError("the library takes CUDA tensors of one to four dimensions")
+    if not x.is_cuda or x.dim() > 4:
+        raise TypeError("the library takes CUDA tensors of up to four dimensions")
     if x.dim() > 1 and not x[0].is_contiguous():
         x = x.contiguous()
     t.data, t.dtype, t.ndim = x.data_ptr(), code, x.dim()
     for i, s in enumerate(x.shape):
         t.shape[i] = s
-    t.stride0 = x.stride(0) if x.shape[0] > 1 or x.dim() == 1 else max(1, x[0].numel() if x.dim() > 1 else 1)
+    t.stride0 = 1 if x.dim() == 0 else x.stride(0) if x.shape[0] > 1 or x.dim() == 1 else max(1, x[0].numel() if x.dim() > 1 else 1)
     t._keep = x
     return t
 

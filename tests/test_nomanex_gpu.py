@@ -287,7 +287,7 @@ def test_gla_finds_one_loud_key_far_back(dtype, decoded):
     want = plain(x)
     quiet = x.clone()
     quiet[at, 0] = 0.0
-    assert (plain(quiet)[-1] - want[-1]).abs().max() > 0.2 * want.abs().max(), "the last token hangs on the loud one"
+    assert (plain(quiet)[-1] - want[-1]).abs().max() > 0.5 * want[-1].abs().max(), "the last token hangs on the loud one"
     out = in_pieces(bench, part, x, (T - 40,) + (1,) * 40 if decoded else (300, 2, T - 302))
     close(out[at:], want[at:], dtype, "after the loud key", loose=2.0)
 
@@ -532,9 +532,9 @@ def with_shared(layers, order):
 
 
 # M1: both mixers, shared weights of both kinds (an attention layer with two caches), windows of 24 (one and a half pages) and 9,
-# grouped experts.  M2: nothing shared, no token pairs, m = 1, no window, no groups, an attention layer without feed-forward first,
-# pages of 4.  M3: attention only (no recurrent layer), a layer used four times, one bucket.  M4: gated linear attention only,
-# sizes that are multiples of nothing.
+# grouped experts.  M2: nothing shared, m = 1, no window, no groups, an attention layer without feed-forward first,
+# pages of 4.  M3: attention only (no recurrent layer), a layer used four times, one bucket.  M4: gated linear attention only, no
+# token pairs, sizes that are multiples of nothing.
 L1 = [{"type": "gla", "mixer": gla(3, 16, 24, 5.0, 6), "mlp": dense(72, 1.5)},
       {"type": "latent_attention", "mixer": lat(5, 16, 8, 20, 40, 24, base=100.0), "mlp": moe_cfg(12, 3, 24, (4, 2))},
       {"type": "gla", "mixer": gla(2, 40, 16, 16.0, 9), "mlp": None},
@@ -543,6 +543,7 @@ MODELS = {
     "M1": ({"architecture": "Nomanex", "vocab": 97, "width": 64, "norm": {"eps": 3e-5}, "residual_mult": 0.5,
             "embedding": {"bigram": {"buckets": 211, "mul_prev": 37, "mul_cur": 11}}, "layers": with_shared(L1, [0, 1, 0, 2, 3, 1, 0])}, 16),
     "M2": ({"architecture": "Nomanex", "vocab": 151, "width": 112, "norm": {"eps": 1e-6}, "residual_mult": 1.0,
+            "embedding": {"bigram": {"buckets": 75, "mul_prev": 13, "mul_cur": 29}},
             "layers": [{"type": "latent_attention", "mixer": lat(3, 32, 16, 40, 112, 0), "mlp": None},
                        {"type": "gla", "mixer": gla(4, 24, 24, 8.0, 16), "mlp": moe_cfg(6, 1, 32)},
                        {"type": "latent_attention", "mixer": lat(4, 20, 12, 28, 50, 100, base=300.0), "mlp": moe_cfg(16, 4, 24, (16, 5))}]}, 4),
@@ -551,7 +552,6 @@ MODELS = {
             "layers": with_shared([{"type": "latent_attention", "mixer": lat(6, 16, 16, 16, 48, 40), "mlp": moe_cfg(8, 2, 32, (2, 1))},
                                    {"type": "latent_attention", "mixer": lat(2, 48, 8, 32, 248, 64, base=50.0), "mlp": dense(128, 2.5)}], [0, 1, 0, 0, 0])}, 16),
     "M4": ({"architecture": "Nomanex", "vocab": 83, "width": 70, "norm": {"eps": 1e-5}, "residual_mult": 0.6,
-            "embedding": {"bigram": {"buckets": 75, "mul_prev": 13, "mul_cur": 29}},
             "layers": [{"type": "gla", "mixer": gla(2, 9, 11, 3.0, 5), "mlp": dense(50, 1.2)},
                        {"type": "gla", "mixer": gla(1, 70, 37, 12.0, 3), "mlp": moe_cfg(3, 2, 12)}]}, 8),
 }
@@ -714,6 +714,73 @@ def test_greedy_generation_through_the_engine(nomanex_folders):
         top2 = torch.topk(lg, 2).values
         if float(top2[0] - top2[1]) > 0.1 * float(lg.abs().max()):
             assert g16[0] == w[0]
+
+
+def test_blocks_sum_worked_out_for_a_norm_that_takes_plain_branches(nomanex_folders):
+    """The block alone hands on one tensor: m times the sum of its two sublayers."""
+    dtype, d, m = torch.float32, 64, 0.7
+    bench = PartBench(NAME[dtype], [], max_tokens=64)
+    w, b, alpha = 1 + 0.3 * rnd(d, seed=1), 0.4 * rnd(d, seed=2), torch.tensor(0.7)
+    f, c = dense_weights(d, 40, 3), {"router": {"experts": 5, "top": 2}, "expert": {"ff": 16}}
+    e = moe_weights(d, c, 9)
+    spec = mixer_cache_spec("gated_linear_attention", {"hidden_size": d, "num_heads": 2, "key_dim": 8, "value_dim": 8, "tau": 4.0})
+    x = rnd(20, d, seed=5)
+    h = N.dynamic_tanh(x.double(), 0.7 * torch.ones((), dtype=torch.float64), w.double(), b.double())
+    g = gla_weights(d, gla(2, 8, 8, 4.0, 3), 30)
+    G = {"m." + k: v.double() for k, v in g.items()}
+    mix = N.gla(h, G, "m.", gla(2, 8, 8, 4.0, 3), EPS)
+    for kind in ("dense", "moe", None):
+        bench = PartBench(NAME[dtype], [spec], max_tokens=64)
+        norm = bench.build("norm", PartSpec("dynamic_tanh", {"size": d}), {"weight": w.to(DEV), "bias": b.to(DEV), "alpha": alpha.to(DEV)})
+        mixer = bench.build("mixer", PartSpec("gated_linear_attention", {"hidden_size": d, "num_heads": 2, "key_dim": 8, "value_dim": 8, "tau": 4.0, "norm_eps": EPS}),
+                            {GLA_NAMES[k]: v.to(DEV) for k, v in g.items()})
+        parts = {"norm": norm, "mixer": mixer}
+        want = mix
+        if kind == "dense":
+            parts["feed_forward"] = bench.build("feed_forward", PartSpec("gated_mlp", {"hidden_size": d, "intermediate_size": 40, "activation": "clipped", "limit": 1.0}),
+                                                {"gate_proj": f["gate"].to(DEV), "up_proj": f["up"].to(DEV), "down_proj": f["down"].to(DEV)})
+            want = mix + N.dense_ff(h, {"f." + k: v.double() for k, v in f.items()}, "f.", {"limit": 1.0})
+        elif kind == "moe":
+            parts["feed_forward"] = bench.build("feed_forward", PartSpec("routed_experts", moe_params(d, c)), {moe_names(c)[k]: v.to(DEV) for k, v in e.items()})
+            want = mix + N.moe(h, {"f." + k: v.double() for k, v in e.items()}, "f.", c)
+        block = bench.build_block("parallel", parts, {"residual_mult": m, "has_ffn": kind is not None})
+        ctx = bench.prepare([("a", [1] * 20, [])])
+        torch.cuda.synchronize()
+        out = block.block_forward(x.to(DEV), None, ctx, bench.cache_view(0))
+        bench.sync()
+        close(out, m * want, dtype, f"feed-forward {kind}")
+
+
+def test_unsummed_products_of_both_sublayers_reach_the_norm(tmp_path):
+    """Wide enough that a decode step's output products are cut over the contraction: their parts, both sublayers' at once,
+    are added by the next norm."""
+    from imp_b200 import Engine, EngineConfig, StepEntry
+    cfg = {"architecture": "Nomanex", "vocab": 64, "width": 512, "norm": {"eps": 1e-5}, "residual_mult": 0.3,
+           "embedding": {"bigram": {"buckets": 19, "mul_prev": 3, "mul_cur": 5}},
+           "layers": [{"type": "gla", "mixer": gla(8, 64, 128, 8.0, 16), "mlp": dense(2048, 2.0)},
+                      {"type": "latent_attention", "mixer": lat(16, 64, 16, 64, 112, 20), "mlp": moe_cfg(4, 2, 256)},
+                      {"type": "gla", "mixer": gla(8, 64, 128, 8.0, 16), "mlp": None}]}
+    W = make_weights(cfg, 5)
+    (tmp_path / "config.json").write_text(json.dumps(file_config(cfg)))
+    save_safetensors(str(tmp_path / "model.safetensors"), W)
+    Wd = {k: v.double() for k, v in W.items()}
+    g = torch.Generator().manual_seed(1)
+    seqs = {r: torch.randint(0, 64, (30,), generator=g).tolist() for r in "abc"}
+    margins = {r: [] for r in seqs}
+    want = {r: N.forward(ids, Wd, cfg, margins=margins[r]) for r, ids in seqs.items()}
+    sure = {r: torch.stack(m).min(dim=0).values > 0.03 for r, m in margins.items()}
+    eng = Engine.from_folder(str(tmp_path), EngineConfig(compute_dtype="bfloat16", kv_block_size=16, kv_cache_tokens=256, max_batch_size=4, max_seq_len=64,
+                                                         max_batch_tokens=128))
+    eng.step_tokens([StepEntry(r, ids[:20], []) for r, ids in seqs.items()])
+    rel = []
+    for t in range(20, 30):
+        got = eng.step_tokens([StepEntry(r, [ids[t]], [0]) for r, ids in seqs.items()])
+        for i, r in enumerate(seqs):
+            if sure[r][t]:
+                err = torch.from_numpy(np.asarray(got[i])).double() - want[r][t]
+                rel.append(float(err.pow(2).mean().sqrt() / want[r].pow(2).mean().sqrt()))
+    assert len(rel) > 15 and max(rel) < 0.05, rel
+    assert eng.info()["split_norm_calls"] > 0
 
 
 def test_preemption_recomputes_state_and_predecessor(nomanex_folders):
