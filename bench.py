@@ -30,6 +30,7 @@ Other runs, each printing its own JSON line:
     python bench.py --arch kuzipel [--layers N] [--batch B]    Kuzipel beside Kazedra and Qwen3 at equal sizes
     python bench.py --arch pemidra [--layers N] [--batch B]    Pemidra beside Kazedra and Qwen3 at equal sizes
     python bench.py --arch nizorax [--layers N] [--batch B]    Nizorax beside Pemidra, Kuzipel and Qwen3 at equal sizes
+    python bench.py --arch nomanex [--layers N] [--batch B]    Nomanex beside Kuzipel, Pemidra and Qwen3 at equal sizes
     python bench.py --workload 14b                        8 prompts of 8,192 tokens in 2,048-token portions, 512 tokens at T=0.7
 (`--context` may exceed the configured 4096: the cache and the position table grow with it.)
 """
@@ -772,8 +773,25 @@ def nizorax_config(width, heads, kv_heads, ff, layers, vocab):
             "canon": {"taps": 4}, "layers": lays, "max_positions": 8192}
 
 
+def nomanex_config(width, heads, kv_heads, ff, layers, vocab):
+    """Layers cycle through gated linear attention (heads of 128 keys and 128 values: Pemidra's retention geometry) with the
+    dense feed-forward of the models beside it, latent attention (Kuzipel's geometry, without its query latent, a window of 1,024
+    positions) with routed experts (16 in 4 groups of which 2 are kept, two chosen, together the dense inner size), and the
+    same two mixers with the feed-forwards exchanged; token pairs hashed into 65,536 rows."""
+    wide = width >= 2048
+    latent = {"heads": heads, "dim": 128 if wide else 64, "rot_dim": 64 if wide else 32, "vdim": 128 if wide else 64, "kv_rank": 192 if wide else 96,
+              "scale": (192 if wide else 96) ** -0.5, "mask": {"size": 1024}, "rot": {"base": 10000.0, "dims": 64 if wide else 32}}
+    gla = {"heads": width // 128, "dim": 128, "vdim": 128, "tau": 16.0, "decay_rank": 16}
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": ff // 2}, "router": {"experts": 16, "top": 2, "groups": {"count": 4, "keep": 2}}}
+    kinds = [("gla", gla, dense), ("latent_attention", latent, moe), ("gla", gla, moe), ("latent_attention", latent, dense)]
+    lays = [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": kinds[i % 4][2]} for i in range(layers)]
+    return {"architecture": "Nomanex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.3,
+            "embedding": {"bigram": {"buckets": 65536, "mul_prev": 40503, "mul_cur": 30011}}, "layers": lays, "max_positions": 8192}
+
+
 def run_arch(args):
-    """Prefill and decode of Kazedra, Kuzipel, Pemidra or Nizorax beside the models the engine already had at equal sizes (random weights): a
+    """Prefill and decode of Kazedra, Kuzipel, Pemidra, Nizorax or Nomanex beside the models the engine already had at equal sizes (random weights): a
     2,048-token prompt whole and in 512-token portions, and decode steps of `--batch` sequences at context 2,048, device
     time between CUDA events."""
     if args.arch == "kuzipel":
@@ -782,6 +800,8 @@ def run_arch(args):
         return run_arch_beside(args, "pemidra", pemidra_config)
     if args.arch == "nizorax":
         return run_arch_beside(args, "nizorax", nizorax_config, beside={"pemidra": pemidra_config, "kuzipel": kuzipel_config})
+    if args.arch == "nomanex":
+        return run_arch_beside(args, "nomanex", nomanex_config, beside={"kuzipel": kuzipel_config, "pemidra": pemidra_config})
     peaks, peak_src = read_peaks()
     layers, vocab, B = args.layers or 4, 32768, args.batch
     if args.only in ("prefill", "decode"):
@@ -927,7 +947,7 @@ def main():
     ap.add_argument("--only", default="", choices=["", "decode", "prefill", "timeline", "mixed"],
                     help="run one phase only and print its timing (for profiling small cases)")
     ap.add_argument("--workload", default="", choices=["", "0.6b", "14b"], help="one of the two other workloads of the baseline record")
-    ap.add_argument("--arch", default="", choices=["", "kazedra", "kuzipel", "pemidra", "nizorax"],
+    ap.add_argument("--arch", default="", choices=["", "kazedra", "kuzipel", "pemidra", "nizorax", "nomanex"],
                     help="prefill and decode of this architecture beside the Qwen3 decoder at equal sizes (not the default workload)")
     ap.add_argument("--shape", default="8b", choices=["1b", "8b"], help="with --arch and --only: which of the shapes")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="with --workload: the compute type")

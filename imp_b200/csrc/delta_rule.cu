@@ -524,8 +524,7 @@ IMP_API int imp_gdr_output(void* y, const float* o, const void* gate, int64_t ga
 // The general form of these recurrences: a matrix state S [D, Dv] per head that decays per key channel,
 // loses one direction and gains one outer product per token,
 //     S <- diag(w) S - p (z^T S) + kw v^T,      o = S^T q      (the read-out sees the token's own write)
-// with w, p, z, kw, q vectors over the key dimension.  Four mixers are instances of it:
-//     gated linear attention w per head and key channel, p = z = 0, kw = k
+// with w, p, z, kw, q vectors over the key dimension.  Three mixers are instances of it:
 //     retention              w = a constant per head, p = z = 0, kw = k
 //     delta rule, decay per  w = g (per head and key channel), z = g k, p = kw = beta k
 //       key channel            (S <- g S; u = beta (v - S^T k); S <- S + k u^T)
@@ -536,11 +535,11 @@ IMP_API int imp_gdr_output(void* y, const float* o, const void* gate, int64_t ga
 // (made once per token and head by the prepare kernels):
 //     s <- w s - p a + kw v;      o = c - qp a + qk v
 // so the two sums over the key dimension start from the old state together: one round of shuffles per token.
-enum { LSR_RETENTION = 0, LSR_DELTA = 1, LSR_GENERAL = 2, LSR_CHANNEL = 3 };   // LSR_CHANNEL: a decay per channel, nothing removed
+enum { LSR_RETENTION = 0, LSR_DELTA = 1, LSR_GENERAL = 2 };
 
 // Rows of one token in the ring, by mode: k (kw), q always; w for the modes with a decay per channel; p and z for the
 // general form.
-__host__ __device__ constexpr int lsr_rows(int mode) { return mode == LSR_RETENTION ? 2 : mode == LSR_DELTA || mode == LSR_CHANNEL ? 3 : 5; }
+__host__ __device__ constexpr int lsr_rows(int mode) { return mode == LSR_RETENTION ? 2 : mode == LSR_DELTA ? 3 : 5; }
 __host__ __device__ constexpr int lsr_chunk(int dpl) { return dpl <= 8 ? 16 : 8; }
 
 // kw, q, w, p, z: [T, H, D] float32 (w, p, z only where the mode reads them); v: [T, H, Dv]; scal: [T, H, 2] = (qk, qp);
@@ -647,7 +646,7 @@ __global__ void __launch_bounds__(GS_BLOCK, 1) lsr_scan_kernel(
                         const float4 kk = k4[i];       // a = k . (w s)
                         a0 = fmaf(d0, kk.x, a0); a1 = fmaf(d1, kk.y, a1);
                         a0 = fmaf(d2, kk.z, a0); a1 = fmaf(d3, kk.w, a1);
-                    } else if (MODE == LSR_GENERAL) {
+                    } else {
                         const float4 zz = z4[i];       // the unit key: a = u . s on the state before the decay
                         a0 = fmaf(s[4 * i], zz.x, a0);     a1 = fmaf(s[4 * i + 1], zz.y, a1);
                         a0 = fmaf(s[4 * i + 2], zz.z, a0); a1 = fmaf(s[4 * i + 3], zz.w, a1);
@@ -655,7 +654,7 @@ __global__ void __launch_bounds__(GS_BLOCK, 1) lsr_scan_kernel(
                 }
             }
             float a = a0 + a1, c = c0 + c1;
-            if (MODE != LSR_RETENTION && MODE != LSR_CHANNEL) {
+            if (MODE != LSR_RETENTION) {
                 a += __shfl_xor_sync(0xffffffffu, a, 1);
                 a += __shfl_xor_sync(0xffffffffu, a, 2);
                 a += __shfl_xor_sync(0xffffffffu, a, 4);
@@ -678,12 +677,6 @@ __global__ void __launch_bounds__(GS_BLOCK, 1) lsr_scan_kernel(
                     s[4 * i + 1] = fmaf(kk.y, u, ww.y * s[4 * i + 1]);
                     s[4 * i + 2] = fmaf(kk.z, u, ww.z * s[4 * i + 2]);
                     s[4 * i + 3] = fmaf(kk.w, u, ww.w * s[4 * i + 3]);
-                } else if (MODE == LSR_CHANNEL) {
-                    const float4 ww = w4[i];
-                    s[4 * i] = fmaf(kk.x, vv, ww.x * s[4 * i]);
-                    s[4 * i + 1] = fmaf(kk.y, vv, ww.y * s[4 * i + 1]);
-                    s[4 * i + 2] = fmaf(kk.z, vv, ww.z * s[4 * i + 2]);
-                    s[4 * i + 3] = fmaf(kk.w, vv, ww.w * s[4 * i + 3]);
                 } else {
                     const float4 ww = w4[i], pp = p4[i];
                     s[4 * i] = fmaf(kk.x, vv, fmaf(-pp.x, a, ww.x * s[4 * i]));
@@ -696,7 +689,6 @@ __global__ void __launch_bounds__(GS_BLOCK, 1) lsr_scan_kernel(
                 float o;
                 if (MODE == LSR_RETENTION) o = fmaf(qk, vv, hd * c);
                 else if (MODE == LSR_DELTA) o = fmaf(qk, vv - a, c);
-                else if (MODE == LSR_CHANNEL) o = fmaf(qk, vv, c);
                 else o = fmaf(qk, vv, fmaf(-qp, a, c));
                 o_s[tt * GS_COLS + ci] = o;
             }
@@ -733,14 +725,14 @@ static cudaError_t lsr_launch(dim3 grid, cudaStream_t s, const float* kw, const 
 }
 
 // mode: 0 retention (head_decay [H]; w, p, z unused), 1 delta rule with a decay per key channel (kw = k, w = g,
-// scal = (beta q . k, beta); p, z unused), 2 the general form, 3 a decay per key channel alone (p, z unused).  state: [slots, imp_gdr_state_floats(H, D, Dv)], zero at a request's start, updated in place.
+// scal = (beta q . k, beta); p, z unused), 2 the general form.  state: [slots, imp_gdr_state_floats(H, D, Dv)], zero at a request's start, updated in place.
 // All vectors are [n_tokens, H, D] float32, v and out [n_tokens, H, Dv], scal [n_tokens, H, 2] = (q . kw, q . p).
 IMP_API int imp_lsr_scan(int mode, const float* kw, const float* q, const float* w, const float* p, const float* z, const float* v,
                          const float* scal, const float* head_decay, float* state, float* out, const int* q_start, const int* slots,
                          int n_seqs, int D, int H, int Dv, void* stream) {
     if (n_seqs == 0) return 0;
     IMP_CHECK_ARG(kw && q && v && scal && state && out && q_start && slots, "imp_lsr_scan: null pointer");
-    IMP_CHECK_ARG(mode >= 0 && mode <= 3, "imp_lsr_scan: unknown mode %d", mode);
+    IMP_CHECK_ARG(mode >= 0 && mode <= 2, "imp_lsr_scan: unknown mode %d", mode);
     IMP_CHECK_ARG(mode == LSR_RETENTION ? head_decay != nullptr : w != nullptr, "imp_lsr_scan: the mode's decay is missing");
     IMP_CHECK_ARG(mode != LSR_GENERAL || (p && z), "imp_lsr_scan: the general form reads p and z");
     IMP_CHECK_ARG(D > 0 && Dv > 0 && H > 0 && H <= 65535 && n_seqs <= 65535, "imp_lsr_scan: bad sizes");
@@ -761,7 +753,6 @@ IMP_API int imp_lsr_scan(int mode, const float* kw, const float* q, const float*
     do {                                                \
         if (mode == LSR_RETENTION) LSR_SCAN_M(DPL, 0);  \
         else if (mode == LSR_DELTA) LSR_SCAN_M(DPL, 1); \
-        else if (mode == LSR_CHANNEL) LSR_SCAN_M(DPL, 3); \
         else LSR_SCAN_M(DPL, 2);                        \
     } while (0)
     switch (gdr_dims_per_lane(D)) {
@@ -973,172 +964,6 @@ __global__ void __launch_bounds__(GC_MAX_WARPS * 32) gdrc_prepare_kernel(
     }
 }
 
-// ------------------------------------------------------------------------------- gated linear attention
-// proj columns [q: H*D | k: H*D | v: H*Dv | gate: H*Dv | low: R | ...]; the decay of head h's key channel d is
-//   alpha = sigmoid(z)^(1/tau),  z = sum_j low[j] * W_a2[h*D + d, j] + bias[h*D + d]
-// made as exp(-softplus(-z) / tau), everything after the projections in 32-bit.  w2t: W_a2 transposed, float32 [R, H*D], so that
-// neighbouring channels read neighbouring words.  q is scaled by q_scale.
-__device__ __forceinline__ float gla_decay(float z, float inv_tau) {
-    const float sp = fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z)));   // softplus(-z) = -log sigmoid(z)
-    return expf(-sp * inv_tau);
-}
-
-// The vectors of imp_lsr_scan (mode 3): a CTA per (head, GLA_TOKENS tokens), a thread per key channel; W_a2's column is read
-// once for the CTA's tokens.  z sums over j ascending; q . k per warp of 32 channels, then the warps in order.
-constexpr int GLA_TOKENS = 8;
-template <typename TA>
-__global__ void __launch_bounds__(LP_MAX_D) gla_prepare_kernel(const TA* __restrict__ proj, int64_t ld, int n_tokens, int H, int D, int Dv, int R,
-                                                               const float* __restrict__ w2t, const float* __restrict__ bias, float inv_tau,
-                                                               float q_scale, float* __restrict__ q, float* __restrict__ kw, float* __restrict__ w,
-                                                               float* __restrict__ v, float* __restrict__ scal) {
-    pdl_wait();
-    pdl_launch_dependents();
-    extern __shared__ __align__(16) float gla_low[];   // [R][GLA_TOKENS]
-    __shared__ float red[GLA_TOKENS][LP_MAX_D / 32];
-    const int d = threadIdx.x, lane = d & 31, warp = d >> 5, n_warps = blockDim.x >> 5;
-    const int h = blockIdx.y, t0 = blockIdx.x * GLA_TOKENS, nt = min(GLA_TOKENS, n_tokens - t0);
-    const int64_t HD = (int64_t)H * D, HV = (int64_t)H * Dv, low0 = 2 * HD + 2 * HV;
-    for (int e = d; e < R * GLA_TOKENS; e += blockDim.x) {
-        const int tt = e / R, j = e - tt * R;
-        gla_low[j * GLA_TOKENS + tt] = tt < nt ? to_float(proj[(int64_t)(t0 + tt) * ld + low0 + j]) : 0.f;
-    }
-    __syncthreads();
-    const bool on = d < D;
-    float z[GLA_TOKENS];
-#pragma unroll
-    for (int tt = 0; tt < GLA_TOKENS; ++tt) z[tt] = 0.f;
-    if (on) {
-        const float* col = w2t + (int64_t)h * D + d;
-#pragma unroll 4
-        for (int j = 0; j < R; ++j) {
-            const float wv = col[(int64_t)j * HD];
-            const float4 a = *reinterpret_cast<const float4*>(gla_low + j * GLA_TOKENS), b = *reinterpret_cast<const float4*>(gla_low + j * GLA_TOKENS + 4);
-            z[0] = fmaf(a.x, wv, z[0]), z[1] = fmaf(a.y, wv, z[1]), z[2] = fmaf(a.z, wv, z[2]), z[3] = fmaf(a.w, wv, z[3]);
-            z[4] = fmaf(b.x, wv, z[4]), z[5] = fmaf(b.y, wv, z[5]), z[6] = fmaf(b.z, wv, z[6]), z[7] = fmaf(b.w, wv, z[7]);
-        }
-    }
-    const float zb = on ? bias[(int64_t)h * D + d] : 0.f;
-#pragma unroll
-    for (int tt = 0; tt < GLA_TOKENS; ++tt) {
-        if (tt >= nt) break;
-        const int64_t t = t0 + tt;
-        const TA* row = proj + t * ld + (int64_t)h * D;
-        float qq = 0.f, kk = 0.f;
-        if (on) {
-            qq = to_float(row[d]) * q_scale;
-            kk = to_float(row[HD + d]);
-            const int64_t o = (t * H + h) * D + d;
-            q[o] = qq;
-            kw[o] = kk;
-            w[o] = gla_decay(z[tt] + zb, inv_tau);
-        }
-        const float dot = warp_sum(qq * kk);
-        if (lane == 0) red[tt][warp] = dot;
-        for (int c = d; c < Dv; c += blockDim.x) v[(t * H + h) * Dv + c] = to_float(proj[t * ld + 2 * HD + (int64_t)h * Dv + c]);
-    }
-    __syncthreads();
-    if (d < nt) {
-        float dot = 0.f;
-        for (int i = 0; i < n_warps; ++i) dot += red[d][i];
-        scal[((t0 + d) * (int64_t)H + h) * 2] = dot;
-        scal[((t0 + d) * (int64_t)H + h) * 2 + 1] = 0.f;
-    }
-}
-
-// A step of single tokens in one kernel: the vectors of a token's head, the recurrence on that head's state, the read-out's norm
-// and its gate.  A CTA per (head, sequence); the state has the scan's layout, and every sum has the order of the kernels that
-// run for portions (gla_prepare, lsr_scan, gdr_output), so a decoded token's state and read-out are theirs to the bit.
-template <typename TA, int DPL>
-__global__ void __launch_bounds__(GS_BLOCK) gla_decode_kernel(const TA* __restrict__ proj, int64_t ld, int H, int D, int Dv, int R,
-                                                              const float* __restrict__ w2t, const float* __restrict__ bias, float inv_tau,
-                                                              float q_scale, const float* __restrict__ out_w, float eps, float* __restrict__ state,
-                                                              const int* __restrict__ slots, TA* __restrict__ y) {
-    pdl_wait();
-    pdl_launch_dependents();
-    constexpr int ROW = DPL + 4;
-    extern __shared__ __align__(16) float gla_smem[];   // o [Dv], low [R]
-    __shared__ __align__(16) float k_s[GS_LANES * ROW], q_s[GS_LANES * ROW], w_s[GS_LANES * ROW];
-    __shared__ float red[GS_BLOCK / 32];
-    float* o_s = gla_smem;
-    float* low_s = gla_smem + Dv;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, r = tid & (GS_LANES - 1), ci = tid / GS_LANES;
-    const int h = blockIdx.x;
-    const int64_t t = blockIdx.y;
-    const int64_t HD = (int64_t)H * D, HV = (int64_t)H * Dv;
-    const TA* row = proj + t * ld;
-    const int n_blocks = (Dv + GS_COLS - 1) / GS_COLS;
-    float* S = state + (((int64_t)slots[t] * H + h) * n_blocks) * DPL * GS_BLOCK + tid;
-    float s[DPL];
-#pragma unroll
-    for (int i = 0; i < DPL; ++i) s[i] = S[i * GS_BLOCK];
-    for (int j = tid; j < R; j += GS_BLOCK) low_s[j] = to_float(row[2 * HD + 2 * HV + j]);
-    __syncthreads();
-    float qq = 0.f, kk = 0.f, ww = 0.f;
-    if (tid < D) {
-        qq = to_float(row[(int64_t)h * D + tid]) * q_scale;
-        kk = to_float(row[HD + (int64_t)h * D + tid]);
-        float z = 0.f;
-        const float* col = w2t + (int64_t)h * D + tid;
-#pragma unroll 4
-        for (int j = 0; j < R; ++j) z = fmaf(low_s[j], col[(int64_t)j * HD], z);
-        ww = gla_decay(z + bias[(int64_t)h * D + tid], inv_tau);
-    }
-    if (tid < GS_LANES * DPL) {
-        const int at = (tid / DPL) * ROW + tid % DPL;
-        q_s[at] = qq;
-        k_s[at] = kk;
-        w_s[at] = ww;
-    }
-    const float part = warp_sum(qq * kk);
-    if (lane == 0) red[warp] = part;
-    __syncthreads();
-    float qk = 0.f;
-    for (int i = 0; i < (D + 31) / 32; ++i) qk += red[i];
-    const float4* k4 = reinterpret_cast<const float4*>(k_s + r * ROW);
-    const float4* q4 = reinterpret_cast<const float4*>(q_s + r * ROW);
-    const float4* w4 = reinterpret_cast<const float4*>(w_s + r * ROW);
-    for (int cb = 0; cb < n_blocks; ++cb) {
-        float next[DPL];
-        if (cb + 1 < n_blocks) {
-#pragma unroll
-            for (int i = 0; i < DPL; ++i) next[i] = S[(int64_t)(cb + 1) * DPL * GS_BLOCK + i * GS_BLOCK];
-        }
-        const int c = cb * GS_COLS + ci;
-        const float vv = c < Dv ? to_float(row[2 * HD + (int64_t)h * Dv + c]) : 0.f;
-        float c0 = 0.f, c1 = 0.f;
-#pragma unroll
-        for (int i = 0; i < DPL / 4; ++i) {
-            const float4 qv = q4[i], wv = w4[i], kv = k4[i];
-            const float d0 = wv.x * s[4 * i], d1 = wv.y * s[4 * i + 1], d2 = wv.z * s[4 * i + 2], d3 = wv.w * s[4 * i + 3];
-            c0 = fmaf(d0, qv.x, c0), c1 = fmaf(d1, qv.y, c1);
-            c0 = fmaf(d2, qv.z, c0), c1 = fmaf(d3, qv.w, c1);
-            s[4 * i] = fmaf(kv.x, vv, d0);
-            s[4 * i + 1] = fmaf(kv.y, vv, d1);
-            s[4 * i + 2] = fmaf(kv.z, vv, d2);
-            s[4 * i + 3] = fmaf(kv.w, vv, d3);
-        }
-        float o = c0 + c1;
-        o += __shfl_xor_sync(0xffffffffu, o, 1);
-        o += __shfl_xor_sync(0xffffffffu, o, 2);
-        o += __shfl_xor_sync(0xffffffffu, o, 4);
-        if (r == 0 && c < Dv) o_s[c] = fmaf(qk, vv, o);
-#pragma unroll
-        for (int i = 0; i < DPL; ++i) {
-            S[(int64_t)cb * DPL * GS_BLOCK + i * GS_BLOCK] = s[i];
-            s[i] = next[i];
-        }
-    }
-    __syncthreads();
-    float ss = 0.f;
-    for (int c = lane; c < Dv; c += 32) ss = fmaf(o_s[c], o_s[c], ss);
-    ss = warp_sum(ss);
-    const float inv = rsqrtf(ss / (float)Dv + eps);
-    for (int c = tid; c < Dv; c += GS_BLOCK) {
-        const float g = to_float(row[2 * HD + HV + (int64_t)h * Dv + c]);
-        y[(t * H + h) * Dv + c] = from_float<TA>(o_s[c] * inv * out_w[c] * silu_f(g));
-    }
-}
-
 static unsigned lp_grid(int64_t items) { return (unsigned)((items + GP_BLOCK / 32 - 1) / (GP_BLOCK / 32)); }
 
 IMP_API int imp_retention_prepare_ex(const void* proj, int64_t ld, int n_tokens, int H, int D, int Dv, float k_scale, int act, float* q, float* kw,
@@ -1208,60 +1033,4 @@ IMP_API int imp_gdrc_prepare(const void* proj, int64_t ld, const float* conv_w, 
 #undef GDRC_PREPARE_T
 #undef GDRC_PREPARE
     IMP_RETURN_LAUNCH();
-}
-
-// Gated linear attention, see gla_prepare_kernel: the vectors of imp_lsr_scan mode 3.
-IMP_API int imp_gla_prepare(const void* proj, int64_t ld, int n_tokens, int H, int D, int Dv, int R, const float* w2t, const float* bias, float tau,
-                            float q_scale, float* q, float* kw, float* w, float* v, float* scal, int act_dtype, void* stream) {
-    if (n_tokens == 0) return 0;
-    IMP_CHECK_ARG(proj && w2t && bias && q && kw && w && v && scal, "imp_gla_prepare: null pointer");
-    IMP_CHECK_ARG(H > 0 && H <= 65535 && D > 0 && D <= LP_MAX_D && Dv > 0 && R > 0 && tau > 0.f && ld >= 2 * ((int64_t)H * D + (int64_t)H * Dv) + R,
-                  "imp_gla_prepare: bad sizes (key size %d of at most %d)", D, LP_MAX_D);
-    const size_t smem = (size_t)R * GLA_TOKENS * 4;
-    IMP_CHECK_ARG(smem <= 46 * 1024, "imp_gla_prepare: an inner size of %d is more than this kernel holds", R);
-    cudaStream_t s = (cudaStream_t)stream;
-    const dim3 grid((n_tokens + GLA_TOKENS - 1) / GLA_TOKENS, H), block(32 * ((D + 31) / 32));
-    if (act_dtype == IMP_F32)
-        imp_launch(gla_prepare_kernel<float>, grid, block, smem, s, (const float*)proj, ld, n_tokens, H, D, Dv, R, w2t, bias, 1.f / tau, q_scale, q, kw, w,
-                   v, scal);
-    else
-        imp_launch(gla_prepare_kernel<__nv_bfloat16>, grid, block, smem, s, (const __nv_bfloat16*)proj, ld, n_tokens, H, D, Dv, R, w2t, bias, 1.f / tau,
-                   q_scale, q, kw, w, v, scal);
-    IMP_RETURN_LAUNCH();
-}
-
-// A step of single tokens (token t belongs to sequence t): projection to gated read-out y [n_tokens, H * Dv], the state updated.
-IMP_API int imp_gla_decode(const void* proj, int64_t ld, int n_tokens, int H, int D, int Dv, int R, const float* w2t, const float* bias, float tau,
-                           float q_scale, const float* out_w, float eps, float* state, const int* slots, void* y, int act_dtype, void* stream) {
-    if (n_tokens == 0) return 0;
-    IMP_CHECK_ARG(proj && w2t && bias && out_w && state && slots && y, "imp_gla_decode: null pointer");
-    IMP_CHECK_ARG(H > 0 && D > 0 && D <= LP_MAX_D && Dv > 0 && R > 0 && tau > 0.f && n_tokens <= 65535 &&
-                      ld >= 2 * ((int64_t)H * D + (int64_t)H * Dv) + R,
-                  "imp_gla_decode: bad sizes (key size %d of at most %d)", D, LP_MAX_D);
-    const size_t smem = (size_t)(Dv + R) * 4;
-    if (smem > 40 * 1024) return IMP_ERR_UNSUPPORTED;
-    cudaStream_t s = (cudaStream_t)stream;
-    const dim3 grid(H, n_tokens);
-    cudaError_t e;
-#define GLA_DECODE_T(TA, DPL)                                                                                                                \
-    e = imp_launch(gla_decode_kernel<TA, DPL>, grid, dim3(GS_BLOCK), smem, s, (const TA*)proj, ld, H, D, Dv, R, w2t, bias, 1.f / tau, q_scale, \
-                   out_w, eps, state, slots, (TA*)y)
-#define GLA_DECODE(DPL)                                      \
-    do {                                                     \
-        if (act_dtype == IMP_F32) GLA_DECODE_T(float, DPL);  \
-        else GLA_DECODE_T(__nv_bfloat16, DPL);               \
-    } while (0)
-    switch (gdr_dims_per_lane(D)) {
-        case 4: GLA_DECODE(4); break;
-        case 8: GLA_DECODE(8); break;
-        case 16: GLA_DECODE(16); break;
-        default: GLA_DECODE(32); break;
-    }
-#undef GLA_DECODE
-#undef GLA_DECODE_T
-    if (e != cudaSuccess) {
-        imp_set_error("imp_gla_decode: %s", cudaGetErrorString(e));
-        return (int)e;
-    }
-    return 0;
 }

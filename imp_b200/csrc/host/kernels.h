@@ -151,12 +151,16 @@ int imp_gdrc_prepare(const void* proj, int64_t ld, const float* conv_w, int taps
                      const int* q_start, const int* slots, int n_tokens, int n_seqs, int G, int D, int H, int Dv, const float* dpre,
                      const float* a_log, const float* dt_bias, float unit_eps, float* q, float* kw, float* w, float* v, float* scal,
                      int act_dtype, int* status, void* stream);
-int imp_gla_prepare(const void* proj, int64_t ld, int n_tokens, int H, int D, int Dv, int R, const float* w2t, const float* bias, float tau,
-                    float q_scale, float* q, float* kw, float* w, float* v, float* scal, int act_dtype, void* stream);
-int imp_gla_decode(const void* proj, int64_t ld, int n_tokens, int H, int D, int Dv, int R, const float* w2t, const float* bias, float tau,
-                   float q_scale, const float* out_w, float eps, float* state, const int* slots, void* y, int act_dtype, void* stream);
 int imp_gdr_output_ex(void* y, const float* o, const void* gate, int64_t gate_ld, const float* w, int w_head_stride, int gate_act,
                       float eps, int n_tokens, int H, int Dv, int act_dtype, void* stream);
+// gated linear attention (gla.cu)
+int64_t imp_gla_state_floats(int H, int D, int Dv);
+int imp_gla_decay(float* alpha, const void* low, int64_t ld, int n_tokens, int n, int R, const float* w2t, const float* bias, float tau, int act_dtype,
+                  void* stream);
+int imp_gla_scan(const void* proj, int64_t ld, const float* alpha, float q_scale, float* state, float* out, const int* q_start, const int* slots,
+                 int n_seqs, int D, int H, int Dv, int act_dtype, void* stream);
+int imp_gla_decode(const void* proj, int64_t ld, int n_tokens, int H, int D, int Dv, int R, const float* w2t, const float* bias, float tau,
+                   float q_scale, const float* out_w, float eps, float* state, const int* slots, void* y, int act_dtype, void* stream);
 // attention with normalised, partly rotated, scaled and gated heads; blocks of two mixers (qkv_prepare.cu)
 int imp_qkv_prepare(const void* proj, int64_t ld, int n_tokens, int Hq, int Hkv, int D, int Dv, int Dc, const float* q_norm_w,
                     const float* k_norm_w, float eps, int v_norm, const float* inv_freq, int rot, const float* head_mult,

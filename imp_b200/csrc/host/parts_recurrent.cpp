@@ -1,5 +1,5 @@
-// Part kinds: four recurrent mixers over the general scan of csrc/delta_rule.cu (retention, gated linear attention, the generalised
-// delta rule, the delta rule with a decay per key channel), softmax attention whose heads are normalised, rotated in part,
+// Part kinds: three recurrent mixers over the general scan of csrc/delta_rule.cu (retention, the generalised delta rule, the
+// delta rule with a decay per key channel), gated linear attention over the scan of csrc/gla.cu, softmax attention whose heads are normalised, rotated in part,
 // scaled, masked by chunks and gated, and a post-norm block (the normalised sum is the stream) that holds one mixer
 // or two side by side.  Every size and constant is a parameter; no kind knows which model it is in.
 #include <cmath>
@@ -174,8 +174,8 @@ struct Retention : Mixer {
 // q = query_scale W_q x, k = W_k x (H heads of D), v = W_v x (H heads of Dv); a decay per head and key channel,
 // alpha = sigmoid(W_a2 (W_a1 x) + b_a)^(1/tau);
 //   S <- diag(alpha) S + k v^T;  o = S^T q;  y = o / rms(o) per head * w_norm [Dv] * silu(W_g x);  out = W_o y.
-// Portions run prepare, scan (the general scan with a decay per channel and nothing removed) and output kernels; a step of single
-// tokens is one kernel from the projections to y (csrc/delta_rule.cu).
+// Portions run a kernel for the decays, the scan and the read-out's norm and gate; a step of single tokens is one kernel from the
+// projections to y (csrc/gla.cu).
 // State per request: S (H heads of D x Dv, float32), zero at the start.
 // params: hidden_size, num_heads, key_dim, value_dim, tau, query_scale (default key_dim^-1/2), norm_eps, decay_rank (0 or absent: the
 //         rows of the checkpoint's W_a1).
@@ -210,7 +210,10 @@ struct GatedLinearAttention : Mixer {
     }
     static CacheSpec cache(const Json& p) {
         const Sizes z = sizes(p);
-        return scan_state(z.H, z.D, z.Dv);
+        CacheSpec s;
+        s.kind = CacheSpec::State;
+        s.states.push_back(StateTensorSpec{"S", {imp_gla_state_floats((int)z.H, (int)z.D, (int)z.Dv)}, F32});   // in the kernels' own layout
+        return s;
     }
     explicit GatedLinearAttention(BuildArgs& a) {
         const char* me = "gated_linear_attention";
@@ -249,16 +252,18 @@ struct GatedLinearAttention : Mixer {
             rc = imp_gla_decode(proj.data, proj.stride0, (int)T, H, D, Dv, rank, (const float*)w2t.data, (const float*)a_bias.data, tau, q_scale,
                                 (const float*)out_norm.data, eps, S, st.view.state_slots, y.data, rt.dtype, rt.stream);
         if (rc == -2) {
-            ScanBuffers b(rt, T, H, D, Dv, true, false);
+            const int64_t HD = (int64_t)H * D, HV = (int64_t)H * Dv;
+            float* alpha = rt.arena->take<float>((size_t)(T * HD));
+            float* o = rt.arena->take<float>((size_t)(T * HV));
             rt.launches += 3;
-            check_launch(imp_gla_prepare(proj.data, proj.stride0, (int)T, H, D, Dv, rank, (const float*)w2t.data, (const float*)a_bias.data, tau, q_scale,
-                                         b.q, b.kw, b.w, b.v, b.scal, rt.dtype, rt.stream),
-                         "gla_prepare");
-            check_launch(imp_lsr_scan(3, b.kw, b.q, b.w, nullptr, nullptr, b.v, b.scal, nullptr, S, b.o, st.view.q_start, st.view.state_slots, st.B(), D,
-                                      H, Dv, rt.stream),
-                         "lsr_scan");
-            const Tensor gate = col_slice(proj, (int64_t)2 * H * D + (int64_t)H * Dv, (int64_t)H * Dv);
-            check_launch(imp_gdr_output_ex(y.data, b.o, gate.data, gate.stride0, (const float*)out_norm.data, 0, 0, eps, (int)T, H, Dv, rt.dtype, rt.stream),
+            check_launch(imp_gla_decay(alpha, col_slice(proj, 2 * HD + 2 * HV, rank).data, proj.stride0, (int)T, (int)HD, rank, (const float*)w2t.data,
+                                       (const float*)a_bias.data, tau, rt.dtype, rt.stream),
+                         "gla_decay");
+            check_launch(imp_gla_scan(proj.data, proj.stride0, alpha, q_scale, S, o, st.view.q_start, st.view.state_slots, st.B(), D, H, Dv, rt.dtype,
+                                      rt.stream),
+                         "gla_scan");
+            const Tensor gate = col_slice(proj, 2 * HD + HV, HV);
+            check_launch(imp_gdr_output_ex(y.data, o, gate.data, gate.stride0, (const float*)out_norm.data, 0, 0, eps, (int)T, H, Dv, rt.dtype, rt.stream),
                          "gdr_output");
         } else {
             ++rt.launches;
