@@ -108,17 +108,50 @@ struct BigramEmbedding : Embedding {
 // ------------------------------------------------------------------------------------ sublayers side by side
 // x = norm(h);  h += m (mixer(x) + ffn(x)): one norm, read by both sublayers.  The two outputs travel as the two summands of one
 // branch, unsummed parts and routed rows included, to the norm that adds them; where that norm takes plain branches only, the sum
-// is worked out first.
+// is worked out first.  In steps of single tokens, where each sublayer is a chain of short launches, the feed-forward runs on a
+// stream of its own beside the mixer (a fork after the norm, a join before the branch is handed on; a captured graph has the same
+// two paths); IMP_B200_PARALLEL_STREAMS=0 runs them one after the other.
 // Slots: norm, mixer, and with has_ffn (default true) feed_forward.  params: residual_mult (default 1), has_ffn.
 struct ParallelBlock : Block {
     Norm* norm;
     Mixer* mixer_;
     FeedForward* ffn = nullptr;
     float mult;
+    cudaStream_t side = nullptr;
+    cudaEvent_t fork = nullptr, join = nullptr;
+    ~ParallelBlock() override {
+        if (side) cudaStreamDestroy(side);
+        if (fork) cudaEventDestroy(fork);
+        if (join) cudaEventDestroy(join);
+    }
     explicit ParallelBlock(BuildArgs& a)
         : norm(part_cast<Norm>(a.part("norm"), "a norm")), mixer_(part_cast<Mixer>(a.part("mixer"), "a mixer")),
           mult((float)a.params.get_double("residual_mult", 1.0)) {
-        if (a.params.get_bool("has_ffn", true)) ffn = part_cast<FeedForward>(a.part("feed_forward"), "a feed-forward");
+        if (!a.params.get_bool("has_ffn", true)) return;
+        ffn = part_cast<FeedForward>(a.part("feed_forward"), "a feed-forward");
+        if (mixer_->graph_safe() && ffn->graph_safe() && env_flag("IMP_B200_PARALLEL_STREAMS", true)) {
+            IMP_CUDA(cudaStreamCreateWithFlags(&side, cudaStreamNonBlocking));
+            IMP_CUDA(cudaEventCreateWithFlags(&fork, cudaEventDisableTiming));
+            IMP_CUDA(cudaEventCreateWithFlags(&join, cudaEventDisableTiming));
+        }
+    }
+    // The feed-forward on the side stream, from what the step's stream holds so far; `join` stands behind it.
+    Branch forked_ffn(Step& st, const Tensor& x) {
+        Runtime& rt = *st.rt;
+        const cudaStream_t main = rt.stream;
+        IMP_CUDA(cudaEventRecord(fork, main));
+        IMP_CUDA(cudaStreamWaitEvent(side, fork, 0));
+        rt.stream = side;
+        Branch f;
+        try {
+            f = ffn->forward(st, x);
+        } catch (...) {
+            rt.stream = main;
+            throw;
+        }
+        rt.stream = main;
+        IMP_CUDA(cudaEventRecord(join, side));
+        return f;
     }
     static std::vector<Slot> slots(const Json& p) {
         std::vector<Slot> s = {{"norm", "norm"}, {"mixer", "mixer"}};
@@ -143,12 +176,18 @@ struct ParallelBlock : Block {
     Branch forward(Step& st, Tensor h, const Branch& pending, LayerCache* cache) override {
         Tensor x = norm->add_norm(st, h, pending);
         mixer_->defer_out = defer_pending && pair_pending;
-        Branch out = mixer_->forward(st, x, cache);
-        stage(st, "mixer", out);
         if (ffn) {
             ffn->defer_out = defer_pending && pair_pending;
             ffn->defer_rows = pair_pending;
-            const Branch f = ffn->forward(st, x);
+        }
+        const bool forked = ffn && side && st.decode_only() && !st.diag;
+        Branch f;
+        if (forked) f = forked_ffn(st, x);
+        Branch out = mixer_->forward(st, x, cache);
+        stage(st, "mixer", out);
+        if (ffn) {
+            if (forked) IMP_CUDA(cudaStreamWaitEvent(st.rt->stream, join, 0));
+            else f = ffn->forward(st, x);
             stage(st, "feed_forward", f.rows.y ? Branch() : f);
             if (f.col_scale || f.own_norm.weight || f.mult != 1.f || !f.second.empty()) fail(IMP_ERROR_INTERNAL, "parallel: a feed-forward returns a plain branch");
             out.second.t = f.t;

@@ -7,6 +7,8 @@
 // head's latent-space query; latent_prepare can do this as well, where the query's product is done before it.  A page's vector
 // and a head's query may be padded with zeros to a whole multiple of 16.  Norms, angles and rotations are 32-bit; the rotation
 // pairs entry i with i + dims/2 (pairing 0) or 2i with 2i + 1 (pairing 1).
+#include <algorithm>
+
 #include "common.cuh"
 
 namespace {
@@ -49,7 +51,9 @@ __global__ void __launch_bounds__(LP_BLOCK_MAX) latent_prepare_kernel(
     const int t = blockIdx.x, tid = threadIdx.x, n_thr = blockDim.x;
     const TA* row = proj + (int64_t)t * ld;
     float ss = 0.f, inv;
-    if (q_rank > 0) {
+    // CTA (t, 0) does the norms and the cache write of token t, CTAs (t, 1 ...) share its query heads
+    const bool query_cta = blockIdx.y > 0;
+    if (q_rank > 0 && !query_cta) {
         // the query latent
         for (int i = tid; i < q_rank; i += n_thr) {
             const float v = to_float(row[i]);
@@ -66,15 +70,16 @@ __global__ void __launch_bounds__(LP_BLOCK_MAX) latent_prepare_kernel(
     }
     const float* cos_row = cos_tab + (int64_t)pos * (rot_dims / 2);
     const float* sin_row = sin_tab + (int64_t)pos * (rot_dims / 2);
-    if (qp.H > 0) {
+    if (query_cta) {
         // the rotated part of every head's query, behind that head's latent-space query
         const int per = rot + qp.pad;
-        for (int e = tid; e < qp.H * per; e += n_thr) {
+        for (int e = (blockIdx.y - 1) * n_thr + tid; e < qp.H * per; e += (gridDim.y - 1) * n_thr) {
             const int h = e / per, i = e - h * per;
             const TA* src = qp.q + (int64_t)t * qp.q_ld + (int64_t)h * qp.q_head;
             qp.out[(int64_t)t * qp.out_ld + (int64_t)h * qp.out_head + i] =
                 from_float<TA>(i < rot ? rotated_entry(src, i, rot_dims, pairing, cos_row, sin_row) : 0.f);
         }
+        return;
     }
     // the key/value latent and the rotated key part go to the token's place in the pages
     if (!pages) return;
@@ -129,7 +134,10 @@ cudaError_t launch_prepare(const void* proj, int64_t ld, int n_tokens, int q_ran
                            int page_len, int page_size, int num_pages, const void* q, int64_t q_ld, int q_head, void* q_out, int64_t q_out_ld, int H,
                            int* status, cudaStream_t s) {
     QueryParts<TA> qp{(const TA*)q, q_ld, q_head, (TA*)q_out, q_out_ld, page_len, q ? H : 0, page_len - kv_rank - rot};
-    return imp_launch(latent_prepare_kernel<TA>, dim3(n_tokens), dim3(qp.H * rot > 512 ? LP_BLOCK_MAX : LP_BLOCK), 0, s, (const TA*)proj, ld, q_rank,
+    // a step of few tokens spreads a token's query heads over several CTAs
+    const int block = qp.H * rot > 512 ? LP_BLOCK_MAX : LP_BLOCK, work = (qp.H * (page_len - kv_rank) + block - 1) / block;
+    const int query_ctas = qp.H > 0 ? std::max(1, std::min(work, 2 * imp_sm_count() / std::max(n_tokens, 1))) : 0;
+    return imp_launch(latent_prepare_kernel<TA>, dim3(n_tokens, 1 + query_ctas), dim3(block), 0, s, (const TA*)proj, ld, q_rank,
                       kv_rank, rot, wq, wkv, eps, (TA*)cq, cq_ld, cos_tab, sin_tab, rot_dims, pairing, max_pos, positions, seq_of_token, block_table,
                       bt_stride, n_seqs, (TA*)pages, page_len, page_size, num_pages, qp, status);
 }
