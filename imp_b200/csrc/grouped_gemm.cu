@@ -38,6 +38,7 @@ struct GroupedArgs {
     int vec;   // rows of A and W start on 16 bytes and K is a multiple of 8 (bfloat16) / 4 (float32)
     const void* gate;   // GG_SIGMOID_GATE: rows gate_ld apart, in the activations' type
     int64_t gate_ld;
+    int pairs; // bfloat16 outputs (and gates) may move two at a time: N even, rows and groups of C (and the gate) on 4 bytes
     int il;    // the gated epilogue's two matrices are one, gate and up rows alternating in runs of 8 (W2 unused)
 };
 
@@ -176,6 +177,22 @@ __global__ void __launch_bounds__(128) grouped_gemm_bf16_kernel(const GroupedArg
                 if (SWIGLU) acu[i][j][e] = 0.f;
             }
 
+    // the gate's values are asked for before the walk over k, so that they are there when it ends
+    uint32_t gate_z[EPI == GG_SIGMOID_GATE ? MI : 1][2][2 * NJ];
+    if (EPI == GG_SIGMOID_GATE && p.pairs) {
+#pragma unroll
+        for (int i = 0; i < MI; ++i)
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                const int lr = row0 + wm + i * 16 + gid + half * 8;
+#pragma unroll
+                for (int j = 0; j < 2 * NJ; ++j) {
+                    const int n = n0 + wn + j * 8 + 2 * tig;
+                    gate_z[i][half][j] = lr < row_end && n < p.N ? *reinterpret_cast<const uint32_t*>((const __nv_bfloat16*)p.gate + lr * p.gate_ld + p.c_group_cols * g + n) : 0u;
+                }
+            }
+    }
+
     const int n_k = (p.K + GB_BK - 1) / GB_BK;
     auto fetch = [&](int kb) {
         if (kb < n_k) {
@@ -229,16 +246,34 @@ __global__ void __launch_bounds__(128) grouped_gemm_bf16_kernel(const GroupedArg
             if (lr >= row_end) continue;
             __nv_bfloat16* crow = C + (int64_t)lr * p.ldc;
 #pragma unroll
-            for (int j = 0; j < 2 * NJ; ++j)
+            for (int j = 0; j < 2 * NJ; ++j) {
+                const int n = n0 + wn + j * 8 + 2 * tig;
+                if (n >= p.N) continue;
+                float v[2] = {acc[i][j][half * 2], acc[i][j][half * 2 + 1]};
+                if (SWIGLU) {
 #pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const int n = n0 + wn + j * 8 + 2 * tig + e;
-                    if (n >= p.N) continue;
-                    float v = acc[i][j][half * 2 + e];
-                    if (SWIGLU) v = silu_f(v) * acu[i][j][half * 2 + e];   // the activation on the 32-bit sums
-                    else v = plain_epilogue<EPI, __nv_bfloat16>(p, v, lr, g, n);
-                    crow[n] = __float2bfloat16_rn(v);
+                    for (int e = 0; e < 2; ++e) v[e] = silu_f(v[e]) * acu[i][j][half * 2 + e];   // the activation on the 32-bit sums
+                } else if constexpr (EPI == GG_SIGMOID_GATE) {
+                    if (!p.pairs) {
+#pragma unroll
+                        for (int e = 0; e < 2; ++e)
+                            if (n + e < p.N) v[e] = plain_epilogue<EPI, __nv_bfloat16>(p, v[e], lr, g, n + e);
+                    } else {
+                        const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gate_z[i][half][j]));
+                        v[0] /= 1.f + expf(-z.x), v[1] /= 1.f + expf(-z.y);
+                    }
+                } else {
+#pragma unroll
+                    for (int e = 0; e < 2; ++e)
+                        if (n + e < p.N) v[e] = plain_epilogue<EPI, __nv_bfloat16>(p, v[e], lr, g, n + e);
                 }
+                if (p.pairs) {
+                    *reinterpret_cast<__nv_bfloat162*>(crow + n) = __floats2bfloat162_rn(v[0], v[1]);
+                } else {
+                    crow[n] = __float2bfloat16_rn(v[0]);
+                    if (n + 1 < p.N) crow[n + 1] = __float2bfloat16_rn(v[1]);
+                }
+            }
         }
 }
 
@@ -364,6 +399,7 @@ IMP_API int imp_grouped_gemm_ex(void* C, int64_t ldc, int64_t c_group_cols, cons
              aligned(A) && aligned(W) && aligned(W2))
                 ? 1
                 : 0;
+    p.pairs = N % 2 == 0 && ldc % 2 == 0 && c_group_cols % 2 == 0 && (uintptr_t)C % 4 == 0 && (!gate || (gate_ld % 2 == 0 && (uintptr_t)gate % 4 == 0)) ? 1 : 0;
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t e = cudaSuccess;
     // few rows a group (a decode step's experts, its per-head products): 16-row tiles
