@@ -112,7 +112,7 @@ typedef struct {
 typedef struct {
     void* user;
     const char* (*tensor_specs)(void* user, const char* params_json);
-    const char* (*cache_spec)(void* user, const char* params_json);       /* mixers */
+    const char* (*cache_spec)(void* user, const char* params_json);       /* mixers; embeddings that own state */
     const char* (*part_slots)(void* user, const char* params_json);       /* blocks */
     /* tensors: this part's weights on the device, by local name; parts: a block's built parts by slot */
     void* (*create)(void* user, const char* params_json, int n_tensors, const char* const* tensor_names,
