@@ -20,7 +20,8 @@ from ..capi import CacheError, OutOfPages  # noqa: F401  (re-exported)
 @dataclass(frozen=True)
 class PagedKVSpec:
     """Keys and values per token: [kv_heads, head_dim] each.  window == 0 keeps every token;
-    window == W keeps what a query at position p may still see: positions > p - W."""
+    window == W keeps what a query at position p may still see: positions > p - W; window == -C keeps
+    the chunk of C positions that p is in, chunks counted from position 0."""
 
     num_kv_heads: int
     head_dim: int
@@ -82,7 +83,9 @@ class _Group:
 
     def first_live_page(self, length: int) -> int:
         w = self._j().get("window", 0)
-        return 0 if w <= 0 else max(0, length - w + 1) // self._mgr.page_size
+        if w < 0:
+            return (length - length % -w) // self._mgr.page_size
+        return 0 if w == 0 else max(0, length - w + 1) // self._mgr.page_size
 
 
 @dataclass

@@ -251,3 +251,26 @@ class NomanexConfig(ModelConfig):
         while self.raw["layers"][i].get("weights_of") is not None:
             i = int(self.raw["layers"][i]["weights_of"])
         return i
+
+
+class RibovikConfig(ModelConfig):
+    """Ribovik (`"architecture": "Ribovik"`): `vocab`, `width`, `norm.eps`, and a list `layers`, each entry with `type`
+    ("attention"), the mixer's sizes and constants under `mixer` (`heads`, `kv_heads`, `dim`, `vdim`, `scale`, `mask.size`: the
+    chunk, `rot`: `{"base", "dims", "scaling": {"factor", "original", "fast", "slow"} | null}`) and `mlp` (`{"kind": "dense", "ff"}`,
+    `{"kind": "moe", "expert": {"ff", "limit"}, "router": {"experts", "identity", "top"}, "shared": {"ff", "limit"} | null}` or
+    null)."""
+
+    KNOWN_KEYS = ("architecture", "vocab", "width", "norm", "layers", "torch_dtype", "dtype", "eos_token_id", "bos_token_id",
+                  "max_positions")
+
+    @property
+    def vocab_size(self) -> int:
+        return int(self.raw["vocab"])
+
+    @property
+    def hidden_size(self) -> int:
+        return int(self.raw["width"])
+
+    @property
+    def num_hidden_layers(self) -> int:
+        return len(self.raw["layers"])

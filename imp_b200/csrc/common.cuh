@@ -176,11 +176,14 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
 //   0  silu(g) * u        1  gelu(g) * u, tanh form
 //   2  both clipped: g <- min(g, limit), u <- min(max(u, -limit), limit);  g * sigmoid(1.702 g) * (u + 1)
 //   3  max(v, 0)^2 (products without a gate)
+// `bias` (gated products; null: none): a number per row of the stacked gate and up matrix, in that matrix's order, added to the
+// 32-bit sums before the activation.
 enum : int { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_CLIPPED = 2, ACT_RELU2 = 3 };
 struct GateAct {
     int kind;
     float limit;
-    __host__ __device__ GateAct(int k = 0, float l = 0.f) : kind(k), limit(l) {}
+    const float* bias;
+    __host__ __device__ GateAct(int k = 0, float l = 0.f, const float* b = nullptr) : kind(k), limit(l), bias(b) {}
 };
 __device__ __forceinline__ float gated_f(float g, float u, const GateAct& a) {
     if (a.kind == ACT_SILU) return g / (1.f + expf(-g)) * u;

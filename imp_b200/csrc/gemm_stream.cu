@@ -177,6 +177,10 @@ __global__ void __launch_bounds__(GS_WARPS * 32 * RG) gemm_stream_kernel(TO* __r
                 }
                 const int col = (c_tile * RG + rg) * 8 + (l >> 2);
                 const int tok = 8 * nt + 2 * (l & 3) + c;
+                if (gate_act.bias && n0 + (l >> 2) + 8 < N) {
+                    gate += gate_act.bias[n0 + (l >> 2)];
+                    up += gate_act.bias[n0 + (l >> 2) + 8];
+                }
                 if (n0 + (l >> 2) + 8 < N && tok < M)
                     C[(int64_t)tok * ldc + col] = from_float<TO>(gated_f(gate, up, gate_act));
             }
@@ -289,9 +293,9 @@ IMP_API int imp_gemm_bf16_stream(void* C, int64_t ldc, int out_dtype, const void
 // C[M, N/2] = silu(gate) * up where W[N, K] holds gate and up rows interleaved in blocks of 8
 // (rows 16j..16j+7 = gate rows 8j..8j+7, rows 16j+8..16j+15 = up rows 8j..8j+7); bfloat16 output.
 // imp_gemm_bf16_stream_gated: the same with the gate's activation chosen (0 silu, 1 the tanh form of gelu, 2 clipped to
-// `limit`, see GateAct).
+// `limit`, see GateAct) and optionally a bias per row of W in front of it.
 IMP_API int imp_gemm_bf16_stream_gated(void* C, int64_t ldc, const void* A, int64_t lda, const void* W, int64_t ldw,
-                                       int M, int N, int K, int act, float limit, void* stream) {
+                                       int M, int N, int K, int act, float limit, const float* bias, void* stream) {
     if (M == 0 || N == 0) return 0;
     IMP_CHECK_ARG(act >= ACT_SILU && act <= ACT_CLIPPED, "imp_gemm_bf16_stream_gated: unknown activation %d", act);
     IMP_CHECK_ARG(C && A && W && M > 0 && N > 0 && K > 0, "imp_gemm_bf16_stream_swiglu: bad argument");
@@ -300,10 +304,10 @@ IMP_API int imp_gemm_bf16_stream_gated(void* C, int64_t ldc, const void* A, int6
     IMP_CHECK_ARG(ldc >= N / 2 && lda >= K && ldw >= K, "imp_gemm_bf16_stream_swiglu: leading dimension too small");
     if (K % 8 || lda % 8 || ldw % 8 || (uintptr_t)A % 16 || (uintptr_t)W % 16) return IMP_ERR_UNSUPPORTED;
     return launch_stream<__nv_bfloat16, true>((__nv_bfloat16*)C, ldc, (const __nv_bfloat16*)A, lda,
-                                              (const __nv_bfloat16*)W, ldw, M, N, K, (cudaStream_t)stream, GateAct(act, limit));
+                                              (const __nv_bfloat16*)W, ldw, M, N, K, (cudaStream_t)stream, GateAct(act, limit, bias));
 }
 
 IMP_API int imp_gemm_bf16_stream_swiglu(void* C, int64_t ldc, const void* A, int64_t lda, const void* W, int64_t ldw,
                                         int M, int N, int K, void* stream) {
-    return imp_gemm_bf16_stream_gated(C, ldc, A, lda, W, ldw, M, N, K, 0, 0.f, stream);
+    return imp_gemm_bf16_stream_gated(C, ldc, A, lda, W, ldw, M, N, K, 0, 0.f, nullptr, stream);
 }

@@ -39,17 +39,33 @@ constexpr int TC_TMEM_COLS = 256;
 enum TcEpilogue : int { TC_OUT_BF16 = 0, TC_OUT_F32 = 1, TC_OUT_SWIGLU_BF16 = 2, TC_OUT_QKV_ROPE = 3, TC_OUT_GEGLU_BF16 = 4,
                         TC_OUT_CLIPGLU_BF16 = 5, TC_OUT_RELU2_BF16 = 6 };
 // The kernels' own epilogue and activation of an entry point's epilogue.
-static GateAct split_epilogue(int* epilogue, float limit) {
+static GateAct split_epilogue(int* epilogue, float limit, const float* bias = nullptr) {
     switch (*epilogue) {
-        case TC_OUT_GEGLU_BF16: *epilogue = TC_OUT_SWIGLU_BF16; return GateAct(ACT_GELU_TANH);
-        case TC_OUT_CLIPGLU_BF16: *epilogue = TC_OUT_SWIGLU_BF16; return GateAct(ACT_CLIPPED, limit);
+        case TC_OUT_GEGLU_BF16: *epilogue = TC_OUT_SWIGLU_BF16; return GateAct(ACT_GELU_TANH, 0.f, bias);
+        case TC_OUT_CLIPGLU_BF16: *epilogue = TC_OUT_SWIGLU_BF16; return GateAct(ACT_CLIPPED, limit, bias);
         case TC_OUT_RELU2_BF16: *epilogue = TC_OUT_BF16; return GateAct(ACT_RELU2);
-        default: return GateAct();
+        default: return GateAct(ACT_SILU, 0.f, *epilogue == TC_OUT_SWIGLU_BF16 ? bias : nullptr);
     }
 }
 
-// The activation of a product without a gate, on 32 accumulator columns.
-template <int EPI> __device__ __forceinline__ void plain_act(float (&v)[32], const GateAct& act) {
+// 32 accumulator columns of a gated product, from column col0 of the stacked gate and up matrix on (N columns, a multiple of
+// 16), plus the columns' bias.
+__device__ __forceinline__ void gate_bias32(float (&v)[32], const GateAct& act, int col0, int N) {
+    if (!act.bias) return;
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+        if (col0 + 16 * j < N) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float4 b = *reinterpret_cast<const float4*>(act.bias + col0 + 16 * j + 4 * i);
+                v[16 * j + 4 * i] += b.x, v[16 * j + 4 * i + 1] += b.y, v[16 * j + 4 * i + 2] += b.z, v[16 * j + 4 * i + 3] += b.w;
+            }
+        }
+}
+
+// What happens to 32 accumulator columns before they are stored: the activation of a product without a gate, the bias of a gated one.
+template <int EPI> __device__ __forceinline__ void plain_act(float (&v)[32], const GateAct& act, int col0, int N) {
+    if (EPI == TC_OUT_SWIGLU_BF16) gate_bias32(v, act, col0, N);
     if (EPI == TC_OUT_BF16 && act.kind == ACT_RELU2) {
 #pragma unroll
         for (int i = 0; i < 32; ++i) v[i] = relu2_f(v[i]);
@@ -195,7 +211,7 @@ __global__ void __launch_bounds__(128, 1) gemm_tc_kernel(const __grid_constant__
         for (int c = 0; c < TC_BN / 32; ++c) {
             float v[32];
             tc_ld32(lane_base + (uint32_t)(c * 32), v);
-            plain_act<EPI>(v, gate_act);
+            plain_act<EPI>(v, gate_act, n0 + c * 32, N);
             tc_store32<EPI>(Cv, ldc, row, n0 + c * 32, M, N, v, gate_act);
         }
     }
@@ -323,7 +339,7 @@ __global__ void __launch_bounds__(TCP_THREADS, 1) gemm_tc_persistent_kernel(cons
             for (int c = 0; c < TC_BN / 32; ++c) {
                 float v[32];
                 tc_ld32(taddr + (uint32_t)(c * 32), v);
-                plain_act<EPI>(v, gate_act);
+                plain_act<EPI>(v, gate_act, n0 + c * 32, N);
                 tc_store32<EPI>(Cv, ldc, row, n0 + c * 32, M, N, v, gate_act);
             }
             tc_fence_before_sync();
@@ -758,7 +774,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TCP_THREADS, 1)
                         for (int cc = 0; cc < 2; ++cc) {
                             float v[32];
                             tc_ld32(taddr + (uint32_t)((2 * j + cc) * 32), v);
-                            plain_act<EPI>(v, gate_act);
+                            plain_act<EPI>(v, gate_act, n0 + (2 * j + cc) * 32, N);
 #pragma unroll
                             for (int i = 0; i < 4; ++i) q[4 * cc + i] = tc2_pack8(v + 8 * i);
                         }
@@ -768,6 +784,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TCP_THREADS, 1)
                         for (int cc = 0; cc < 4; ++cc) {
                             float v[32], o[16];
                             tc_ld32(taddr + (uint32_t)((4 * j + cc) * 32), v);
+                            gate_bias32(v, gate_act, n0 + (4 * j + cc) * 32, N);
 #pragma unroll
                             for (int h = 0; h < 2; ++h)
 #pragma unroll
@@ -794,7 +811,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TCP_THREADS, 1)
                 for (int c = 0; c < TC2_BN / 32; ++c) {
                     float v[32];
                     tc_ld32(taddr + (uint32_t)(c * 32), v);
-                    plain_act<EPI>(v, gate_act);
+                    plain_act<EPI>(v, gate_act, n0 + c * 32, N);
                     tc_store32<EPI == TC_OUT_QKV_ROPE ? TC_OUT_BF16 : EPI>(Cz, ldc, row, n0 + c * 32, M, N, v, gate_act);
                 }
             }
@@ -975,6 +992,9 @@ __global__ void __launch_bounds__(128, 1) gemm_tc_swap_kernel(const __grid_const
                 __nv_bfloat16* base = reinterpret_cast<__nv_bfloat16*>(Cv);
                 const bool is_gate = (r & 8) == 0;
                 const int ocol = (col >> 4) * 8 + (r & 7);
+                const float bias = gate_act.bias && col < N ? gate_act.bias[col] : 0.f;
+#pragma unroll
+                for (int i = 0; i < 32; ++i) v[i] += bias;
 #pragma unroll
                 for (int i = 0; i < 32; ++i) {
                     const float up = __shfl_xor_sync(0xffffffffu, v[i], 8);   // lane r + 8 holds the matching up row
@@ -992,7 +1012,7 @@ __global__ void __launch_bounds__(128, 1) gemm_tc_swap_kernel(const __grid_const
                     }
                 } else {
                     __nv_bfloat16* base = reinterpret_cast<__nv_bfloat16*>(Cv);
-                    plain_act<EPI>(v, gate_act);
+                    plain_act<EPI>(v, gate_act, 0, 0);
 #pragma unroll
                     for (int i = 0; i < 32; ++i) {
                         const int tok = c * 32 + i;
@@ -1151,12 +1171,14 @@ static int launch_tc(void* C, int64_t ldc, const CUtensorMap& ma, const CUtensor
 // gate and up rows of W interleaved in runs of 8; 4 = the same with the tanh form of gelu on the gate.
 // Returns IMP_ERR_UNSUPPORTED when the operands do not meet the alignment rules of the tensor copies
 // (bases on 16-byte boundaries, row strides multiples of 8 elements): the caller uses another kernel.
+// `bias` (gated epilogues, or null): float32 [N] in the order of W's rows, added before the activation.
 // 5 = the gated form with both values clipped to `limit` (ACT_CLIPPED), 6 = bfloat16 C[M,N] = max(A W^T, 0)^2.
-IMP_API int imp_gemm_bf16_tc_act(void* C, int64_t ldc, int epilogue, float limit, const void* A, int64_t lda, const void* W, int64_t ldw,
+IMP_API int imp_gemm_bf16_tc_act(void* C, int64_t ldc, int epilogue, float limit, const float* bias, const void* A, int64_t lda, const void* W, int64_t ldw,
                                  int M, int N, int K, int* status, void* stream) {
     if (M == 0 || N == 0) return 0;
     IMP_CHECK_ARG(C && A && W && M > 0 && N > 0 && K > 0, "imp_gemm_bf16_tc: bad argument");
-    const GateAct gate_act = split_epilogue(&epilogue, limit);
+    const GateAct gate_act = split_epilogue(&epilogue, limit, bias);
+    IMP_CHECK_ARG(!bias || (epilogue == TC_OUT_SWIGLU_BF16 && (uintptr_t)bias % 16 == 0), "imp_gemm_bf16_tc: a bias goes with the gated epilogues and starts on 16 bytes");
     IMP_CHECK_ARG(epilogue >= 0 && epilogue <= 2, "imp_gemm_bf16_tc: unknown epilogue %d", epilogue);
     IMP_CHECK_ARG(lda >= K && ldw >= K && ldc >= (epilogue == 2 ? N / 2 : N), "imp_gemm_bf16_tc: leading dimension too small");
     if (epilogue == 2) IMP_CHECK_ARG(N % 16 == 0, "imp_gemm_bf16_tc: %d interleaved rows are not a multiple of 16", N);
@@ -1175,7 +1197,7 @@ IMP_API int imp_gemm_bf16_tc_act(void* C, int64_t ldc, int epilogue, float limit
 IMP_API int imp_gemm_bf16_tc(void* C, int64_t ldc, int epilogue, const void* A, int64_t lda, const void* W, int64_t ldw, int M, int N,
                              int K, int* status, void* stream) {
     IMP_CHECK_ARG(epilogue != TC_OUT_CLIPGLU_BF16, "imp_gemm_bf16_tc: the clipped gate needs a limit (imp_gemm_bf16_tc_act)");
-    return imp_gemm_bf16_tc_act(C, ldc, epilogue, 0.f, A, lda, W, ldw, M, N, K, status, stream);
+    return imp_gemm_bf16_tc_act(C, ldc, epilogue, 0.f, nullptr, A, lda, W, ldw, M, N, K, status, stream);
 }
 
 // ---- many rows, few tiles: the K range in parts ------------------------------------------------------
@@ -1300,13 +1322,14 @@ static int launch_tcs(void* C, int64_t ldc, int64_t split_stride, const CUtensor
 
 // C = A[M,K] * W[N,K]^T for 1 <= M <= 128 with the weights on the M side of the MMA.
 // epilogue as for imp_gemm_bf16_tc.  `scratch` must hold imp_gemm_bf16_tc_swap_scratch_floats() floats.
-static int gemm_bf16_tc_swap_impl(void* C, int64_t ldc, int epilogue, float limit, const void* A, int64_t lda, const void* W, int64_t ldw,
+static int gemm_bf16_tc_swap_impl(void* C, int64_t ldc, int epilogue, float limit, const float* bias, const void* A, int64_t lda, const void* W, int64_t ldw,
                                   int M, int N, int K, float* scratch, int* status, void* stream, bool partials_only) {
     if (M == 0 || N == 0) return 0;
     IMP_CHECK_ARG((C || partials_only) && A && W && M > 0 && N > 0 && K > 0, "imp_gemm_bf16_tc_swap: bad argument");
     IMP_CHECK_ARG(M <= 128, "imp_gemm_bf16_tc_swap: M %d exceeds 128", M);
     const int splits = tcs_splits(M, N, K, epilogue);
-    const GateAct gate_act = split_epilogue(&epilogue, limit);
+    const GateAct gate_act = split_epilogue(&epilogue, limit, bias);
+    IMP_CHECK_ARG(!bias || epilogue == TC_OUT_SWIGLU_BF16, "imp_gemm_bf16_tc_swap: a bias goes with the gated epilogues");
     IMP_CHECK_ARG(epilogue >= 0 && epilogue <= 2, "imp_gemm_bf16_tc_swap: unknown epilogue %d", epilogue);
     if (epilogue == 2) IMP_CHECK_ARG(N % 16 == 0, "imp_gemm_bf16_tc_swap: %d interleaved rows are not a multiple of 16", N);
     IMP_CHECK_ARG(lda >= K && ldw >= K && ldc >= (epilogue == 2 ? N / 2 : N), "imp_gemm_bf16_tc_swap: leading dimension too small");
@@ -1381,11 +1404,11 @@ IMP_API int imp_gemm_tc_test_hooks(unsigned wait_limit, int skip_kb) {
 IMP_API int imp_gemm_bf16_tc_swap(void* C, int64_t ldc, int epilogue, const void* A, int64_t lda, const void* W, int64_t ldw,
                                   int M, int N, int K, float* scratch, int* status, void* stream) {
     IMP_CHECK_ARG(epilogue != TC_OUT_CLIPGLU_BF16, "imp_gemm_bf16_tc_swap: the clipped gate needs a limit (imp_gemm_bf16_tc_swap_act)");
-    return gemm_bf16_tc_swap_impl(C, ldc, epilogue, 0.f, A, lda, W, ldw, M, N, K, scratch, status, stream, false);
+    return gemm_bf16_tc_swap_impl(C, ldc, epilogue, 0.f, nullptr, A, lda, W, ldw, M, N, K, scratch, status, stream, false);
 }
-IMP_API int imp_gemm_bf16_tc_swap_act(void* C, int64_t ldc, int epilogue, float limit, const void* A, int64_t lda, const void* W, int64_t ldw,
+IMP_API int imp_gemm_bf16_tc_swap_act(void* C, int64_t ldc, int epilogue, float limit, const float* bias, const void* A, int64_t lda, const void* W, int64_t ldw,
                                       int M, int N, int K, float* scratch, int* status, void* stream) {
-    return gemm_bf16_tc_swap_impl(C, ldc, epilogue, limit, A, lda, W, ldw, M, N, K, scratch, status, stream, false);
+    return gemm_bf16_tc_swap_impl(C, ldc, epilogue, limit, bias, A, lda, W, ldw, M, N, K, scratch, status, stream, false);
 }
 
 // How many partial results imp_gemm_bf16_tc_swap_partials leaves for this shape (1: it does not split, call the
@@ -1399,7 +1422,7 @@ IMP_API int imp_gemm_bf16_tc_swap_partials(float* scratch, const void* A, int64_
                                            int N, int K, int* status, void* stream) {
     IMP_CHECK_ARG(scratch, "imp_gemm_bf16_tc_swap_partials: no scratch memory");
     if (tcs_splits(M, N, K, TC_OUT_F32) < 2) return IMP_ERR_UNSUPPORTED;
-    return gemm_bf16_tc_swap_impl(nullptr, N, TC_OUT_F32, 0.f, A, lda, W, ldw, M, N, K, scratch, status, stream, true);
+    return gemm_bf16_tc_swap_impl(nullptr, N, TC_OUT_F32, 0.f, nullptr, A, lda, W, ldw, M, N, K, scratch, status, stream, true);
 }
 
 // C[M, N] (bfloat16 or float32, by `epilogue`) = the sum of the partial results, in split order.

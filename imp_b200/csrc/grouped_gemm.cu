@@ -7,7 +7,7 @@
 //              launch does not depend on the routing): routed experts.  Row r of the list reads A row a_rows[r]
 //              (null: r) and writes C row r.  The grid covers the most tiles any routing can make
 //              (rows / BM + groups); a CTA finds its group by walking seg, and leaves if there is no tile for it.
-// Epilogues on the 32-bit sums: none; silu(A Wg^T) * (A Wu^T) with two weight matrices per group; max(A W^T, 0)^2; or A W^T
+// Epilogues on the 32-bit sums: none; a gated activation of A Wg^T and A Wu^T (GateAct) with two weight matrices per group; max(A W^T, 0)^2; or A W^T
 // times sigmoid of a gate that stands beside C (row r, column c_group_cols * g + n of `gate`).
 //
 // bfloat16: mma.sync m16n8k16 with 32-bit accumulation, 64 x 64 x 64 tiles through a cp.async ring of three or four stages,
@@ -39,6 +39,7 @@ struct GroupedArgs {
     const void* gate;   // GG_SIGMOID_GATE: rows gate_ld apart, in the activations' type
     int64_t gate_ld;
     int pairs; // bfloat16 outputs (and gates) may move two at a time: N even, rows and groups of C (and the gate) on 4 bytes
+    GateAct act;   // GG_SWIGLU: silu(g) * u unless said otherwise
     int il;    // the gated epilogue's two matrices are one, gate and up rows alternating in runs of 8 (W2 unused)
 };
 
@@ -69,8 +70,6 @@ __device__ __forceinline__ bool find_tile(const GroupedArgs& p, int& g, int& row
     }
     return false;
 }
-
-__device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 
 // The epilogue of a product with one weight matrix: row lr of C, column n of the group.
 template <int EPI, typename T>
@@ -252,7 +251,7 @@ __global__ void __launch_bounds__(128) grouped_gemm_bf16_kernel(const GroupedArg
                 float v[2] = {acc[i][j][half * 2], acc[i][j][half * 2 + 1]};
                 if (SWIGLU) {
 #pragma unroll
-                    for (int e = 0; e < 2; ++e) v[e] = silu_f(v[e]) * acu[i][j][half * 2 + e];   // the activation on the 32-bit sums
+                    for (int e = 0; e < 2; ++e) v[e] = gated_f(v[e], acu[i][j][half * 2 + e], p.act);   // the activation on the 32-bit sums
                 } else if constexpr (EPI == GG_SIGMOID_GATE) {
                     if (!p.pairs) {
 #pragma unroll
@@ -366,7 +365,7 @@ __global__ void __launch_bounds__(256) grouped_gemm_f32_kernel(const GroupedArgs
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int gn = n0 + tn + j;
-            if (gn < p.N) C[(int64_t)lr * p.ldc + gn] = SWIGLU ? silu_f(acc[i][j]) * acu[i][j] : plain_epilogue<EPI, float>(p, acc[i][j], lr, g, gn);
+            if (gn < p.N) C[(int64_t)lr * p.ldc + gn] = SWIGLU ? gated_f(acc[i][j], acu[i][j], p.act) : plain_epilogue<EPI, float>(p, acc[i][j], lr, g, gn);
         }
     }
 }
@@ -376,10 +375,12 @@ __global__ void __launch_bounds__(256) grouped_gemm_f32_kernel(const GroupedArgs
 // A: activations (dtype), rows lda apart.  W (and W2 with swiglu == 1): [G][N, K], groups w_group_stride elements apart,
 // rows ldw apart; swiglu == 2: W is [G][2N, K] with gate and up rows alternating in runs of 8 (W2 unused, N a multiple
 // of 8).  C: rows ldc apart.  seg == null: uniform groups of M rows each; else the list has M rows in all.
+// `act`, `limit`: the gated epilogue's activation (GateAct, kinds 0 to 2).
 // `epi` (0 where swiglu is set): 0 none, 2 max(., 0)^2, 3 times sigmoid(gate), gate's rows gate_ld apart and its columns C's own.
 IMP_API int imp_grouped_gemm_ex(void* C, int64_t ldc, int64_t c_group_cols, const void* A, int64_t lda, int64_t a_group_cols,
                                 const int* a_rows, const void* W, const void* W2, int64_t w_group_stride, int64_t ldw, const int* seg,
-                                int M, int N, int K, int G, int swiglu, int epi, const void* gate, int64_t gate_ld, int dtype, void* stream) {
+                                int M, int N, int K, int G, int swiglu, int epi, const void* gate, int64_t gate_ld, int act, float limit, int dtype,
+                                void* stream) {
     if (M == 0 || N == 0 || G == 0) return 0;
     IMP_CHECK_ARG(C && A && W && M > 0 && N > 0 && K > 0 && G > 0, "imp_grouped_gemm: bad argument");
     IMP_CHECK_ARG(swiglu != 1 || W2, "imp_grouped_gemm: the gated epilogue needs a second weight");
@@ -392,6 +393,8 @@ IMP_API int imp_grouped_gemm_ex(void* C, int64_t ldc, int64_t c_group_cols, cons
     p.C = C, p.ldc = ldc, p.c_group_cols = c_group_cols, p.seg = seg;
     p.M = M, p.N = N, p.K = K, p.G = G;
     p.gate = gate, p.gate_ld = gate_ld;
+    IMP_CHECK_ARG(act >= ACT_SILU && act <= ACT_CLIPPED, "imp_grouped_gemm: unknown activation %d", act);
+    p.act = GateAct(act, limit);
     p.il = swiglu == 2 ? 1 : 0;
     const int el = dtype == IMP_F32 ? 4 : 2, per16 = 16 / el;
     auto aligned = [&](const void* q) { return q == nullptr || (uintptr_t)q % 16 == 0; };
@@ -439,7 +442,7 @@ IMP_API int imp_grouped_gemm(void* C, int64_t ldc, int64_t c_group_cols, const v
                              const int* a_rows, const void* W, const void* W2, int64_t w_group_stride, int64_t ldw, const int* seg,
                              int M, int N, int K, int G, int swiglu, int dtype, void* stream) {
     return imp_grouped_gemm_ex(C, ldc, c_group_cols, A, lda, a_group_cols, a_rows, W, W2, w_group_stride, ldw, seg, M, N, K, G, swiglu, 0, nullptr, 0,
-                               dtype, stream);
+                               ACT_SILU, 0.f, dtype, stream);
 }
 
 // dst[g][c][r] = src[g][r][c]: per-group transposes of small weight matrices, at load time.

@@ -46,8 +46,7 @@ void PagedGroup::ensure_width(int n_logical, int num_slots) {
 }
 
 int PagedGroup::first_live_page(int length) const {
-    if (spec.window <= 0) return 0;
-    return std::max(0, length - spec.window + 1) / page_size;
+    return first_visible(length, spec.window) / page_size;   // of the next query, at position `length`
 }
 
 int PagedGroup::pages_needed_n(int entries, int cur_len, int new_len) const {
@@ -186,7 +185,7 @@ int CacheManager::commit(int64_t rid, int new_len) {
     l.length = new_len;
     int freed = 0;
     for (auto& g : paged_) {
-        if (g.spec.window <= 0) continue;
+        if (g.spec.window == 0) continue;
         int32_t* row = g.row(l.slot);
         const int hi = std::min(g.first_live_page(new_len), g.n_entries[(size_t)l.slot]);
         const int lo = g.first_live_page(old_len);

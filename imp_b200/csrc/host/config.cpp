@@ -1374,6 +1374,219 @@ ModelPlan nomanex_plan(const NomanexConfig& cfg) {
     return plan;
 }
 
+// ------------------------------------------------------------------------------------ Ribovik
+RibovikConfig RibovikConfig::from_json(const Json& d, const std::string& where) {
+    RibovikConfig c;
+    c.architecture = d.get_string("architecture", "Ribovik");
+    c.vocab_size = positive("vocab", require_int(d, "vocab", where), where);
+    c.hidden_size = positive("width", require_int(d, "width", where), where);
+    c.max_position_embeddings = positive("max_positions", d.get_int("max_positions", 1 << 20), where);
+    c.torch_dtype = d.get_string("torch_dtype", d.get_string("dtype", "bfloat16"));
+    if (c.torch_dtype != "bfloat16" && c.torch_dtype != "float32")
+        bad(where + ": torch_dtype '" + c.torch_dtype + "' is not supported (bfloat16 or float32)");
+    if (const Json* eos = d.find("eos_token_id")) {
+        if (eos->is_array()) {
+            for (const auto& e : eos->items())
+                if (e.is_int()) c.eos_token_ids.push_back((int)e.as_int());
+        } else if (eos->is_int()) {
+            c.eos_token_ids.push_back((int)eos->as_int());
+        }
+    }
+    c.bos_token_id = d.get_int("bos_token_id", -1);
+    c.raw = d;
+    c.norm_eps = require_float(require_object(d, "norm", where), "eps", where + ": norm");
+    if (!(c.norm_eps > 0)) bad(where + ": norm.eps must be positive");
+    auto optional_object = [&](const Json& in, const char* key, const std::string& w) -> const Json* {
+        const Json* v = in.find(key);
+        if (!v || v->is_null()) return nullptr;
+        if (!v->is_object()) bad(w + ": '" + key + "' must be an object or null");
+        return v;
+    };
+    auto limit = [&](const Json& in, const std::string& w) {
+        const double l = require_float(in, "limit", w);
+        if (!(l > 0)) bad(w + ": limit must be positive");
+        return l;
+    };
+    const Json& layers = require(d, "layers", where);
+    if (!layers.is_array() || layers.size() == 0) bad(where + ": 'layers' must be a non-empty list");
+    for (const Json& lj : layers.items()) {
+        const std::string lw = where + ": layers[" + std::to_string(c.layers.size()) + "]";
+        if (!lj.is_object()) bad(lw + " must be an object");
+        Layer l;
+        l.type = lj.get_string("type", "");
+        if (l.type != "attention") bad(lw + ": unknown layer type '" + l.type + "' (known: attention)");
+        const Json& m = require_object(lj, "mixer", lw);
+        const std::string mw = lw + ".mixer";
+        l.heads = positive("heads", require_int(m, "heads", mw), mw);
+        l.kv_heads = positive("kv_heads", m.get_int("kv_heads", l.heads), mw);
+        if (l.heads % l.kv_heads) bad(mw + ": " + std::to_string(l.heads) + " heads are not a multiple of " + std::to_string(l.kv_heads) + " kv_heads");
+        l.dim = positive("dim", require_int(m, "dim", mw), mw);
+        l.vdim = positive("vdim", m.get_int("vdim", l.dim), mw);
+        l.scale = m.find("scale") ? require_float(m, "scale", mw) : 1.0 / std::sqrt((double)l.dim);
+        if (!(l.scale > 0)) bad(mw + ": scale must be positive");
+        if (const Json* mask = optional_object(m, "mask", mw)) l.chunk = positive("size", require_int(*mask, "size", mw + ".mask"), mw + ".mask");
+        if (const Json* rot = optional_object(m, "rot", mw)) {
+            const std::string rw = mw + ".rot";
+            l.rot_base = require_float(*rot, "base", rw);
+            l.rot_dims = positive("dims", rot->get_int("dims", l.dim), rw);
+            if (!(l.rot_base > 0)) bad(rw + ": base must be positive");
+            if (l.rot_dims % 2 || l.rot_dims > l.dim) bad(rw + ": dims " + std::to_string(l.rot_dims) + " must be even and at most dim " + std::to_string(l.dim));
+            if (const Json* sc = optional_object(*rot, "scaling", rw)) {
+                const std::string sw = rw + ".scaling";
+                l.rot_scaled = true;
+                l.rot_factor = require_float(*sc, "factor", sw);
+                l.rot_original = require_float(*sc, "original", sw);
+                l.rot_fast = require_float(*sc, "fast", sw);
+                l.rot_slow = require_float(*sc, "slow", sw);
+                if (!(l.rot_factor > 0) || !(l.rot_original > 0) || !(l.rot_fast > 0) || !(l.rot_slow > 0) || l.rot_base == 1.0)
+                    bad(sw + ": factor, original, fast and slow must be positive, and the base not 1");
+            }
+        }
+        if (const Json* f = optional_object(lj, "mlp", lw)) {
+            const std::string fw = lw + ".mlp";
+            l.mlp = f->get_string("kind", "");
+            if (l.mlp == "dense") {
+                l.ff = positive("ff", require_int(*f, "ff", fw), fw);
+            } else if (l.mlp == "moe") {
+                const Json& e = require_object(*f, "expert", fw);
+                l.expert_ff = positive("ff", require_int(e, "ff", fw + ".expert"), fw + ".expert");
+                l.expert_limit = limit(e, fw + ".expert");
+                const Json& r = require_object(*f, "router", fw);
+                const std::string rw = fw + ".router";
+                l.experts = positive("experts", require_int(r, "experts", rw), rw);
+                l.identity = r.get_int("identity", 0);
+                if (l.identity < 0) bad(rw + ": identity must not be negative");
+                l.top = positive("top", require_int(r, "top", rw), rw);
+                if (l.top > l.experts + l.identity) bad(rw + ": top " + std::to_string(l.top) + " exceeds the " + std::to_string(l.experts + l.identity) + " router outputs");
+                if (const Json* sh = optional_object(*f, "shared", fw)) {
+                    l.shared_ff = positive("ff", require_int(*sh, "ff", fw + ".shared"), fw + ".shared");
+                    l.shared_limit = limit(*sh, fw + ".shared");
+                }
+            } else {
+                bad(fw + ": unknown kind '" + l.mlp + "' (known: dense, moe)");
+            }
+        }
+        c.layers.push_back(l);
+    }
+    c.num_hidden_layers = (int64_t)c.layers.size();
+    return c;
+}
+
+Json RibovikConfig::to_json() const {
+    Json j = raw.is_object() ? raw : Json::object();
+    j["architecture"] = architecture;
+    j["vocab"] = vocab_size;
+    j["width"] = hidden_size;
+    j["torch_dtype"] = torch_dtype;
+    j.erase("dtype");
+    return j;
+}
+
+// Layer i's tensors are 'l<i>.norm1', 'l<i>.mix.*' and, with a feed-forward, 'l<i>.norm2' and 'l<i>.mlp.*'.
+ModelPlan ribovik_plan(const RibovikConfig& cfg) {
+    const int64_t d = cfg.hidden_size;
+    ModelPlan plan;
+    plan.architecture = cfg.architecture;
+    plan.hidden_size = d;
+    plan.vocab_size = cfg.vocab_size;
+    plan.max_positions = cfg.max_position_embeddings;
+    auto norm = [&](const std::string& tensor) {
+        PartSpec n;
+        n.kind = "rmsnorm";
+        n.params["size"] = d;
+        n.params["eps"] = cfg.norm_eps;
+        n.tensors = {{"weight", tensor}};
+        return n;
+    };
+    for (size_t i = 0; i < cfg.layers.size(); ++i) {
+        const RibovikConfig::Layer& l = cfg.layers[i];
+        const std::string p = "l" + std::to_string(i) + ".", a = p + "mix.", f = p + "mlp.";
+        PartSpec mixer;
+        mixer.kind = "gated_head_attention";
+        mixer.params["hidden_size"] = d;
+        mixer.params["num_heads"] = l.heads;
+        mixer.params["num_kv_heads"] = l.kv_heads;
+        mixer.params["head_dim"] = l.dim;
+        mixer.params["value_dim"] = l.vdim;
+        mixer.params["scale"] = l.scale;
+        mixer.params["norm_eps"] = cfg.norm_eps;
+        mixer.params["qkv_bias"] = true;
+        mixer.params["qk_norm"] = true;
+        mixer.params["qk_norm_weight"] = false;
+        mixer.params["qk_norm_position"] = "after_rotation";
+        mixer.params["rot_dims"] = l.rot_dims;
+        mixer.params["rot_base"] = l.rot_base;
+        mixer.params["rot_pairing"] = "neighbours";
+        if (l.rot_scaled) {
+            Json sc = Json::object();
+            sc["kind"] = "yarn";
+            sc["factor"] = l.rot_factor;
+            sc["original"] = l.rot_original;
+            sc["fast"] = l.rot_fast;
+            sc["slow"] = l.rot_slow;
+            mixer.params["rot_scaling"] = sc;
+        }
+        mixer.params["chunk"] = l.chunk;
+        mixer.params["sink"] = true;
+        mixer.tensors = {{"q_proj", a + "q"}, {"q_bias", a + "q.b"}, {"k_proj", a + "k"}, {"k_bias", a + "k.b"}, {"v_proj", a + "v"}, {"v_bias", a + "v.b"},
+                         {"o_proj", a + "o"}};
+        LayerSpec layer;
+        layer.block = "output_norm";
+        layer.block_params["has_ffn"] = !l.mlp.empty();
+        layer.parts = {{"mixer", mixer}, {"mixer_post_norm", norm(p + "norm1")}};
+        if (!l.mlp.empty()) {
+            PartSpec ffn;
+            ffn.params["hidden_size"] = d;
+            if (l.mlp == "dense") {
+                ffn.kind = "gated_mlp";
+                ffn.params["intermediate_size"] = l.ff;
+                ffn.params["activation"] = "silu";
+                ffn.params["bias"] = true;
+                ffn.tensors = {{"gate_proj", f + "gate"}, {"gate_bias", f + "gate.b"}, {"up_proj", f + "up"}, {"up_bias", f + "up.b"},
+                               {"down_proj", f + "down"}, {"down_bias", f + "down.b"}};
+            } else {
+                ffn.kind = "routed_experts";
+                ffn.params["num_experts"] = l.experts;
+                ffn.params["num_identity"] = l.identity;
+                ffn.params["top_k"] = l.top;
+                ffn.params["expert_size"] = l.expert_ff;
+                ffn.params["expert"] = "clipped";
+                ffn.params["expert_limit"] = l.expert_limit;
+                ffn.params["router_bias"] = false;
+                ffn.params["scores"] = "softmax_all";
+                ffn.params["choice_bias"] = true;
+                ffn.params["renormalise"] = true;
+                ffn.tensors = {{"router", f + "router"}, {"choice_bias", f + "correction"}};
+                if (l.shared_ff > 0) {
+                    ffn.params["shared_size"] = l.shared_ff;
+                    ffn.params["shared_limit"] = l.shared_limit;
+                    ffn.params["shared_gate"] = false;
+                    for (const char* n : {"gate", "up", "down"}) ffn.tensors.emplace_back(std::string("shared_") + n, f + "shared." + n);
+                }
+                for (int64_t e = 0; e < l.experts; ++e) {
+                    const std::string n = std::to_string(e), t = f + "e" + n + ".";
+                    for (const char* m : {"gate", "up", "down"}) ffn.tensors.emplace_back(std::string(m) + "_" + n, t + m);
+                }
+            }
+            layer.parts.emplace_back("feed_forward", ffn);
+            layer.parts.emplace_back("ffn_post_norm", norm(p + "norm2"));
+        }
+        plan.layers.push_back(layer);
+    }
+    plan.embedding.kind = "token_embedding";
+    plan.embedding.params["vocab_size"] = cfg.vocab_size;
+    plan.embedding.params["hidden_size"] = d;
+    plan.embedding.params["norm"] = true;
+    plan.embedding.params["norm_eps"] = cfg.norm_eps;
+    plan.embedding.tensors = {{"weight", "embed"}, {"norm", "embed.norm"}};
+    plan.final_norm = norm("final.norm");
+    plan.head.kind = "linear_head";
+    plan.head.params["vocab_size"] = cfg.vocab_size;
+    plan.head.params["hidden_size"] = d;
+    plan.head.tensors = {{"weight", "embed"}};
+    return plan;
+}
+
 // ------------------------------------------------------------------------------------ registry
 namespace {
 std::mutex g_arch_mutex;
@@ -1426,6 +1639,13 @@ void ensure_builtin_archs() {
         };
         nm.plan = [](const Json& d) { return nomanex_plan(NomanexConfig::from_json(d, "config.json")); };
         archs()[nm.name] = nm;
+        Architecture rb;
+        rb.name = "Ribovik";
+        rb.parse_config = [](const Json& d, const std::string& where) -> std::shared_ptr<ModelConfig> {
+            return std::make_shared<RibovikConfig>(RibovikConfig::from_json(d, where));
+        };
+        rb.plan = [](const Json& d) { return ribovik_plan(RibovikConfig::from_json(d, "config.json")); };
+        archs()[rb.name] = rb;
     });
 }
 }  // namespace

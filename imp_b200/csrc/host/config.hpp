@@ -222,6 +222,34 @@ struct NomanexConfig : ModelConfig {
 
 ModelPlan nomanex_plan(const NomanexConfig& cfg);
 
+// Ribovik ("architecture": "Ribovik"): the sublayers read the stream itself and what they give is normalised before it is added,
+// x <- x + rms(mixer(x)) w1, x <- x + rms(ff(x)) w2.  The embedding is normalised, the head is the embedding table.  The mixer is
+// softmax attention with biases on q, k and v, a rotation of neighbouring pairs with the frequencies of YaRN, an RMS norm without
+// a weight on q and k after it, a mask by chunks of positions and a sink; the feed-forward is dense (biases), a mixture of clipped
+// experts (softmax scores, a bias on the choice, renormalised weights, identity experts, a shared expert), or absent.
+// config.json lists the layers one by one; the keys are this family's own.
+struct RibovikConfig : ModelConfig {
+    struct Layer {
+        std::string type;                         // "attention"
+        int64_t heads = 0, kv_heads = 0, dim = 0, vdim = 0;
+        double scale = 0, rot_base = 10000.0;
+        int64_t chunk = 0, rot_dims = 0;          // 0: no chunks / no rotation
+        bool rot_scaled = false;
+        double rot_factor = 1, rot_original = 1, rot_fast = 1, rot_slow = 1;
+        std::string mlp;                          // "" (none) | "dense" | "moe"
+        int64_t ff = 0;                           // dense
+        int64_t experts = 0, identity = 0, top = 0, expert_ff = 0, shared_ff = 0;   // moe; shared_ff 0: none
+        double expert_limit = 0, shared_limit = 0;
+    };
+    std::vector<Layer> layers;
+    double norm_eps = 1e-5;
+
+    static RibovikConfig from_json(const Json& d, const std::string& where);
+    Json to_json() const override;
+};
+
+ModelPlan ribovik_plan(const RibovikConfig& cfg);
+
 // ------------------------------------------------------------------------------------ registry
 struct Architecture {
     std::string name;

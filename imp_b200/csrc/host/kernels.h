@@ -5,6 +5,9 @@
 
 #include <stdint.h>
 
+#include "../branch_terms.h"
+#include "../qkv_prepare.h"
+
 extern "C" {
 
 const char* imp_last_error(void);
@@ -77,16 +80,16 @@ int imp_gemm_bf16_stream(void* C, int64_t ldc, int out_dtype, const void* A, int
 int imp_gemm_bf16_stream_swiglu(void* C, int64_t ldc, const void* A, int64_t lda, const void* W, int64_t ldw, int M, int N,
                                 int K, void* stream);
 int imp_gemm_bf16_stream_gated(void* C, int64_t ldc, const void* A, int64_t lda, const void* W, int64_t ldw, int M, int N,
-                               int K, int act, float limit, void* stream);
+                               int K, int act, float limit, const float* bias, void* stream);
 int imp_gemm_bf16_tc_splits(int M, int N, int K);
 int imp_gemm_bf16_tc_partials(float* scratch, const void* A, int64_t lda, const void* W, int64_t ldw, int M, int N, int K, int* status,
                               void* stream);
 int imp_gemm_bf16_tc(void* C, int64_t ldc, int epilogue, const void* A, int64_t lda, const void* W, int64_t ldw, int M,
                      int N, int K, int* status, void* stream);
-int imp_gemm_bf16_tc_act(void* C, int64_t ldc, int epilogue, float limit, const void* A, int64_t lda, const void* W, int64_t ldw, int M,
-                         int N, int K, int* status, void* stream);
-int imp_gemm_bf16_tc_swap_act(void* C, int64_t ldc, int epilogue, float limit, const void* A, int64_t lda, const void* W, int64_t ldw,
-                              int M, int N, int K, float* scratch, int* status, void* stream);
+int imp_gemm_bf16_tc_act(void* C, int64_t ldc, int epilogue, float limit, const float* bias, const void* A, int64_t lda, const void* W,
+                         int64_t ldw, int M, int N, int K, int* status, void* stream);
+int imp_gemm_bf16_tc_swap_act(void* C, int64_t ldc, int epilogue, float limit, const float* bias, const void* A, int64_t lda, const void* W,
+                              int64_t ldw, int M, int N, int K, float* scratch, int* status, void* stream);
 int64_t imp_gemm_bf16_tc_swap_scratch_floats(int M, int N, int K, int epilogue);
 int imp_gemm_bf16_tc_swap(void* C, int64_t ldc, int epilogue, const void* A, int64_t lda, const void* W, int64_t ldw, int M,
                           int N, int K, float* scratch, int* status, void* stream);
@@ -116,10 +119,13 @@ int imp_sample_mirostat(const float* logits, int64_t ld, int n_rows, int V, cons
                         const float* mu, const float* uniform, int* out, float* surprise, void* stream);
 
 // a norm without statistics behind the sum of two branches (dynamic_tanh.cu)
-int imp_add_dyt(float* h, float mult, const void* t1, const float* parts1, int n_splits1, const void* y1, const int* row1, const float* wts1,
-                int top1, const void* t2, const float* parts2, int n_splits2, const void* y2, const int* row2, const float* wts2, int top2,
-                const float* alpha, const void* w, const void* b, void* out, const int* rows, int n_stream, int n_out, int d, int act_dtype,
-                int w_dtype, void* stream);
+int imp_add_dyt(float* h, float mult, const ImpBranchTerm* first, const ImpBranchTerm* second, const float* alpha, const void* w,
+                const void* b, void* out, const int* rows, int n_stream, int n_out, int d, int act_dtype, int w_dtype, void* stream);
+// RMS norms of what a sublayer gives, joined with the residual sum, and of a token's embedding (branch_norm.cu)
+int imp_add_rms_branch(float* h, const ImpBranchTerm* first, const ImpBranchTerm* second, const float* bias, const void* w, void* out,
+                       int n, int d, float eps, int act_dtype, int w_dtype, void* stream);
+int imp_embedding_rmsnorm(float* h, void* out, const void* table, const int* ids, const void* w, int n, int d, int vocab, float scale,
+                          float eps, int act_dtype, int table_dtype, int w_dtype, int* status, void* stream);
 // layer norm with the residual sum, and streams whose branches carry a factor per column (layernorm.cu)
 int imp_add_layernorm(float* h, const void* branch, const float* col_scale, const void* w, void* out, const int* rows,
                       int n_out_rows, int d, float eps, int act_dtype, int w_dtype, int write_h, void* stream);
@@ -162,22 +168,14 @@ int imp_gla_scan(const void* proj, int64_t ld, const float* alpha, float q_scale
 int imp_gla_decode(const void* proj, int64_t ld, int n_tokens, int H, int D, int Dv, int R, const float* w2t, const float* bias, float tau,
                    float q_scale, const float* out_w, float eps, float* state, const int* slots, void* y, int act_dtype, void* stream);
 // attention with normalised, partly rotated, scaled and gated heads; blocks of two mixers (qkv_prepare.cu)
-int imp_qkv_prepare(const void* proj, int64_t ld, int n_tokens, int Hq, int Hkv, int D, int Dv, int Dc, const float* q_norm_w,
-                    const float* k_norm_w, float eps, int v_norm, const float* inv_freq, int rot, const float* head_mult,
-                    const int* positions, const int* seq_of_token, const int* block_table, int bt_stride, int n_seqs, void* q_out,
-                    int64_t q_ld, void* k_cache, void* v_cache, int page_size, int num_pages, int act_dtype, int* status,
-                    void* stream);
-int imp_qkv_prepare_ex(const void* proj, int64_t ld, int n_tokens, int Hq, int Hkv, int D, int Dv, int Dc, const float* q_norm_w,
-                       const float* k_norm_w, float eps, int v_norm, const float* inv_freq, int rot, int pairing, int v_share,
-                       const float* head_mult, const int* positions, const int* seq_of_token, const int* block_table, int bt_stride,
-                       int n_seqs, void* q_out, int64_t q_ld, void* k_cache, void* v_cache, int page_size, int num_pages, int act_dtype,
-                       int* status, void* stream);
+int imp_qkv_prepare(const ImpQkvPrepare* args, int* status, void* stream);
 int imp_diff_combine(void* y, const void* attn, int64_t ld, int n_tokens, int G, int R, int Dc, int Dv, const float* lambda, float eps,
                      float out_scale, int dtype, void* stream);
 int imp_head_gate(void* y, int64_t y_ld, const void* g, int64_t g_ld, int n_tokens, int H, int Dv, int dtype, void* stream);
 int imp_rms_pair_mean(void* out, const void* a, const float* wa, float ca, const void* b, const float* wb, float cb, int n_rows, int d,
                       float eps, int dtype, void* stream);
-int imp_gated_act(void* out, const void* gate_up, int n_tokens, int F, int block, int act, float limit, int dtype, void* stream);
+int imp_gated_act(void* out, const void* gate_up, int n_tokens, int F, int block, int act, float limit, const float* bias, int dtype,
+                  void* stream);
 int imp_act_rows(void* out, const void* x, int64_t ld, int n_tokens, int n, int act, int dtype, void* stream);
 int imp_gather_head_cols(void* dst, const void* src, int n_tokens, int H, int ds, int n, int dtype, void* stream);
 // a short causal convolution added to its input; a normalised polynomial as activation (short_conv.cu)
@@ -190,7 +188,8 @@ int imp_grouped_gemm(void* C, int64_t ldc, int64_t c_group_cols, const void* A, 
                      int M, int N, int K, int G, int swiglu, int dtype, void* stream);
 int imp_grouped_gemm_ex(void* C, int64_t ldc, int64_t c_group_cols, const void* A, int64_t lda, int64_t a_group_cols,
                         const int* a_rows, const void* W, const void* W2, int64_t w_group_stride, int64_t ldw, const int* seg,
-                        int M, int N, int K, int G, int swiglu, int epi, const void* gate, int64_t gate_ld, int dtype, void* stream);
+                        int M, int N, int K, int G, int swiglu, int epi, const void* gate, int64_t gate_ld, int act, float limit, int dtype,
+                        void* stream);
 int imp_transpose_groups(void* dst, const void* src, int G, int R, int Cn, int dtype, void* stream);
 // latent attention (latent_attention.cu)
 int imp_latent_prepare(const void* proj, int64_t ld, int n_tokens, int q_rank, int kv_rank, int rot, const float* wq,
@@ -221,12 +220,12 @@ int imp_wkv_output(void* y, const float* o, const void* g, int64_t ldg, const fl
 int imp_moe_route(const void* x, int64_t ldx, int n_tokens, int d, const float* wr, const float* br, int E, int top, const float* wg,
                   int* idx, float* wts, float* gate, int act_dtype, void* stream);
 int imp_moe_route_ex(const void* x, int64_t ldx, int n_tokens, int d, const float* wr, const float* br, int E, int top, const float* wg,
-                     int* idx, float* wts, float* gate, int score_mode, int n_groups, int keep, int group_top, float weight_scale, int act_dtype,
-                     void* stream);
+                     int* idx, float* wts, float* gate, int score_mode, int n_groups, int keep, int group_top, float weight_scale,
+                     const float* choice_bias, int renormalise, int act_dtype, void* stream);
 int imp_moe_sort(const int* idx, int n_tokens, int top, int E, int* seg, int* row_token, int* pair_row, void* stream);
 int imp_gather_rows(void* dst, const void* src, int64_t ld, const int* idx, int n_rows, int d, int dtype, void* stream);
 int imp_moe_combine(void* out, const void* y, const int* pair_row, const float* wts, int n_tokens, int top, const void* shared,
-                    const float* gate, int d, int act_dtype, void* stream);
+                    const float* gate, const void* input, int64_t input_ld, int d, int act_dtype, void* stream);
 }
 
 // Epilogues of the products over groups (imp_grouped_gemm_ex).

@@ -58,13 +58,19 @@ void swiglu(Runtime& rt, Tensor out, const Tensor& gate_up, int interleave) {
 }
 
 void gated_act(Runtime& rt, Tensor out, const Tensor& gate_up, int interleave, GatedAct act) {
-    if (act.kind == 0) return swiglu(rt, out, gate_up, interleave);
+    if (act.kind == 0 && !act.bias) return swiglu(rt, out, gate_up, interleave);
     need(cols(gate_up) == 2 * cols(out) && rows(gate_up) == rows(out) && gate_up.dtype == out.dtype && contiguous(out) &&
              contiguous(gate_up),
          "gated_act: gate_up must be [T, 2F] beside out [T, F], both dense");
     ++rt.launches;
-    check_launch(imp_gated_act(out.data, gate_up.data, (int)rows(out), (int)cols(out), interleave, act.kind, act.limit, out.dtype, rt.stream),
+    check_launch(imp_gated_act(out.data, gate_up.data, (int)rows(out), (int)cols(out), interleave, act.kind, act.limit, act.bias, out.dtype,
+                               rt.stream),
                  "gated_act");
+}
+
+void add_bias(Runtime& rt, Tensor x, const float* bias) {
+    ++rt.launches;
+    check_launch(imp_add_bias(x.data, x.stride0, (int)rows(x), (int)cols(x), bias, x.dtype, rt.stream), "add_bias");
 }
 
 void embedding(Runtime& rt, Tensor out, const Tensor& table, const int32_t* ids, int n, float scale) {
@@ -105,7 +111,7 @@ static void gemm_stream(Runtime& rt, Tensor out, const Tensor& a, const Tensor& 
     check_launch(rc, "gemm_bf16_stream");
 }
 
-static bool gemm_tc(Runtime& rt, Tensor out, const Tensor& a, const Tensor& w, int epilogue = -1, float limit = 0.f) {
+static bool gemm_tc(Runtime& rt, Tensor out, const Tensor& a, const Tensor& w, int epilogue = -1, float limit = 0.f, const float* bias = nullptr) {
     if (epilogue < 0) epilogue = out.dtype == F32 ? TC_OUT_F32 : TC_OUT_BF16;
     if (epilogue == TC_OUT_BF16 || epilogue == TC_OUT_F32) {
         // few 256 x 256 tiles for the device's CTA pairs (a portion of a prompt): the K range in parts, then their sum
@@ -124,7 +130,7 @@ static bool gemm_tc(Runtime& rt, Tensor out, const Tensor& a, const Tensor& w, i
             rt.arena->restore(mark);
         }
     }
-    const int rc = imp_gemm_bf16_tc_act(out.data, out.stride0, epilogue, limit, a.data, a.stride0, w.data, w.stride0, (int)rows(a),
+    const int rc = imp_gemm_bf16_tc_act(out.data, out.stride0, epilogue, limit, bias, a.data, a.stride0, w.data, w.stride0, (int)rows(a),
                                     (int)rows(w), (int)cols(a), rt.status, rt.stream);
     if (rc == -2) return false;
     ++rt.launches;
@@ -132,12 +138,12 @@ static bool gemm_tc(Runtime& rt, Tensor out, const Tensor& a, const Tensor& w, i
     return true;
 }
 
-static bool gemm_tc_swap(Runtime& rt, Tensor out, const Tensor& a, const Tensor& w, int epilogue = -1, float limit = 0.f) {
+static bool gemm_tc_swap(Runtime& rt, Tensor out, const Tensor& a, const Tensor& w, int epilogue = -1, float limit = 0.f, const float* bias = nullptr) {
     if (epilogue < 0) epilogue = out.dtype == F32 ? TC_OUT_F32 : TC_OUT_BF16;
     const int M = (int)rows(a), N = (int)rows(w), K = (int)cols(a);
     const int64_t n_scratch = imp_gemm_bf16_tc_swap_scratch_floats(M, N, K, epilogue);
     float* scratch = n_scratch > 0 ? (float*)rt.arena->alloc((size_t)n_scratch * 4) : nullptr;
-    const int rc = imp_gemm_bf16_tc_swap_act(out.data, out.stride0, epilogue, limit, a.data, a.stride0, w.data, w.stride0, M, N, K, scratch,
+    const int rc = imp_gemm_bf16_tc_swap_act(out.data, out.stride0, epilogue, limit, bias, a.data, a.stride0, w.data, w.stride0, M, N, K, scratch,
                                          rt.status, rt.stream);
     if (rc == -2) return false;
     rt.launches += n_scratch > 0 ? 2 : 1;
@@ -170,13 +176,15 @@ static void sum_term(Runtime& rt, const Tensor& t, const float* parts, int n_spl
     if (r.y) {
         need(contiguous(t), "summed: routed rows are added into a dense tensor");
         ++rt.launches;
-        check_launch(imp_moe_combine(t.data, r.y, r.pair_row, r.wts, (int)rows(t), r.top, nullptr, nullptr, (int)cols(t), t.dtype == F32 ? 0 : 1, rt.stream),
+        check_launch(imp_moe_combine(t.data, r.y, r.pair_row, r.wts, (int)rows(t), r.top, nullptr, nullptr, r.input, r.input_ld, (int)cols(t),
+                                     t.dtype == F32 ? 0 : 1, rt.stream),
                      "moe_combine");
     }
 }
 
 Tensor summed(Runtime& rt, const Branch& b) {
     sum_term(rt, b.t, b.parts, b.n_splits, b.rows);
+    if (b.bias && !b.empty()) add_bias(rt, b.t, b.bias);
     if (b.own_norm.weight && !b.empty()) {
         need(contiguous(b.t), "summed: a branch with a norm of its own must be dense");
         ++rt.launches;
@@ -263,10 +271,10 @@ void linear_gated(Runtime& rt, Tensor out, const Tensor& x, const Tensor& w, Gat
     const int epi = act.kind == 0 ? TC_OUT_SWIGLU : act.kind == 1 ? TC_OUT_GEGLU : TC_OUT_CLIPGLU;
     const bool bf16 = x.dtype == BF16 && w.dtype == BF16 && out.dtype == BF16;
     const bool lib = use_library_gemm();
-    if (bf16 && M > stream_m_max() && M <= SMALL_M_MAX && !lib && gemm_tc_swap(rt, out, x, w, epi, act.limit)) return;
+    if (bf16 && M > stream_m_max() && M <= SMALL_M_MAX && !lib && gemm_tc_swap(rt, out, x, w, epi, act.limit, act.bias)) return;
     if (bf16 && M <= SMALL_M_MAX) {
         const int rc = imp_gemm_bf16_stream_gated(out.data, out.stride0, x.data, x.stride0, w.data, w.stride0, (int)M, (int)(2 * F),
-                                                  (int)cols(x), act.kind, act.limit, rt.stream);
+                                                  (int)cols(x), act.kind, act.limit, act.bias, rt.stream);
         if (rc != -2) {
             ++rt.launches;
             check_launch(rc, "gemm_bf16_stream_gated");
@@ -274,8 +282,8 @@ void linear_gated(Runtime& rt, Tensor out, const Tensor& x, const Tensor& w, Gat
         }
     }
     if (bf16 && !lib) {
-        if (M <= TC_SWAP_MAX_M && gemm_tc_swap(rt, out, x, w, epi, act.limit)) return;
-        if (gemm_tc(rt, out, x, w, epi, act.limit)) return;
+        if (M <= TC_SWAP_MAX_M && gemm_tc_swap(rt, out, x, w, epi, act.limit, act.bias)) return;
+        if (gemm_tc(rt, out, x, w, epi, act.limit, act.bias)) return;
     }
     Tensor gu = rt.empty(M, 2 * F, x.dtype);
     linear(rt, gu, x, w);
@@ -338,6 +346,22 @@ Tensor to_float32(Runtime& rt, WeightStore& store, const Tensor& t) {
     if (t.dtype == F32) IMP_CUDA(cudaMemcpyAsync(f.data, t.data, (size_t)numel(t) * 4, cudaMemcpyDeviceToDevice, rt.stream));
     else cast(rt, f, t);
     return f;
+}
+
+Tensor upload_f32(Runtime& rt, WeightStore& store, const std::vector<float>& v) {
+    Tensor t = store.alloc(F32, {(int64_t)v.size()});
+    IMP_CUDA(cudaMemcpyAsync(t.data, v.data(), v.size() * 4, cudaMemcpyHostToDevice, rt.stream));
+    IMP_CUDA(cudaStreamSynchronize(rt.stream));
+    return t;
+}
+
+std::vector<float> download_f32(Runtime& rt, WeightStore& store, const Tensor& t) {
+    Tensor f = to_float32(rt, store, t);
+    std::vector<float> v((size_t)numel(f));
+    IMP_CUDA(cudaMemcpyAsync(v.data(), f.data, v.size() * 4, cudaMemcpyDeviceToHost, rt.stream));
+    IMP_CUDA(cudaStreamSynchronize(rt.stream));
+    store.release(f.data);
+    return v;
 }
 
 Tensor cat_rows(Runtime& rt, WeightStore& store, const std::vector<Tensor>& parts) {

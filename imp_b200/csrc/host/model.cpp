@@ -110,9 +110,15 @@ void Diagnostics::dump_stream(Step& st, int run, const Tensor& h, const Branch& 
             } else if (r.y) {
                 const size_t P = T * (size_t)r.top;
                 const std::vector<char> y = fetch(r.y, P * d * el), row = fetch(r.pair_row, P * 4), w = fetch(r.wts, P * 4);
-                for (size_t q = 0; q < P; ++q)
+                const std::vector<char> in = r.input ? fetch(r.input, ((T - 1) * (size_t)r.input_ld + d) * el) : std::vector<char>();
+                for (size_t q = 0; q < P; ++q) {
+                    const size_t t = q / (size_t)r.top;
+                    const int32_t place = ((const int32_t*)row.data())[q];   // negative: an identity expert gives the input
+                    if (place < 0 && !r.input) continue;
                     for (size_t c = 0; c < d; ++c)
-                        hs[q / (size_t)r.top * d + c] += pending.mult * ((const float*)w.data())[q] * widen1(y, (size_t)((const int32_t*)row.data())[q] * d + c);
+                        hs[t * d + c] += pending.mult * ((const float*)w.data())[q] *
+                                         (place < 0 ? widen1(in, t * (size_t)r.input_ld + c) : widen1(y, (size_t)place * d + c));
+                }
             } else {
                 const std::vector<char> v = fetch(t.data, n * el);
                 for (size_t i = 0; i < n; ++i) hs[i] += pending.mult * widen1(v, i);
@@ -494,6 +500,7 @@ Tensor DeviceModel::forward(Step& st) {
     st.diag = diag_.get();
     st.layer = -1;
     if (diag_) diag_->begin(st);
+    st.stream_copy = Tensor{};
     Tensor h = embedding_->forward(st, embedding_cache_position_ >= 0 ? &embedding_cache_ : nullptr);
     stage(st, "embedding", h);
     st.embedding_out = Tensor{};
@@ -503,7 +510,6 @@ Tensor DeviceModel::forward(Step& st) {
         IMP_CUDA(cudaMemcpyAsync(st.embedding_out.data, h.data, (size_t)numel(h) * elem_size(h.dtype), cudaMemcpyDeviceToDevice, rt_->stream));
     }
     Branch pending;
-    st.stream_copy = Tensor{};
     for (size_t j = 0; j < order_.size(); ++j) {
         rt_->arena->next_layer();
         st.layer = order_[j];

@@ -2,6 +2,8 @@
 // and the choice of the attention kernel for a step.  Nothing here computes on the host.
 #pragma once
 
+#include "../branch_terms.h"
+#include "../qkv_prepare.h"
 #include "parts.hpp"
 
 namespace imp {
@@ -26,6 +28,8 @@ Tensor interleave_gate_up(Runtime& rt, WeightStore& store, const Tensor& gate, c
 // Stack matrices along the output dimension (widening to float32 if their types differ).
 Tensor cat_rows(Runtime& rt, WeightStore& store, const std::vector<Tensor>& parts);
 Tensor to_float32(Runtime& rt, WeightStore& store, const Tensor& t);   // a 32-bit copy of a small weight
+Tensor upload_f32(Runtime& rt, WeightStore& store, const std::vector<float>& v);
+std::vector<float> download_f32(Runtime& rt, WeightStore& store, const Tensor& t);
 
 void swiglu(Runtime& rt, Tensor out, const Tensor& gate_up, int interleave);
 // The same with the activation chosen: 0 silu(g) u, 1 gelu(g) u (tanh form), 2 both clipped to `limit`:
@@ -33,17 +37,28 @@ void swiglu(Runtime& rt, Tensor out, const Tensor& gate_up, int interleave);
 struct GatedAct {
     int kind;
     float limit;
-    GatedAct(int k, float l = 0.f) : kind(k), limit(l) {}
+    const float* bias;   // a number per row of the stacked gate and up matrix, in its order, added first; or null
+    GatedAct(int k, float l = 0.f, const float* b = nullptr) : kind(k), limit(l), bias(b) {}
 };
 void gated_act(Runtime& rt, Tensor out, const Tensor& gate_up, int interleave, GatedAct act);
 void linear_gated(Runtime& rt, Tensor out, const Tensor& x, const Tensor& w_interleaved, GatedAct act);
 // out = max(x w^T, 0)^2, in the product's epilogue where that kernel runs.
 void linear_relu2(Runtime& rt, Tensor out, const Tensor& x, const Tensor& w);
 void cast(Runtime& rt, Tensor dst, const Tensor& src);
+void add_bias(Runtime& rt, Tensor x, const float* bias);   // x[r, c] += bias[c]
 
 // The tensor a branch stands for (runs the summing kernel if its parts are still apart).
 Tensor summed(Runtime& rt, const Branch& b);
 inline Tensor summed(Step& st, const Branch& b) { return summed(*st.rt, b); }
+
+// A branch's summand as the kernels take it (csrc/branch_terms.h); the input of identity experts, if given, must be dense.
+inline ImpBranchTerm branch_term(const Tensor& t, const float* parts, int n_splits, const RoutedRows& r) {
+    ImpBranchTerm b{};
+    if (parts) b.parts = parts, b.n_splits = n_splits;
+    else if (r.y) b.y = r.y, b.pair_row = r.pair_row, b.wts = r.wts, b.top = r.top, b.input = r.input;
+    else b.t = t.data;
+    return b;
+}
 
 // h (+= branch); out = rmsnorm(h) * (weight + offset).  With `rows`, output row r reads stream row
 // rows[r] and h is left untouched.  A branch with unsummed parts is added on the way.
@@ -57,6 +72,18 @@ struct AttentionGeometry {
     int hq, hkv, dh, window;
     float scale;
 };
+// The part of imp_qkv_prepare's arguments that the step, the cache and the geometry give; D and Dv are the caller's.
+inline ImpQkvPrepare qkv_prepare_args(const Step& st, const ImpCacheView& cv, const AttentionGeometry& g, const Tensor& proj, const Tensor& q) {
+    ImpQkvPrepare p;
+    p.proj = proj.data, p.ld = proj.stride0, p.n_tokens = (int)rows(proj);
+    p.Hq = g.hq, p.Hkv = g.hkv, p.Dc = g.dh;
+    p.positions = st.view.positions, p.seq_of_token = st.view.seq_of_token;
+    p.block_table = cv.block_table, p.bt_stride = cv.bt_stride, p.n_seqs = st.B();
+    p.q_out = q.data, p.q_ld = q.stride0;
+    p.k_cache = cv.writes ? cv.k_pages : nullptr, p.v_cache = cv.writes ? cv.v_pages : nullptr;
+    p.page_size = cv.page_size, p.num_pages = cv.num_pages, p.act_dtype = st.rt->dtype;
+    return p;
+}
 struct QkNorm {
     const float* q_w = nullptr;   // 32-bit copies of the per-head norm weights, or null
     const float* k_w = nullptr;

@@ -74,14 +74,15 @@ IMP_EXPORT int imp_op_linear_swiglu(const ImpTensor* out, const ImpTensor* x, co
     });
 }
 
-// The same with the activation chosen: 0 silu, 1 the tanh form of gelu, 2 both values clipped to `limit` (see GatedAct).
+// The same with the activation chosen: 0 silu, 1 the tanh form of gelu, 2 both values clipped to `limit`; behind a bias per row of the
+// weight, or null (see GatedAct).
 IMP_EXPORT int imp_op_linear_gated(const ImpTensor* out, const ImpTensor* x, const ImpTensor* w_interleaved, int act, float limit,
-                                   void* stream, int32_t* status) {
+                                   const float* bias, void* stream, int32_t* status) {
     return guarded([&] {
         if (!out || !x || !w_interleaved) fail(IMP_ERROR_INVALID_ARG, "imp_op_linear_gated: null tensor");
         Runtime rt = runtime_for(stream, status);
         rt.dtype = x->dtype;
-        linear_gated(rt, *out, *x, *w_interleaved, GatedAct(act, limit));
+        linear_gated(rt, *out, *x, *w_interleaved, GatedAct(act, limit, bias));
         g_fallbacks += rt.fallback_calls;
     });
 }

@@ -57,8 +57,8 @@ CacheSpec CacheSpec::from_json(const Json& j) {
         s.head_dim = (int)j.at("head_dim").as_int();
         s.window = (int)j.get_int("window", 0);
         s.keys_only = j.get_bool("keys_only", false);
-        if (s.num_kv_heads <= 0 || s.head_dim <= 0 || s.window < 0)
-            fail(IMP_ERROR_INVALID_ARG, "cache spec: kv heads and head size must be positive, the window not negative");
+        if (s.num_kv_heads <= 0 || s.head_dim <= 0)
+            fail(IMP_ERROR_INVALID_ARG, "cache spec: kv heads and head size must be positive");
     } else if (kind == "state") {
         s.kind = State;
         for (const auto& t : j.at("tensors").items()) {
@@ -223,6 +223,9 @@ static void copy_out(Step& st, const Tensor& produced, ImpTensor& out) {
 
 void Norm::call(Step& st, ImpCall& c) {
     copy_out(st, add_norm(st, c.h, branch_of(c.branch), c.rows, c.rows ? c.n_rows : 0), c.out);
+}
+Tensor Norm::add_normed(Step&, Tensor, const Branch&) {
+    fail(IMP_ERROR_UNSUPPORTED, "this norm cannot normalise a branch before it is added");
 }
 Tensor Norm::add_norm_store(Step&, Tensor, float, const Branch&) {
     fail(IMP_ERROR_UNSUPPORTED, "this norm cannot store its result as the stream");

@@ -44,7 +44,8 @@ struct StateTensorSpec {
 
 // What a mixer asks of the cache.  Paged: keys and values per token, [kv_heads, head_dim] each;
 // window == 0 keeps every token, window == W keeps what a query at position p may still see
-// (positions > p - W).  State: named tensors of fixed size per request, zero at a request's start.
+// (positions > p - W), window == -C keeps the chunk of C positions that p is in, chunks counted from
+// position 0.  State: named tensors of fixed size per request, zero at a request's start.
 struct CacheSpec {
     enum Kind { None = 0, Paged = 1, State = 2 } kind = None;
     int num_kv_heads = 0, head_dim = 0, window = 0;
@@ -62,6 +63,13 @@ struct CacheSpec {
         return s;
     }
 };
+
+// The first position a query at `pos` may see (imp_first_key of csrc/common.cuh, for the host).
+inline int first_visible(int pos, int window) {
+    if (window > 0) return pos - window + 1 > 0 ? pos - window + 1 : 0;
+    if (window < 0) return pos - pos % (-window);
+    return 0;
+}
 
 // How a mixer wants the new tokens of each sequence cut: runs of up to `tile` consecutive tokens
 // of one sequence, over the sequences whose portion holds min_len <= n < max_len tokens
@@ -98,8 +106,8 @@ struct Step {
     struct Diagnostics* diag = nullptr;        // stage timers / statistics when a debugging switch is set
     int layer = -1;                            // index of the layer that is running (for stage names)
     Tensor embedding_out{};                    // a copy of the embedding's output, kept when a block asks for it (Block::wants_embedding)
-    Tensor stream_copy{};                      // the stream in the activation type, when the block that just ran left one (post-norm
-                                               // blocks: their last norm writes it beside the 32-bit stream); else null
+    Tensor stream_copy{};                      // the stream in the activation type, when the block (or the embedding) that just ran
+                                               // left one: its last norm writes it beside the 32-bit stream; else null
     RowOp* row_op = nullptr;                   // set around one add_norm call by a block that offers its reader's per-row operation
     int context = 0;                           // the sequences' mean length after this step, rounded to a power of two: what
                                                // launch choices may depend on (a decode graph is kept per batch size and context)
@@ -134,12 +142,16 @@ struct BranchNorm {
     float eps = 0.f;
     int dtype = F32;                // of weight and bias
 };
-// Rows of routed experts that nobody has added up yet: row t of the branch is sum_k wts[t, k] * y[pair_row[t, k]].
+// Rows of routed experts that nobody has added up yet: row t of the branch is sum_k wts[t, k] * y[pair_row[t, k]].  A negative
+// pair_row stands for an identity expert, whose output is row t of the sublayer's input: `input`, or with input == null the
+// stream that the branch is added into.
 struct RoutedRows {
     const void* y = nullptr;        // dense [T * top, cols], in the branch tensor's type; null: the branch is not of this form
     const int* pair_row = nullptr;  // [T, top]
     const float* wts = nullptr;     // [T, top]
     int top = 0;
+    const void* input = nullptr;    // rows input_ld apart, in the branch tensor's type
+    int64_t input_ld = 0;
 };
 // One more summand of a branch: a tensor, its unsummed parts, or rows of routed experts (`t` then is where the sum belongs).
 struct BranchTerm {
@@ -160,9 +172,10 @@ struct Branch {
     // says takes_branch_pair(); summed() works it out for everyone else.
     float mult = 1.f;
     BranchTerm second{};
+    const float* bias = nullptr;        // float32 [cols] that is still to be added to the first summand (FeedForward::defer_terms)
     bool empty() const { return t.data == nullptr; }
     bool split() const { return parts != nullptr; }
-    bool compound() const { return rows.y || mult != 1.f || !second.empty(); }
+    bool compound() const { return rows.y || mult != 1.f || !second.empty() || bias; }
     static Branch of(const Tensor& t) { Branch b; b.t = t; return b; }
 };
 
@@ -188,6 +201,11 @@ struct Norm : Part {
     // the activation type.  Only norms that say stores_stream() implement it.
     virtual bool stores_stream() const { return false; }
     virtual Tensor add_norm_store(Step& st, Tensor h, float h_mult, const Branch& branch);
+    // The norm of what a sublayer gives: h <- h + norm(branch), the sum stored as the stream (32-bit); returns its copy in the
+    // activation type.  The branch may come in any form without a col_scale, an own_norm or a factor.  Only norms that say
+    // norms_branches() implement it.
+    virtual bool norms_branches() const { return false; }
+    virtual Tensor add_normed(Step& st, Tensor h, const Branch& branch);
     void call(Step& st, ImpCall& c) override;
 };
 
@@ -218,6 +236,7 @@ struct FeedForward : Part {
     const char* category() const override { return "feed_forward"; }
     bool defer_out = false;
     bool defer_rows = false;                             // may return rows of routed experts that are not added up (Branch::rows)
+    bool defer_terms = false;                            // may return a second summand (a shared expert's output) and a bias with its branch
     virtual Branch forward(Step& st, Tensor x) = 0;
     void call(Step& st, ImpCall& c) override;
 };

@@ -36,6 +36,26 @@ struct RMSNorm : Norm {
         add_rmsnorm(*st.rt, h, branch, weight, out, eps, offset, rows_idx, n_rows);
         return out;
     }
+    // h += rmsnorm(branch) (csrc/branch_norm.cu); the branch's summands, unsummed or not, and its bias enter in 32-bit.
+    bool norms_branches() const override { return offset == 0.f; }
+    Tensor add_normed(Step& st, Tensor h, const Branch& branch) override {
+        Runtime& rt = *st.rt;
+        const int d = (int)cols(h);
+        if (h.dtype != F32 || !contiguous(h) || numel(weight) != d) fail(IMP_ERROR_INVALID_ARG, "rmsnorm: the stream must be dense float32 [T, d], the weight [d]");
+        Branch b = branch;
+        const bool far_input = (b.rows.input && b.rows.input_ld != d) || (b.second.rows.input && b.second.rows.input_ld != d);
+        if (b.col_scale || b.own_norm.weight || b.mult != 1.f || far_input) b = Branch::of(summed(rt, b));
+        Tensor out = rt.empty(rows(h), d);
+        for (const Tensor* t : {&b.t, &b.second.t})
+            if (t->data && (rows(*t) != rows(h) || cols(*t) != d || t->dtype != out.dtype || !contiguous(*t)))
+                fail(IMP_ERROR_INVALID_ARG, "rmsnorm: a branch must be dense, of the stream's shape and the output's type");
+        const ImpBranchTerm first = branch_term(b.t, b.parts, b.n_splits, b.rows), second = branch_term(b.second.t, b.second.parts, b.second.n_splits, b.second.rows);
+        ++rt.launches;
+        rt.split_norm_calls += b.parts || b.second.parts;
+        check_launch(imp_add_rms_branch((float*)h.data, &first, &second, b.bias, weight.data, out.data, (int)rows(h), d, eps, out.dtype, weight.dtype, rt.stream),
+                     "add_rms_branch");
+        return out;
+    }
 };
 
 // ----------------------------------------------------------------------------------- position
@@ -207,18 +227,26 @@ struct GQAAttention : Mixer {
 // down( act(x Wg^T) * (x Wu^T) ), activation in 32-bit (src/graph/executor_forward.cu:933-951,
 // 1124-1140; src/compute/activation.cu:67-87).  params: hidden_size, intermediate_size, activation ("silu", the default,
 // "gelu_tanh": 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))), or "clipped": with `limit`, g = min(gate, limit) and
-// u = min(max(up, -limit), limit) become g sigmoid(1.702 g) (u + 1)).  Registered as "swiglu" and as "gated_mlp".
+// u = min(max(up, -limit), limit) become g sigmoid(1.702 g) (u + 1)), bias (default false: all three products have one; with
+// defer_terms the last one rides with the branch).  Registered as "swiglu" and as "gated_mlp".
 struct SwiGLU : FeedForward {
     int64_t f;
     bool interleaved;
+    bool has_bias = false;
     GatedAct act{0};
     Tensor w_gu, w_down;
+    Tensor gu_bias{}, down_bias{};   // float32; gu_bias in the order of w_gu's rows
     static TensorSpecs specs(const Json& p) {
         const int64_t d = need_int(p, "hidden_size", "swiglu"), f = need_int(p, "intermediate_size", "swiglu");
         TensorSpecs s;
         s.emplace_back("gate_proj", TensorSpec{{f, d}});
         s.emplace_back("up_proj", TensorSpec{{f, d}});
         s.emplace_back("down_proj", TensorSpec{{d, f}});
+        if (p.get_bool("bias", false)) {
+            s.emplace_back("gate_bias", TensorSpec{{f}, "vector", "normal"});
+            s.emplace_back("up_bias", TensorSpec{{f}, "vector", "normal"});
+            s.emplace_back("down_bias", TensorSpec{{d}, "vector", "normal"});
+        }
         return s;
     }
     explicit SwiGLU(BuildArgs& a) {
@@ -239,9 +267,25 @@ struct SwiGLU : FeedForward {
         interleaved = f % SWIGLU_INTERLEAVE == 0 && gate.dtype == up.dtype;
         w_gu = interleaved ? interleave_gate_up(rt, *a.store, gate, up) : cat_rows(rt, *a.store, {gate, up});
         w_down = a.tensor("down_proj");
+        has_bias = a.params.get_bool("bias", false);
+        if (has_bias) {
+            const std::vector<float> bg = download_f32(rt, *a.store, a.tensor("gate_bias")), bu = download_f32(rt, *a.store, a.tensor("up_bias"));
+            std::vector<float> b((size_t)(2 * f));
+            const int64_t run = interleaved ? SWIGLU_INTERLEAVE : f;
+            for (int64_t i = 0; i < f; ++i) {
+                const int64_t at = i / run * 2 * run + i % run;
+                b[(size_t)at] = bg[(size_t)i];
+                b[(size_t)(at + run)] = bu[(size_t)i];
+            }
+            gu_bias = upload_f32(rt, *a.store, b);
+            act.bias = (const float*)gu_bias.data;
+            down_bias = to_float32(rt, *a.store, a.tensor("down_bias"));
+        }
         IMP_CUDA(cudaStreamSynchronize(rt.stream));
         a.drop("gate_proj");
         a.drop("up_proj");
+        if (has_bias)
+            for (const char* n : {"gate_bias", "up_bias", "down_bias"}) a.drop(n);
     }
     Branch forward(Step& st, Tensor x) override {
         Runtime& rt = *st.rt;
@@ -255,7 +299,10 @@ struct SwiGLU : FeedForward {
             gated_act(rt, hid, gu, 0, act);
         }
         if (rt.without('d')) return Branch::of(rt.empty(T, rows(w_down)));
-        return linear(rt, rt.empty(T, rows(w_down)), hid, w_down, defer_out);
+        Branch out = linear(rt, rt.empty(T, rows(w_down)), hid, w_down, defer_out && (!has_bias || defer_terms));
+        if (has_bias && defer_terms) out.bias = (const float*)down_bias.data;
+        else if (has_bias) add_bias(rt, out.t, (const float*)down_bias.data);
+        return out;
     }
 };
 
@@ -294,18 +341,35 @@ struct PreNormBlock : Block {
 
 // ---------------------------------------------------------------------------- embedding, head
 // h[t] = E[id[t]] * scale into the 32-bit stream (src/graph/executor_forward.cu:2786-2797).
-// params: vocab_size, hidden_size, scale (default 1).
+// With `norm` the row is then RMS-normalised with a weight (tensor `norm`), in the same kernel, which also leaves the stream's
+// copy in the activation type (Step::stream_copy).
+// params: vocab_size, hidden_size, scale (default 1), norm (default false), norm_eps.
 struct TokenEmbedding : Embedding {
-    Tensor weight;
-    float scale;
-    explicit TokenEmbedding(BuildArgs& a) : weight(a.tensor("weight")), scale((float)a.params.get_double("scale", 1.0)) {}
+    Tensor weight, norm{};
+    float scale, eps;
+    explicit TokenEmbedding(BuildArgs& a)
+        : weight(a.tensor("weight")), scale((float)a.params.get_double("scale", 1.0)), eps((float)a.params.get_double("norm_eps", 1e-6)) {
+        if (a.params.get_bool("norm", false)) norm = a.tensor("norm");
+    }
     static TensorSpecs specs(const Json& p) {
+        const int64_t d = need_int(p, "hidden_size", "token_embedding");
         TensorSpecs s;
-        s.emplace_back("weight", TensorSpec{{need_int(p, "vocab_size", "token_embedding"), need_int(p, "hidden_size", "token_embedding")}});
+        s.emplace_back("weight", TensorSpec{{need_int(p, "vocab_size", "token_embedding"), d}});
+        if (p.get_bool("norm", false)) s.emplace_back("norm", TensorSpec{{d}, "norm", "one_plus_normal"});
         return s;
     }
     Tensor forward(Step& st, LayerCache*) override {
         Tensor out = st.rt->empty(st.T(), cols(weight), F32, /*step=*/true);
+        if (norm.data) {
+            Runtime& rt = *st.rt;
+            Tensor copy = rt.empty(st.T(), cols(weight));
+            ++rt.launches;
+            check_launch(imp_embedding_rmsnorm((float*)out.data, copy.data, weight.data, st.view.token_ids, norm.data, st.T(), (int)cols(weight),
+                                               (int)rows(weight), scale, eps, copy.dtype, weight.dtype, norm.dtype, rt.status, rt.stream),
+                         "embedding_rmsnorm");
+            st.stream_copy = copy;
+            return out;
+        }
         embedding(*st.rt, out, weight, st.view.token_ids, st.T(), scale);
         return out;
     }

@@ -45,17 +45,16 @@ struct DynamicTanh : Norm {
         Tensor out = rt.empty(n, d, -1, /*step=*/rows_idx != nullptr);
         if (h.dtype != F32 || !contiguous(h) || numel(weight) != d) fail(IMP_ERROR_INVALID_ARG, "dynamic_tanh: the stream must be dense float32 [T, d], the weight [d]");
         Branch b = branch;
-        if (b.col_scale || b.own_norm.weight) b = Branch::of(summed(rt, b));
+        const bool far_input = (b.rows.input && b.rows.input_ld != d) || (b.second.rows.input && b.second.rows.input_ld != d);
+        if (b.col_scale || b.own_norm.weight || b.bias || far_input) b = Branch::of(summed(rt, b));
         for (const Tensor* t : {&b.t, &b.second.t})
             if (t->data && (rows(*t) != rows(h) || cols(*t) != d || t->dtype != out.dtype || !contiguous(*t)))
                 fail(IMP_ERROR_INVALID_ARG, "dynamic_tanh: a branch must be dense, of the stream's shape and the output's type");
-        auto dense = [](const Tensor& t, const float* parts, const RoutedRows& r) { return parts || r.y ? nullptr : t.data; };
+        const ImpBranchTerm first = branch_term(b.t, b.parts, b.n_splits, b.rows), second = branch_term(b.second.t, b.second.parts, b.second.n_splits, b.second.rows);
         ++rt.launches;
         rt.split_norm_calls += b.parts || b.second.parts;
-        check_launch(imp_add_dyt((float*)h.data, b.mult, dense(b.t, b.parts, b.rows), b.parts, b.n_splits, b.rows.y, b.rows.pair_row, b.rows.wts, b.rows.top,
-                                 dense(b.second.t, b.second.parts, b.second.rows), b.second.parts, b.second.n_splits, b.second.rows.y,
-                                 b.second.rows.pair_row, b.second.rows.wts, b.second.rows.top, (const float*)alpha.data, weight.data, bias.data, out.data,
-                                 rows_idx, (int)rows(h), (int)n, d, out.dtype, weight.dtype, rt.stream),
+        check_launch(imp_add_dyt((float*)h.data, b.mult, &first, &second, (const float*)alpha.data, weight.data, bias.data, out.data, rows_idx, (int)rows(h),
+                                 (int)n, d, out.dtype, weight.dtype, rt.stream),
                      "add_dyt");
         return out;
     }
@@ -189,7 +188,7 @@ struct ParallelBlock : Block {
             if (forked) IMP_CUDA(cudaStreamWaitEvent(st.rt->stream, join, 0));
             else f = ffn->forward(st, x);
             stage(st, "feed_forward", f.rows.y ? Branch() : f);
-            if (f.col_scale || f.own_norm.weight || f.mult != 1.f || !f.second.empty()) fail(IMP_ERROR_INTERNAL, "parallel: a feed-forward returns a plain branch");
+            if (f.col_scale || f.own_norm.weight || f.mult != 1.f || !f.second.empty() || f.bias) fail(IMP_ERROR_INTERNAL, "parallel: a feed-forward returns a plain branch");
             out.second.t = f.t;
             out.second.parts = f.parts;
             out.second.n_splits = f.n_splits;

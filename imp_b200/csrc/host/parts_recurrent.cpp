@@ -7,6 +7,7 @@
 #include "kernels.h"
 #include "ops.hpp"
 #include "parts.hpp"
+#include "rotation.hpp"
 
 namespace imp {
 
@@ -39,13 +40,6 @@ Tensor cat_rows_padded(Runtime& rt, WeightStore& store, std::vector<Tensor> in) 
     IMP_CUDA(cudaStreamSynchronize(rt.stream));
     if (pad) store.release(zeros.data);
     return out;
-}
-
-Tensor upload_f32(Runtime& rt, WeightStore& store, const std::vector<float>& v) {
-    Tensor t = store.alloc(F32, {(int64_t)v.size()});
-    IMP_CUDA(cudaMemcpyAsync(t.data, v.data(), v.size() * 4, cudaMemcpyHostToDevice, rt.stream));
-    IMP_CUDA(cudaStreamSynchronize(rt.stream));
-    return t;
 }
 
 // The vectors of one step for imp_lsr_scan, from the layer's workspace.
@@ -490,8 +484,11 @@ struct ChannelDeltaRule : Mixer {
 
 // ------------------------------------------------------------------------------- attention with gated heads
 // Grouped-query softmax attention over the paged cache with, each optional:
-//   an RMS norm per head on q and k (one weight [head_dim] each, shared by the heads), before the rotation;
-//   a rotation of the first rot_dims entries of every q and k head (pairs i, i + rot_dims/2, angle pos * rot_base^(-2i/rot_dims));
+//   biases of the q, k and v products (qkv_bias: tensors q_bias, k_bias, v_bias);
+//   an RMS norm per head on q and k (qk_norm; one weight [head_dim] each, shared by the heads, or with qk_norm_weight false none),
+//   before the rotation or after it (qk_norm_position: "before_rotation", the default, or "after_rotation");
+//   a rotation of the first rot_dims entries of every q and k head (pairs i, i + rot_dims/2, or with rot_pairing "neighbours"
+//   2i, 2i + 1; angle pos * rot_base^(-2i/rot_dims), with the optional scalings of host/rotation.hpp under rot_scaling);
 //   values divided by their root mean square per head before they are cached (value_norm);
 //   a factor per query head on the scores (head_temp, tensor [heads]);
 //   a mask by chunks: a query sees the earlier keys of its own chunk of `chunk` positions, counted from position 0;
@@ -500,13 +497,15 @@ struct ChannelDeltaRule : Mixer {
 // Keys have head_dim entries and values value_dim; the cache's head size is the larger of the two, rounded up to a multiple
 // of 16, and the rest of a cached row is zero.
 // params: hidden_size, num_heads, num_kv_heads, head_dim, value_dim (default head_dim), scale (default head_dim^-1/2), norm_eps,
-//         qk_norm, value_norm, rot_dims (0: none), rot_base, head_temp, chunk (0: none), window (0: all), sink, head_gate.
+//         qkv_bias, qk_norm, qk_norm_weight (default true), qk_norm_position, value_norm, rot_dims (0: none), rot_base,
+//         rot_pairing ("halves", the default, or "neighbours"), rot_scaling, head_temp, chunk (0: none), window (0: all), sink, head_gate.
 struct GatedHeadAttention : Mixer {
     AttentionGeometry g;     // over the cache's head size
     int D, Dv, rot, chunk;
-    bool qk_norm, v_norm, has_temp, has_gate, sink;
-    float eps;
-    Tensor w_in, w_o, q_norm, k_norm, inv_freq, temp, sink0, sink0_l2;
+    int qk_norm = QK_NORM_NONE, pairing = 0;
+    bool norm_weight, has_bias, v_norm, has_temp, has_gate, sink;
+    float eps, rot_mult = 1.f;
+    Tensor w_in, w_o, q_norm{}, k_norm{}, qkv_bias{}, turns{}, temp, sink0, sink0_l2;
 
     struct Sizes {
         int64_t d, H, G, D, Dv, Dc;
@@ -526,7 +525,12 @@ struct GatedHeadAttention : Mixer {
         s.emplace_back("q_proj", TensorSpec{{z.H * z.D, z.d}});
         s.emplace_back("k_proj", TensorSpec{{z.G * z.D, z.d}});
         s.emplace_back("v_proj", TensorSpec{{z.G * z.Dv, z.d}});
-        if (p.get_bool("qk_norm", false)) {
+        if (p.get_bool("qkv_bias", false)) {
+            s.emplace_back("q_bias", TensorSpec{{z.H * z.D}, "vector", "normal"});
+            s.emplace_back("k_bias", TensorSpec{{z.G * z.D}, "vector", "normal"});
+            s.emplace_back("v_bias", TensorSpec{{z.G * z.Dv}, "vector", "normal"});
+        }
+        if (p.get_bool("qk_norm", false) && p.get_bool("qk_norm_weight", true)) {
             s.emplace_back("q_norm", TensorSpec{{z.D}, "norm", "one_plus_normal"});
             s.emplace_back("k_norm", TensorSpec{{z.D}, "norm", "one_plus_normal"});
         }
@@ -537,7 +541,8 @@ struct GatedHeadAttention : Mixer {
     }
     static CacheSpec cache(const Json& p) {
         const Sizes z = sizes(p);
-        return CacheSpec::paged((int)z.G, (int)z.Dc, (int)p.get_int("window", 0));
+        const int chunk = (int)p.get_int("chunk", 0);
+        return CacheSpec::paged((int)z.G, (int)z.Dc, chunk > 0 ? -chunk : (int)p.get_int("window", 0));
     }
     explicit GatedHeadAttention(BuildArgs& a) {
         const char* me = "gated_head_attention";
@@ -552,7 +557,14 @@ struct GatedHeadAttention : Mixer {
         const double scale = p.get_double("scale", 0.0);
         g.scale = scale > 0 ? (float)scale : (float)(1.0 / std::sqrt((double)D));
         eps = (float)p.get_double("norm_eps", 1e-6);
-        qk_norm = p.get_bool("qk_norm", false);
+        has_bias = p.get_bool("qkv_bias", false);
+        const std::string np = p.get_string("qk_norm_position", "before_rotation"), pr = p.get_string("rot_pairing", "halves");
+        if (np != "before_rotation" && np != "after_rotation")
+            fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": unknown qk_norm_position '" + np + "' (known: before_rotation, after_rotation)");
+        if (pr != "halves" && pr != "neighbours") fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": unknown rot_pairing '" + pr + "' (known: halves, neighbours)");
+        if (p.get_bool("qk_norm", false)) qk_norm = np == "after_rotation" ? QK_NORM_AFTER_ROTATION : QK_NORM_BEFORE_ROTATION;
+        norm_weight = qk_norm != QK_NORM_NONE && p.get_bool("qk_norm_weight", true);
+        pairing = pr == "neighbours" ? 1 : 0;
         v_norm = p.get_bool("value_norm", false);
         has_temp = p.get_bool("head_temp", false);
         has_gate = p.get_bool("head_gate", false);
@@ -564,16 +576,23 @@ struct GatedHeadAttention : Mixer {
         if (has_gate) in.push_back(a.tensor("gate_proj"));
         w_in = cat_rows_padded(rt, *a.store, in);
         w_o = a.tensor("o_proj");
-        if (qk_norm) {
+        if (has_bias) {
+            std::vector<float> b;
+            for (const char* n : {"q_bias", "k_bias", "v_bias"}) {
+                const std::vector<float> v = download_f32(rt, *a.store, a.tensor(n));
+                b.insert(b.end(), v.begin(), v.end());
+            }
+            qkv_bias = upload_f32(rt, *a.store, b);
+        }
+        if (norm_weight) {
             q_norm = to_float32(rt, *a.store, a.tensor("q_norm"));
             k_norm = to_float32(rt, *a.store, a.tensor("k_norm"));
         }
         if (has_temp) temp = to_float32(rt, *a.store, a.tensor("head_temp"));
         if (rot > 0) {
-            const double base = p.get_double("rot_base", 10000.0);
-            std::vector<float> f((size_t)rot / 2);
-            for (int i = 0; i < rot / 2; ++i) f[(size_t)i] = (float)std::pow(base, -2.0 * i / rot);
-            inv_freq = upload_f32(rt, *a.store, f);
+            const Rotation r = rotation_frequencies(p, rot, me);
+            turns = upload_f32(rt, *a.store, r.turns());
+            rot_mult = (float)r.mult;
         }
         if (sink) {
             sink0 = upload_f32(rt, *a.store, std::vector<float>((size_t)g.hq, 0.f));
@@ -582,7 +601,9 @@ struct GatedHeadAttention : Mixer {
         IMP_CUDA(cudaStreamSynchronize(rt.stream));
         for (const char* n : {"q_proj", "k_proj", "v_proj"}) a.drop(n);
         if (has_gate) a.drop("gate_proj");
-        if (qk_norm) {
+        if (has_bias)
+            for (const char* n : {"q_bias", "k_bias", "v_bias"}) a.drop(n);
+        if (norm_weight) {
             a.drop("q_norm");
             a.drop("k_norm");
         }
@@ -599,12 +620,14 @@ struct GatedHeadAttention : Mixer {
         linear(rt, proj, x, w_in);
         Tensor q = rt.empty(T, (int64_t)g.hq * g.dh);
         ++rt.launches;
-        check_launch(imp_qkv_prepare(proj.data, proj.stride0, (int)T, g.hq, g.hkv, D, Dv, g.dh, qk_norm ? (const float*)q_norm.data : nullptr,
-                                     qk_norm ? (const float*)k_norm.data : nullptr, eps, v_norm ? 1 : 0, rot > 0 ? (const float*)inv_freq.data : nullptr,
-                                     rot, has_temp ? (const float*)temp.data : nullptr, st.view.positions, st.view.seq_of_token, cv.block_table,
-                                     cv.bt_stride, st.B(), q.data, q.stride0, cv.writes ? cv.k_pages : nullptr, cv.writes ? cv.v_pages : nullptr,
-                                     cv.page_size, cv.num_pages, rt.dtype, rt.status, rt.stream),
-                     "qkv_prepare");
+        ImpQkvPrepare pr = qkv_prepare_args(st, cv, g, proj, q);
+        pr.bias = (const float*)qkv_bias.data;
+        pr.D = D, pr.Dv = Dv;
+        pr.qk_norm = qk_norm, pr.q_norm_w = (const float*)q_norm.data, pr.k_norm_w = (const float*)k_norm.data;
+        pr.eps = eps, pr.v_norm = v_norm ? 1 : 0;
+        pr.turns = (const float*)turns.data, pr.rot = rot, pr.pairing = pairing, pr.rot_mult = rot_mult;
+        pr.head_mult = has_temp ? (const float*)temp.data : nullptr;
+        check_launch(imp_qkv_prepare(&pr, rt.status, rt.stream), "qkv_prepare");
         Tensor attn = rt.empty(T, (int64_t)g.hq * g.dh);
         AttentionExtras ex;
         if (sink) {

@@ -286,7 +286,7 @@ struct LatentAttention : Mixer {
         ++rt.launches;
         const Tensor gate = gated ? col_slice(proj, gate_col, (int64_t)H * Dv) : Tensor{};
         check_launch(imp_grouped_gemm_ex(o.data, o.stride0, Dv, attn.data, attn.stride0, L, nullptr, w_uv.data, nullptr, (int64_t)Dv * C, C, nullptr,
-                                         (int)T, Dv, C, H, 0, gated ? GROUPED_SIGMOID_GATE : GROUPED_PLAIN, gate.data, gate.stride0, dt, rt.stream),
+                                         (int)T, Dv, C, H, 0, gated ? GROUPED_SIGMOID_GATE : GROUPED_PLAIN, gate.data, gate.stride0, 0, 0.f, dt, rt.stream),
                      "grouped_gemm (values)");
         return linear(rt, rt.empty(T, rows(w_o)), o, w_o, defer_out);
     }
@@ -422,15 +422,22 @@ struct Wkv : Mixer {
 // that is added as it is (`shared_gate`: false); scores that are the softmax over all experts, a chosen expert weighing its score
 // (`scores`: "softmax_all"); a group counted by its largest score instead of the sum of two (`group_score`: "max", the default with
 // "softmax_all"; else "top2"); experts without a gate, W_down_e max(W_up_e x, 0)^2 (`expert`: "relu2"; default "swiglu"; no
-// shared expert then).  With `defer_rows` set, and no shared expert, the chosen experts' rows are handed on unsummed (Branch::rows).
+// shared expert then), or with both products clipped (`expert`: "clipped", `expert_limit`, and `shared_limit` for the shared
+// expert; see gated_mlp); with "softmax_all" a learned bias on the choice only (`choice_bias`: tensor, one number per router output,
+// the weights are the scores without it) and weights divided by the chosen ones' sum (`renormalise`); `num_identity` more router
+// outputs behind the experts' that stand for the identity, x itself.  With `defer_rows` set the chosen experts' rows are handed on
+// unsummed (Branch::rows), where there is a shared expert only if `defer_terms` is set as well: its output is the second summand.
 //
-// params: hidden_size, num_experts, top_k, expert_size, shared_size (0: no shared expert), router_bias, scores, weight_scale,
-//         num_groups, keep_groups, group_score, shared_gate, expert.
+// params: hidden_size, num_experts, num_identity, top_k, expert_size, shared_size (0: no shared expert), router_bias, scores,
+//         weight_scale, choice_bias, renormalise, num_groups, keep_groups, group_score, shared_gate, expert, expert_limit, shared_limit.
 struct RoutedExperts : FeedForward {
-    int64_t d, E, top, F, Fs;
+    int64_t d, E, I, R, top, F, Fs;    // R = E + I router outputs
     bool has_bias = true, has_sgate = true, gated_expert = true;
     int score_mode = 0, n_groups = 0, keep_groups = 0, group_top = 2;
     float weight_scale = 1.f;
+    bool renormalise = false;
+    GatedAct act{0}, shared_act{0};
+    Tensor choice_bias{};              // float32 [R]
     Tensor w_gate, w_up, w_down;       // [E * F, d], [E * F, d], [E * d, F]; or w_gate [E * 2F, d], gate and up rows alternating in runs of 8
     bool interleaved = false;
     Tensor router, router_bias, sg;    // float32
@@ -439,17 +446,26 @@ struct RoutedExperts : FeedForward {
 
     static bool gated_kind(const Json& p) {
         const std::string k = p.get_string("expert", "swiglu");
-        if (k != "swiglu" && k != "relu2") fail(IMP_ERROR_INVALID_MODEL, "routed_experts: unknown expert '" + k + "' (known: swiglu, relu2)");
-        return k == "swiglu";
+        if (k != "swiglu" && k != "relu2" && k != "clipped")
+            fail(IMP_ERROR_INVALID_MODEL, "routed_experts: unknown expert '" + k + "' (known: swiglu, relu2, clipped)");
+        return k != "relu2";
+    }
+    static GatedAct gated_act_of(const Json& p, const char* limit) {
+        if (p.get_string("expert", "swiglu") != "clipped") return GatedAct(0);
+        const double l = need_double(p, limit, "routed_experts");
+        if (!(l > 0)) fail(IMP_ERROR_INVALID_MODEL, std::string("routed_experts: '") + limit + "' must be positive");
+        return GatedAct(2, (float)l);
     }
     static TensorSpecs specs(const Json& p) {
         const char* me = "routed_experts";
         const int64_t d = need_int(p, "hidden_size", me), E = need_int(p, "num_experts", me), top = need_int(p, "top_k", me),
-                      F = need_int(p, "expert_size", me), Fs = p.get_int("shared_size", 0);
-        if (E <= 0 || top <= 0 || top > E || F <= 0 || Fs < 0) fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": 0 < top_k <= num_experts and positive sizes");
+                      F = need_int(p, "expert_size", me), Fs = p.get_int("shared_size", 0), I = p.get_int("num_identity", 0), R = E + I;
+        if (E <= 0 || I < 0 || top <= 0 || top > R || F <= 0 || Fs < 0)
+            fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": 0 < top_k <= num_experts + num_identity and positive sizes");
         TensorSpecs s;
-        s.emplace_back("router", TensorSpec{{E, d}});
-        if (p.get_bool("router_bias", true)) s.emplace_back("router_bias", TensorSpec{{E}, "vector", "normal"});
+        s.emplace_back("router", TensorSpec{{R, d}});
+        if (p.get_bool("router_bias", true)) s.emplace_back("router_bias", TensorSpec{{R}, "vector", "normal"});
+        if (p.get_bool("choice_bias", false)) s.emplace_back("choice_bias", TensorSpec{{R}, "vector", "zeros"});
         const int64_t ng = p.get_int("num_groups", 0), keep = p.get_int("keep_groups", 0);
         if (ng < 0 || (ng > 0 && (E % ng || keep <= 0 || keep > ng || top > keep * (E / ng))))
             fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": " + std::to_string(ng) + " groups must divide the " + std::to_string(E) + " experts, and the " +
@@ -457,6 +473,9 @@ struct RoutedExperts : FeedForward {
         const std::string sc = p.get_string("scores", "softmax");
         if (sc != "softmax" && sc != "sigmoid" && sc != "softmax_all")
             fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": unknown scores '" + sc + "' (known: softmax, sigmoid, softmax_all)");
+        if ((p.get_bool("choice_bias", false) || p.get_bool("renormalise", false)) && (sc != "softmax_all" || ng > 0))
+            fail(IMP_ERROR_UNSUPPORTED, std::string(me) + ": choice_bias and renormalise go with scores 'softmax_all' without groups");
+        if (I > 0 && ng > 0) fail(IMP_ERROR_UNSUPPORTED, std::string(me) + ": identity experts go without groups");
         const std::string gsc = p.get_string("group_score", sc == "softmax_all" ? "max" : "top2");
         if ((gsc != "max" && gsc != "top2") || (sc == "softmax_all" && gsc != "max"))
             fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": unknown group_score '" + gsc + "' (known: top2, max; softmax_all goes with max)");
@@ -481,6 +500,10 @@ struct RoutedExperts : FeedForward {
         const char* me = "routed_experts";
         d = need_int(a.params, "hidden_size", me), E = need_int(a.params, "num_experts", me), top = need_int(a.params, "top_k", me);
         F = need_int(a.params, "expert_size", me), Fs = a.params.get_int("shared_size", 0);
+        I = a.params.get_int("num_identity", 0), R = E + I;
+        renormalise = a.params.get_bool("renormalise", false);
+        act = gated_act_of(a.params, "expert_limit");
+        if (Fs > 0) shared_act = gated_act_of(a.params, "shared_limit");
         has_bias = a.params.get_bool("router_bias", true);
         has_sgate = a.params.get_bool("shared_gate", true);
         gated_expert = gated_kind(a.params);
@@ -516,6 +539,7 @@ struct RoutedExperts : FeedForward {
         w_down = cat_rows(rt, *a.store, ds);
         router = to_float32(rt, *a.store, a.tensor("router"));
         if (has_bias) router_bias = to_float32(rt, *a.store, a.tensor("router_bias"));
+        if (a.params.get_bool("choice_bias", false)) choice_bias = to_float32(rt, *a.store, a.tensor("choice_bias"));
         if (Fs > 0) {
             Tensor gate = a.tensor("shared_gate"), up = a.tensor("shared_up");
             s_interleaved = Fs % SWIGLU_INTERLEAVE == 0 && gate.dtype == up.dtype;
@@ -532,6 +556,7 @@ struct RoutedExperts : FeedForward {
         }
         a.drop("router");
         if (has_bias) a.drop("router_bias");
+        if (choice_bias.data) a.drop("choice_bias");
         if (Fs > 0) {
             for (const char* n : {"shared_gate", "shared_up"}) a.drop(n);
             if (has_sgate) a.drop("shared_mix");
@@ -550,13 +575,12 @@ struct RoutedExperts : FeedForward {
         int* pair_row = rt.arena->take<int>((size_t)P);
         rt.launches += 5;
         const bool gated = Fs > 0 && has_sgate;
-        check_launch(imp_moe_route_ex(x.data, x.stride0, (int)T, (int)d, (const float*)router.data, has_bias ? (const float*)router_bias.data : nullptr, (int)E,
+        check_launch(imp_moe_route_ex(x.data, x.stride0, (int)T, (int)d, (const float*)router.data, has_bias ? (const float*)router_bias.data : nullptr, (int)R,
                                       (int)top, gated ? (const float*)sg.data : nullptr, idx, wts, gate, score_mode, n_groups, keep_groups, group_top,
-                                      weight_scale, dt,
-                                      rt.stream),
+                                      weight_scale, (const float*)choice_bias.data, renormalise ? 1 : 0, dt, rt.stream),
                      "moe_route");
         check_launch(imp_moe_sort(idx, (int)T, (int)top, (int)E, seg, row_token, pair_row, rt.stream), "moe_sort");
-        Tensor act = rt.empty(P, F);
+        Tensor hid = rt.empty(P, F);
         Tensor y = rt.empty(P, d);
         // Portions of prompts with much work an expert (rows x F x d of 2^31 and more on average): the list's offsets come to
         // the host, and every expert's rows go to the tensor-memory products as a dense matrix (the wait costs one round
@@ -568,7 +592,7 @@ struct RoutedExperts : FeedForward {
         static const double dense_work = [] { const std::string e = env_string("IMP_B200_MOE_DENSE_WORK", ""); return e.empty() ? 2147483648.0 : std::atof(e.c_str()); }();
         const bool tensor_cores = interleaved || (!gated_expert && w_up.dtype == BF16 && w_down.dtype == BF16 && F % 8 == 0 && d % 8 == 0);
         if (tensor_cores && !st.decode_only() && capturing == cudaStreamCaptureStatusNone && dense_work > 0 &&
-            (double)P / (double)E * (double)F * (double)d >= dense_work) {
+            (double)P / (double)R * (double)F * (double)d >= dense_work) {
             std::vector<int> hseg((size_t)E + 1);
             Tensor xs = rt.empty(P, d);
             check_launch(imp_gather_rows(xs.data, x.data, x.stride0, row_token, (int)P, (int)d, dt, rt.stream), "gather_rows");
@@ -579,50 +603,54 @@ struct RoutedExperts : FeedForward {
                 const int64_t a0 = hseg[(size_t)e], n = hseg[(size_t)e + 1] - a0;
                 if (n <= 0) continue;
                 Tensor xe = tensor2d((char*)xs.data + (size_t)(a0 * d) * el, rt.dtype, n, d);
-                Tensor ae = tensor2d((char*)act.data + (size_t)(a0 * F) * el, rt.dtype, n, F);
+                Tensor ae = tensor2d((char*)hid.data + (size_t)(a0 * F) * el, rt.dtype, n, F);
                 Tensor ye = tensor2d((char*)y.data + (size_t)(a0 * d) * el, rt.dtype, n, d);
                 Tensor wd = tensor2d((char*)w_down.data + (size_t)(e * d * F) * el, w_down.dtype, d, F);
                 if (gated_expert)
-                    linear_swiglu(rt, ae, xe, tensor2d((char*)w_gate.data + (size_t)(e * 2 * F * d) * el, w_gate.dtype, 2 * F, d));
+                    linear_gated(rt, ae, xe, tensor2d((char*)w_gate.data + (size_t)(e * 2 * F * d) * el, w_gate.dtype, 2 * F, d), act);
                 else
                     linear_relu2(rt, ae, xe, tensor2d((char*)w_up.data + (size_t)(e * F * d) * el, w_up.dtype, F, d));
                 linear(rt, ye, ae, wd);
             }
         } else {
             if (!gated_expert)
-                check_launch(imp_grouped_gemm_ex(act.data, F, 0, x.data, x.stride0, 0, row_token, w_up.data, nullptr, F * d, d, seg, (int)P, (int)F, (int)d,
-                                                 (int)E, 0, GROUPED_RELU2, nullptr, 0, dt, rt.stream),
+                check_launch(imp_grouped_gemm_ex(hid.data, F, 0, x.data, x.stride0, 0, row_token, w_up.data, nullptr, F * d, d, seg, (int)P, (int)F, (int)d,
+                                                 (int)E, 0, GROUPED_RELU2, nullptr, 0, 0, 0.f, dt, rt.stream),
                              "grouped_gemm (experts, up)");
             else
-                check_launch(imp_grouped_gemm(act.data, F, 0, x.data, x.stride0, 0, row_token, w_gate.data, interleaved ? nullptr : w_up.data,
-                                              (interleaved ? 2 : 1) * F * d, d, seg, (int)P, (int)F, (int)d, (int)E, interleaved ? 2 : 1, dt, rt.stream),
+                check_launch(imp_grouped_gemm_ex(hid.data, F, 0, x.data, x.stride0, 0, row_token, w_gate.data, interleaved ? nullptr : w_up.data,
+                                                 (interleaved ? 2 : 1) * F * d, d, seg, (int)P, (int)F, (int)d, (int)E, interleaved ? 2 : 1, 0, nullptr, 0,
+                                                 act.kind, act.limit, dt, rt.stream),
                              "grouped_gemm (experts, gate and up)");
-            check_launch(imp_grouped_gemm(y.data, d, 0, act.data, F, 0, nullptr, w_down.data, nullptr, d * F, F, seg, (int)P, (int)d, (int)F, (int)E, 0,
+            check_launch(imp_grouped_gemm(y.data, d, 0, hid.data, F, 0, nullptr, w_down.data, nullptr, d * F, F, seg, (int)P, (int)d, (int)F, (int)E, 0,
                                           dt, rt.stream),
                          "grouped_gemm (experts, down)");
         }
-        Tensor shared{};
+        const bool hand_on = defer_rows && (Fs == 0 || (defer_terms && !gated));
+        Branch shared{};
         if (Fs > 0) {
             Tensor sa = rt.empty(T, Fs);
             if (s_interleaved) {
-                linear_swiglu(rt, sa, x, s_gu);
+                linear_gated(rt, sa, x, s_gu, shared_act);
             } else {
                 Tensor gu = rt.empty(T, 2 * Fs);
                 linear(rt, gu, x, s_gu);
-                swiglu(rt, sa, gu, 0);
+                gated_act(rt, sa, gu, 0, shared_act);
             }
-            shared = rt.empty(T, d);
-            linear(rt, shared, sa, s_down);
+            shared = linear(rt, rt.empty(T, d), sa, s_down, hand_on && defer_out);
         }
         Tensor out = rt.empty(T, d);
-        if (defer_rows && Fs == 0) {
+        if (hand_on) {
             --rt.launches;
             Branch b = Branch::of(out);
-            b.rows = RoutedRows{y.data, pair_row, wts, (int)top};
+            b.rows = RoutedRows{y.data, pair_row, wts, (int)top, x.data, x.stride0};
+            b.second.t = shared.t;
+            b.second.parts = shared.parts;
+            b.second.n_splits = shared.n_splits;
             return b;
         }
-        check_launch(imp_moe_combine(out.data, y.data, pair_row, wts, (int)T, (int)top, Fs > 0 ? shared.data : nullptr, gated ? gate : nullptr, (int)d,
-                                     dt, rt.stream),
+        check_launch(imp_moe_combine(out.data, y.data, pair_row, wts, (int)T, (int)top, Fs > 0 ? shared.t.data : nullptr, gated ? gate : nullptr, x.data,
+                                     x.stride0, (int)d, dt, rt.stream),
                      "moe_combine");
         return Branch::of(out);
     }

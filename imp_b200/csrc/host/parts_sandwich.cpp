@@ -1,4 +1,4 @@
-// Part kinds: a block with a norm before and after each sublayer, a short causal convolution added to what a sublayer
+// Part kinds: a block with a norm before and after each sublayer, a block with a norm after each sublayer only, a short causal convolution added to what a sublayer
 // reads, differential softmax attention (two score maps per head over the same values), and a feed-forward whose
 // activation is a normalised polynomial.  Every size and constant is a parameter; no kind knows which model it is in.
 #include <cmath>
@@ -6,6 +6,7 @@
 #include "kernels.h"
 #include "ops.hpp"
 #include "parts.hpp"
+#include "rotation.hpp"
 
 namespace imp {
 
@@ -20,22 +21,6 @@ double need_double(const Json& p, const char* key, const char* part) {
     const Json* v = p.find(key);
     if (!v || !v->is_number()) fail(IMP_ERROR_INVALID_MODEL, std::string(part) + ": parameter '" + key + "' is missing");
     return v->as_double();
-}
-
-Tensor upload_f32(Runtime& rt, WeightStore& store, const std::vector<float>& v) {
-    Tensor t = store.alloc(F32, {(int64_t)v.size()});
-    IMP_CUDA(cudaMemcpyAsync(t.data, v.data(), v.size() * 4, cudaMemcpyHostToDevice, rt.stream));
-    IMP_CUDA(cudaStreamSynchronize(rt.stream));
-    return t;
-}
-
-std::vector<float> download_f32(Runtime& rt, WeightStore& store, const Tensor& t) {
-    Tensor f = to_float32(rt, store, t);
-    std::vector<float> v((size_t)numel(f));
-    IMP_CUDA(cudaMemcpyAsync(v.data(), f.data, v.size() * 4, cudaMemcpyDeviceToHost, rt.stream));
-    IMP_CUDA(cudaStreamSynchronize(rt.stream));
-    store.release(f.data);
-    return v;
 }
 
 // Rows r0 .. r0 + n of a dense matrix.
@@ -107,8 +92,7 @@ struct ResidualConv : Mixer {
 // Grouped-query softmax attention in which every head holds two score maps over the same values:
 //   q [H heads x 2 maps x D], k [G heads x 2 maps x D], v [G heads x Dv] = W x, laid out head by head as [map 1, map 2];
 //   optionally the first rot_dims entries of every map of q and k are rotated (pairs of neighbours 2i, 2i + 1 or halves
-//   i, i + rot_dims/2; angle pos * f_i, f_i = rot_base^(-2i/rot_dims), optionally with long wavelengths slowed down: f kept
-//   where 2 pi / f < original / high, f / factor where 2 pi / f > original / low, blended linearly in between);
+//   i, i + rot_dims/2; angle pos * f_i, f_i = rot_base^(-2i/rot_dims) with the optional scalings of host/rotation.hpp);
 //   a_m = softmax(scale q_m . k_m over the keys a query sees: all earlier ones, or the last `window`) v for m = 1, 2;
 //   lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + lambda_init (four learned vectors of D, one number for the layer);
 //   o = a_1 - lambda a_2;  y = o / rms(o) per head * (1 - lambda_init);  out = W_o y.
@@ -117,12 +101,12 @@ struct ResidualConv : Mixer {
 // of the group's values.  The cache's head size is the larger of D and Dv, rounded up to a multiple of 16.
 // params: hidden_size, num_heads, num_kv_heads, head_dim, value_dim (default head_dim), scale (default head_dim^-1/2),
 //         lambda_init, norm_eps, window (0: all), rot_dims (0: none), rot_base, rot_pairing ("neighbours" | "halves"),
-//         rot_scaling {factor, low, high, original} (optional).
+//         rot_scaling (optional).
 struct DifferentialAttention : Mixer {
     AttentionGeometry g;   // 2H query heads, 2G key heads, over the cache's head size
     int H, G, D, Dv, rot, pairing;
-    float eps, lambda_init;
-    Tensor w_in, w_o, inv_freq, lambda;
+    float eps, lambda_init, rot_mult = 1.f;
+    Tensor w_in, w_o, turns{}, lambda;
 
     struct Sizes {
         int64_t d, H, G, D, Dv, Dc;
@@ -149,36 +133,6 @@ struct DifferentialAttention : Mixer {
     static CacheSpec cache(const Json& p) {
         const Sizes z = sizes(p);
         return CacheSpec::paged((int)(2 * z.G), (int)z.Dc, (int)p.get_int("window", 0));
-    }
-    // f_i for i < rot/2, with the optional slowing of long wavelengths; computed in double, stored in 32-bit.
-    static std::vector<float> frequencies(const Json& p, int rot) {
-        const char* me = "differential_attention";
-        const double base = p.get_double("rot_base", 10000.0);
-        const Json* sc = p.find("rot_scaling");
-        const bool scaled = sc && sc->is_object();
-        double factor = 1, low = 1, high = 1, original = 1;
-        if (scaled) {
-            factor = need_double(*sc, "factor", me), low = need_double(*sc, "low", me), high = need_double(*sc, "high", me);
-            original = need_double(*sc, "original", me);
-            if (!(factor > 0) || !(high > low) || !(low > 0) || !(original > 0))
-                fail(IMP_ERROR_INVALID_MODEL, std::string(me) + ": rot_scaling needs factor > 0, 0 < low < high and original > 0");
-        }
-        std::vector<float> f((size_t)rot / 2);
-        const double two_pi = 6.283185307179586476925286766559;
-        for (int i = 0; i < rot / 2; ++i) {
-            double v = std::pow(base, -2.0 * i / rot);
-            if (scaled) {
-                const double wave = two_pi / v;
-                if (wave > original / low) {
-                    v /= factor;
-                } else if (!(wave < original / high)) {
-                    const double s = (original / wave - low) / (high - low);
-                    v = (1.0 - s) * v / factor + s * v;
-                }
-            }
-            f[(size_t)i] = (float)v;
-        }
-        return f;
     }
     explicit DifferentialAttention(BuildArgs& a) {
         const char* me = "differential_attention";
@@ -218,7 +172,11 @@ struct DifferentialAttention : Mixer {
         IMP_CUDA(cudaStreamSynchronize(rt.stream));
         if (pad) a.store->release(zeros.data);
         w_o = a.tensor("o_proj");
-        if (rot > 0) inv_freq = upload_f32(rt, *a.store, frequencies(p, rot));
+        if (rot > 0) {
+            const Rotation r = rotation_frequencies(p, rot, me);
+            turns = upload_f32(rt, *a.store, r.turns());
+            rot_mult = (float)r.mult;
+        }
         // lambda, one number, in 32-bit
         const std::vector<float> q1 = download_f32(rt, *a.store, a.tensor("lambda_q1")), k1 = download_f32(rt, *a.store, a.tensor("lambda_k1")),
                                  q2 = download_f32(rt, *a.store, a.tensor("lambda_q2")), k2 = download_f32(rt, *a.store, a.tensor("lambda_k2"));
@@ -241,11 +199,10 @@ struct DifferentialAttention : Mixer {
         linear(rt, proj, x, w_in);
         Tensor q = rt.empty(T, (int64_t)g.hq * g.dh);
         rt.launches += 2;
-        check_launch(imp_qkv_prepare_ex(proj.data, proj.stride0, (int)T, g.hq, g.hkv, D, Dv, g.dh, nullptr, nullptr, eps, 0,
-                                        rot > 0 ? (const float*)inv_freq.data : nullptr, rot, pairing, 2, nullptr, st.view.positions, st.view.seq_of_token,
-                                        cv.block_table, cv.bt_stride, st.B(), q.data, q.stride0, cv.writes ? cv.k_pages : nullptr,
-                                        cv.writes ? cv.v_pages : nullptr, cv.page_size, cv.num_pages, rt.dtype, rt.status, rt.stream),
-                     "qkv_prepare");
+        ImpQkvPrepare pr = qkv_prepare_args(st, cv, g, proj, q);
+        pr.D = D, pr.Dv = Dv, pr.v_share = 2;
+        pr.turns = (const float*)turns.data, pr.rot = rot, pr.pairing = pairing, pr.rot_mult = rot_mult;
+        check_launch(imp_qkv_prepare(&pr, rt.status, rt.stream), "qkv_prepare");
         Tensor attn = rt.empty(T, (int64_t)g.hq * g.dh);
         paged_attention(st, attn, q, g, *cache, tiling_ids, nullptr);
         Tensor y = rt.empty(T, (int64_t)H * Dv);
@@ -399,6 +356,72 @@ struct SandwichBlock : Block {
     }
 };
 
+// -------------------------------------------------------------------------------- a norm after each sublayer only
+// h += post1(mixer(h));  h += post2(ffn(h)): the sublayers read the stream itself, and what they give is normalised before it is
+// added.  One launch stands between a sublayer's last product and the next sublayer's first: the norm takes the branch as it
+// comes (unsummed parts, routed rows, a shared expert's output beside them, a bias), adds it and leaves the stream's copy in the
+// activation type, which is what the next sublayer reads (Step::stream_copy).  Identity experts give the 32-bit stream.
+// Slots: mixer, mixer_post_norm, and with has_ffn (default true) feed_forward, ffn_post_norm.  params: has_ffn.
+struct OutputNormBlock : Block {
+    Mixer* mixer_;
+    FeedForward* ffn = nullptr;
+    Norm *post1, *post2 = nullptr;
+    explicit OutputNormBlock(BuildArgs& a)
+        : mixer_(part_cast<Mixer>(a.part("mixer"), "a mixer")), post1(part_cast<Norm>(a.part("mixer_post_norm"), "a norm")) {
+        if (a.params.get_bool("has_ffn", true)) {
+            ffn = part_cast<FeedForward>(a.part("feed_forward"), "a feed-forward");
+            post2 = part_cast<Norm>(a.part("ffn_post_norm"), "a norm");
+            ffn->defer_out = ffn->defer_rows = ffn->defer_terms = true;
+        }
+        mixer_->defer_out = true;
+        if (!post1->norms_branches() || (post2 && !post2->norms_branches()))
+            fail(IMP_ERROR_INVALID_MODEL, "output_norm: its norms must be able to normalise a branch before it is added (rmsnorm without an offset)");
+    }
+    static std::vector<Slot> slots(const Json& p) {
+        std::vector<Slot> s = {{"mixer", "mixer"}, {"mixer_post_norm", "norm"}};
+        if (p.get_bool("has_ffn", true)) {
+            s.push_back({"feed_forward", "feed_forward"});
+            s.push_back({"ffn_post_norm", "norm"});
+        }
+        return s;
+    }
+    Mixer* mixer() const override { return mixer_; }
+    std::vector<Part*> parts() const override {
+        std::vector<Part*> p = {mixer_, post1};
+        if (ffn) {
+            p.push_back(ffn);
+            p.push_back(post2);
+        }
+        return p;
+    }
+    bool graph_safe() const override {
+        for (Part* p : parts())
+            if (!p->graph_safe()) return false;
+        return true;
+    }
+    Branch forward(Step& st, Tensor h, const Branch& pending, LayerCache* cache) override {
+        Runtime& rt = *st.rt;
+        if (!pending.empty())
+            fail(IMP_ERROR_UNSUPPORTED, "output_norm: the block before it left a branch pending; this block follows the embedding or a block that leaves none");
+        Tensor x = st.stream_copy;
+        if (!x.data || rows(x) != rows(h)) {
+            x = rt.empty(rows(h), cols(h));
+            cast(rt, x, h);
+        }
+        Branch a = mixer_->forward(st, x, cache);
+        stage(st, "mixer", a);
+        x = post1->add_normed(st, h, a);
+        if (ffn) {
+            Branch f = ffn->forward(st, x);
+            stage(st, "feed_forward", f.rows.y ? Branch() : f);
+            if (f.rows.input == x.data) f.rows.input = nullptr;   // the sublayer read the stream: the norm has it in 32-bit
+            x = post2->add_normed(st, h, f);
+        }
+        st.stream_copy = x;
+        return Branch();
+    }
+};
+
 template <typename T> PartClass class_of(TensorSpecs (*specs)(const Json&)) {
     PartClass c;
     if (specs) c.tensor_specs = specs;
@@ -419,6 +442,9 @@ void register_sandwich_parts() {
     PartClass block = class_of<SandwichBlock>(nullptr);
     block.part_slots = &SandwichBlock::slots;
     register_part_class("block", "sandwich", block, true);
+    PartClass out = class_of<OutputNormBlock>(nullptr);
+    out.part_slots = &OutputNormBlock::slots;
+    register_part_class("block", "output_norm", out, true);
 }
 
 }  // namespace imp

@@ -1,6 +1,7 @@
 #include "scheduler.hpp"
 
 #include <algorithm>
+#include <cstdlib>
 #include <random>
 
 namespace imp {
@@ -107,9 +108,9 @@ int Scheduler::pages_for_whole(int n_tokens) const {
     const int P = cache_->page_size();
     int need = 0;
     for (const auto& g : cache_->paged()) {
-        if (g.spec.window > 0) {
-            // live span is at most window + one portion; count the window plus one page of slack
-            const int span = std::min(n_tokens, g.spec.window + std::max(prefill_chunk_size, 1) + P);
+        if (g.spec.window != 0) {
+            // live span is at most a window (or a chunk) + one portion; count that plus one page of slack
+            const int span = std::min(n_tokens, std::abs(g.spec.window) + std::max(prefill_chunk_size, 1) + P);
             need = std::max(need, (span + P - 1) / P);
         } else {
             need = std::max(need, (n_tokens + P - 1) / P);

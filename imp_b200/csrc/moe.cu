@@ -4,10 +4,14 @@
 //   chosen    = the `top` experts with the largest z (the lower index wins a tie)
 //   weight    = softmax over the chosen logits only; or, with sigmoid scores s = sigmoid(z): weight = s * weight_scale
 //               or, with softmax scores over all experts: weight = that softmax * weight_scale, not renormalised
+//               or, with softmax scores and a bias on the choice: the `top` largest softmax + c[e] choose, the weight is the
+//               softmax without c, optionally divided by the chosen ones' sum (+ 1e-20)
 //   groups    = optionally the experts form n_groups equal groups of neighbours; a group's score is the sum of its two
 //               largest scores, or its largest one, and only the experts of the `keep` best groups can be chosen
 //   gate[t]   = sigmoid(x[t] . Wg)                         one number per token, for a shared expert (optional)
 //   out[t]    = sum_k weight[t, k] * y[place(t, k)] + gate[t] * shared[t]
+// Router outputs beyond the experts that have matrices are identity experts: they are chosen and weighed like the others, take no
+// part in the list (place -1), and give the input itself, y = x[t].
 //
 // The expert products run over a list of (token, choice) pairs sorted by expert (see grouped_gemm.cu); moe_sort makes
 // that list on the device: seg [E + 1], the token of every list row, and the row of every pair.  Nothing comes back
@@ -47,14 +51,16 @@ __global__ void __launch_bounds__(ROUTE_BLOCK) moe_route_kernel(const TA* __rest
                                                                const float* __restrict__ wr, const float* __restrict__ br, int E, int top,
                                                                const float* __restrict__ wg, int* __restrict__ idx, float* __restrict__ wts,
                                                                float* __restrict__ gate, int vec, int score_mode, int n_groups, int keep,
-                                                               int group_top, float weight_scale) {
+                                                               int group_top, float weight_scale, const float* __restrict__ choice_bias,
+                                                               int renormalise) {
     pdl_wait();
     pdl_launch_dependents();
-    extern __shared__ __align__(16) float sm[];   // x [TPB][d4], then z [TPB][E], then the groups' scores [TPB][n_groups]
+    extern __shared__ __align__(16) float sm[];   // x [TPB][d4], then z [TPB][E], then the groups' scores [TPB][n_groups], then the choice scores [TPB][E] if they are biased
     const int d4 = (d + 3) & ~3;
     float* xs = sm;
     float* z = sm + (size_t)TPB * d4;
     float* gsc = z + (size_t)TPB * E;
+    float* csc = gsc + (size_t)TPB * n_groups;
     const int t0 = blockIdx.x * TPB, nt = min(TPB, n_tokens - t0);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     for (int e = tid; e < TPB * d4; e += ROUTE_BLOCK) {
@@ -103,7 +109,8 @@ __global__ void __launch_bounds__(ROUTE_BLOCK) moe_route_kernel(const TA* __rest
     __syncthreads();
     // `top` rounds of arg-max over the logits that are left, a warp per token; the lower index wins a tie
     for (int tk = warp; tk < nt; tk += ROUTE_BLOCK / 32) {
-        float* zt = z + tk * E;
+        float* zt = z + tk * E;          // what is chosen from
+        const float* zl = z + tk * E;    // the logits, where the choice scores are others
         const int64_t t = t0 + tk;
         float chosen[ROUTE_MAX_TOP];
         // softmax scores: the choice runs on the logits (same order); the weights need the largest and the sum over all experts
@@ -115,6 +122,10 @@ __global__ void __launch_bounds__(ROUTE_BLOCK) moe_route_kernel(const TA* __rest
             float sum = 0.f;
             for (int e = lane; e < E; e += 32) sum += expf(zt[e] - z_max);
             z_sum = warp_sum(sum);
+            if (choice_bias) {
+                zt = csc + tk * E;
+                for (int e = lane; e < E; e += 32) zt[e] = expf(zl[e] - z_max) / z_sum + choice_bias[e];
+            }
             __syncwarp();
         }
         if (n_groups > 0) {
@@ -166,7 +177,8 @@ __global__ void __launch_bounds__(ROUTE_BLOCK) moe_route_kernel(const TA* __rest
                 const int oa = __shfl_xor_sync(0xffffffffu, at, o);
                 if (ov > best || (ov == best && oa < at)) best = ov, at = oa;
             }
-            chosen[k] = best;
+            if (at >= E) at = 0;     // nothing compares above -inf: the row holds NaNs
+            chosen[k] = score_mode == 2 && choice_bias ? zl[at] : best;
             if (lane == 0) {
                 idx[t * top + k] = at;
                 zt[at] = -INFINITY;
@@ -176,7 +188,13 @@ __global__ void __launch_bounds__(ROUTE_BLOCK) moe_route_kernel(const TA* __rest
         if (lane == 0 && score_mode == 1) {
             for (int k = 0; k < top; ++k) wts[t * top + k] = chosen[k] * weight_scale;   // the scores themselves, not renormalised
         } else if (lane == 0 && score_mode == 2) {
-            for (int k = 0; k < top; ++k) wts[t * top + k] = expf(chosen[k] - z_max) / z_sum * weight_scale;
+            float total = 0.f;
+            for (int k = 0; k < top; ++k) {
+                chosen[k] = expf(chosen[k] - z_max) / z_sum;
+                total += chosen[k];
+            }
+            const float f = renormalise ? weight_scale / (total + 1e-20f) : weight_scale;
+            for (int k = 0; k < top; ++k) wts[t * top + k] = chosen[k] * f;
         } else if (lane == 0) {
             const float largest = chosen[0];   // the first chosen is the largest
             float sum = 0.f;
@@ -216,6 +234,8 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ 
         seg[E] = run;
     }
     __syncthreads();
+    for (int p = tid; p < n_pairs; p += blockDim.x)
+        if (idx[p] >= E) pair_row[p] = -1;   // an identity expert: no row of the list
     // every expert's rows in pair order: a warp walks the pairs of one expert at a time
     const int lane = tid & 31, warp = tid >> 5, n_warps = blockDim.x >> 5;
     for (int e = warp; e < E; e += n_warps) {
@@ -236,18 +256,20 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ 
 
 template <typename TA>
 __global__ void moe_combine_kernel(TA* __restrict__ out, const TA* __restrict__ y, const int* __restrict__ pair_row, const float* __restrict__ wts,
-                                   int top, const TA* __restrict__ shared, const float* __restrict__ gate, int d) {
+                                   int top, const TA* __restrict__ shared, const float* __restrict__ gate, const TA* __restrict__ input,
+                                   int64_t input_ld, int d) {
     pdl_wait();
     pdl_launch_dependents();
     const int64_t t = blockIdx.x;
     const float gt = gate ? gate[t] : 1.f;
-    if ((d & 3) == 0) {
+    if ((d & 3) == 0 && (input_ld & 3) == 0) {
         // four columns a thread (rows start on 8 or 16 bytes: dense [*, d] with d a multiple of 4)
         for (int i = threadIdx.x * 4; i < d; i += blockDim.x * 4) {
             float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
             for (int k = 0; k < top; ++k) {
                 const float wk = wts[t * top + k];
-                const float4 v = Vec4<TA>::load(y + (int64_t)pair_row[t * top + k] * d + i);
+                const int row = pair_row[t * top + k];
+                const float4 v = Vec4<TA>::load(row >= 0 ? y + (int64_t)row * d + i : input + t * input_ld + i);
                 acc.x = fmaf(wk, v.x, acc.x), acc.y = fmaf(wk, v.y, acc.y), acc.z = fmaf(wk, v.z, acc.z), acc.w = fmaf(wk, v.w, acc.w);
             }
             if (shared) {
@@ -260,7 +282,10 @@ __global__ void moe_combine_kernel(TA* __restrict__ out, const TA* __restrict__ 
     }
     for (int i = threadIdx.x; i < d; i += blockDim.x) {
         float acc = 0.f;
-        for (int k = 0; k < top; ++k) acc = fmaf(wts[t * top + k], to_float(y[(int64_t)pair_row[t * top + k] * d + i]), acc);
+        for (int k = 0; k < top; ++k) {
+            const int row = pair_row[t * top + k];
+            acc = fmaf(wts[t * top + k], to_float(row >= 0 ? y[(int64_t)row * d + i] : input[t * input_ld + i]), acc);
+        }
         if (shared) acc = fmaf(gt, to_float(shared[t * d + i]), acc);
         out[t * d + i] = from_float<TA>(acc);
     }
@@ -302,31 +327,31 @@ IMP_API int imp_gather_rows(void* dst, const void* src, int64_t ld, const int* i
 
 template <typename TA, int TPB>
 static cudaError_t launch_route(const void* x, int64_t ldx, int n_tokens, int d, const float* wr, const float* br, int E, int top, const float* wg,
-                                int* idx, float* wts, float* gate, int vec, int score_mode, int n_groups, int keep, int group_top, float weight_scale, size_t smem,
+                                int* idx, float* wts, float* gate, int vec, int score_mode, int n_groups, int keep, int group_top, float weight_scale, const float* choice_bias, int renormalise, size_t smem,
                                 cudaStream_t s) {
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(moe_route_kernel<TA, TPB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
     }
     return imp_launch(moe_route_kernel<TA, TPB>, dim3((n_tokens + TPB - 1) / TPB), dim3(ROUTE_BLOCK), smem, s, (const TA*)x, ldx, n_tokens, d, wr, br,
-                      E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale);
+                      E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, choice_bias, renormalise);
 }
 
 template <typename TA>
 static cudaError_t route_by_size(const void* x, int64_t ldx, int n_tokens, int d, const float* wr, const float* br, int E, int top, const float* wg,
                                  int* idx, float* wts, float* gate, int vec, int score_mode, int n_groups, int keep, int group_top, float weight_scale,
-                                 cudaStream_t s) {
+                                 const float* choice_bias, int renormalise, cudaStream_t s) {
     // more tokens a CTA where there are many (a row of the router is read once per CTA), one where there are few (more CTAs)
     int tpb = n_tokens >= 1024 ? 8 : n_tokens >= 256 ? 4 : n_tokens >= 64 ? 2 : 1;
     const int d4 = (d + 3) & ~3;
-    auto bytes = [&](int t) { return ((size_t)t * d4 + (size_t)t * E + (size_t)t * n_groups) * 4; };
+    auto bytes = [&](int t) { return ((size_t)t * d4 + (size_t)t * E * (choice_bias ? 2 : 1) + (size_t)t * n_groups) * 4; };
     while (tpb > 1 && bytes(tpb) > 160 * 1024) tpb /= 2;
     if (bytes(tpb) > 200 * 1024) return cudaErrorInvalidValue;
     switch (tpb) {
-        case 8: return launch_route<TA, 8>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, bytes(8), s);
-        case 4: return launch_route<TA, 4>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, bytes(4), s);
-        case 2: return launch_route<TA, 2>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, bytes(2), s);
-        default: return launch_route<TA, 1>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, bytes(1), s);
+        case 8: return launch_route<TA, 8>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, choice_bias, renormalise, bytes(8), s);
+        case 4: return launch_route<TA, 4>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, choice_bias, renormalise, bytes(4), s);
+        case 2: return launch_route<TA, 2>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, choice_bias, renormalise, bytes(2), s);
+        default: return launch_route<TA, 1>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, choice_bias, renormalise, bytes(1), s);
     }
 }
 
@@ -334,10 +359,11 @@ static cudaError_t route_by_size(const void* x, int64_t ldx, int n_tokens, int d
 // gate is not written).  idx int32 [T, top], wts float32 [T, top], gate float32 [T].
 // score_mode 0: weights are the softmax over the chosen logits; 1: scores are sigmoid(z) and a weight is its score times
 // weight_scale; 2: scores are the softmax over all experts, a weight as in 1.
+// choice_bias float32 [E] (or null) is added to the scores for the choice only; renormalise: the weights over their sum + 1e-20.
 // group_top: how many of its largest scores a group counts by (1 or 2).  n_groups > 0: only experts of the `keep` best of n_groups equal groups of neighbours can be chosen.
 IMP_API int imp_moe_route_ex(const void* x, int64_t ldx, int n_tokens, int d, const float* wr, const float* br, int E, int top, const float* wg,
-                             int* idx, float* wts, float* gate, int score_mode, int n_groups, int keep, int group_top, float weight_scale, int act_dtype,
-                             void* stream) {
+                             int* idx, float* wts, float* gate, int score_mode, int n_groups, int keep, int group_top, float weight_scale,
+                             const float* choice_bias, int renormalise, int act_dtype, void* stream) {
     if (n_tokens == 0) return 0;
     IMP_CHECK_ARG(x && wr && idx && wts && d > 0 && (!wg || gate), "imp_moe_route: bad argument");
     IMP_CHECK_ARG(E > 0 && E <= ROUTE_MAX_E && top > 0 && top <= E && top <= ROUTE_MAX_TOP,
@@ -345,11 +371,13 @@ IMP_API int imp_moe_route_ex(const void* x, int64_t ldx, int n_tokens, int d, co
     IMP_CHECK_ARG(score_mode >= 0 && score_mode <= 2 && (group_top == 1 || group_top == 2) && n_groups >= 0 && (n_groups == 0 || (E % n_groups == 0 && keep > 0 && keep <= n_groups &&
                                                                                              top <= keep * (E / n_groups))),
                   "imp_moe_route: %d groups over %d experts, %d kept, %d chosen", n_groups, E, keep, top);
+    IMP_CHECK_ARG((!choice_bias && !renormalise) || (score_mode == 2 && n_groups == 0),
+                  "imp_moe_route: a bias on the choice and renormalised weights go with softmax scores over all experts without groups");
     IMP_CHECK_ARG(score_mode != 2 || n_groups == 0 || group_top == 1, "imp_moe_route: with softmax scores over all experts groups count by their largest score");
     const int vec = (d % 4 == 0 && (uintptr_t)wr % 16 == 0 && (!wg || (uintptr_t)wg % 16 == 0)) ? 1 : 0;
     cudaStream_t s = (cudaStream_t)stream;
-    cudaError_t e = act_dtype == IMP_F32 ? route_by_size<float>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, s)
-                                         : route_by_size<__nv_bfloat16>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, s);
+    cudaError_t e = act_dtype == IMP_F32 ? route_by_size<float>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, choice_bias, renormalise, s)
+                                         : route_by_size<__nv_bfloat16>(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, vec, score_mode, n_groups, keep, group_top, weight_scale, choice_bias, renormalise, s);
     if (e != cudaSuccess) {
         imp_set_error("imp_moe_route: %s (rows of %d values, %d experts)", cudaGetErrorString(e), d, E);
         return (int)e;
@@ -359,7 +387,7 @@ IMP_API int imp_moe_route_ex(const void* x, int64_t ldx, int n_tokens, int d, co
 
 IMP_API int imp_moe_route(const void* x, int64_t ldx, int n_tokens, int d, const float* wr, const float* br, int E, int top, const float* wg,
                           int* idx, float* wts, float* gate, int act_dtype, void* stream) {
-    return imp_moe_route_ex(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, 0, 0, 0, 2, 1.f, act_dtype, stream);
+    return imp_moe_route_ex(x, ldx, n_tokens, d, wr, br, E, top, wg, idx, wts, gate, 0, 0, 0, 2, 1.f, nullptr, 0, act_dtype, stream);
 }
 
 IMP_API int imp_moe_sort(const int* idx, int n_tokens, int top, int E, int* seg, int* row_token, int* pair_row, void* stream) {
@@ -374,16 +402,18 @@ IMP_API int imp_moe_sort(const int* idx, int n_tokens, int top, int E, int* seg,
     return 0;
 }
 
-// out [T, d] = sum_k wts[t, k] * y[pair_row[t * top + k]] (+ gate[t] * shared[t]); y [T * top, d], all dense.
+// out [T, d] = sum_k wts[t, k] * y[pair_row[t * top + k]] (+ gate[t] * shared[t]); y [T * top, d], all dense.  A negative place
+// stands for row t of `input` (rows input_ld apart; needed only where identity experts can be chosen).
 IMP_API int imp_moe_combine(void* out, const void* y, const int* pair_row, const float* wts, int n_tokens, int top, const void* shared,
-                            const float* gate, int d, int act_dtype, void* stream) {
+                            const float* gate, const void* input, int64_t input_ld, int d, int act_dtype, void* stream) {
     if (n_tokens == 0) return 0;
     IMP_CHECK_ARG(out && y && pair_row && wts && top > 0 && d > 0, "imp_moe_combine: bad argument");
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t e = act_dtype == IMP_F32 ? imp_launch(moe_combine_kernel<float>, dim3(n_tokens), dim3(256), 0, s, (float*)out, (const float*)y,
-                                                      pair_row, wts, top, (const float*)shared, gate, d)
+                                                      pair_row, wts, top, (const float*)shared, gate, (const float*)input, input_ld, d)
                                          : imp_launch(moe_combine_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(256), 0, s, (__nv_bfloat16*)out,
-                                                      (const __nv_bfloat16*)y, pair_row, wts, top, (const __nv_bfloat16*)shared, gate, d);
+                                                      (const __nv_bfloat16*)y, pair_row, wts, top, (const __nv_bfloat16*)shared, gate, (const __nv_bfloat16*)input,
+                                                      input_ld, d);
     if (e != cudaSuccess) {
         imp_set_error("imp_moe_combine: %s", cudaGetErrorString(e));
         return (int)e;

@@ -2,12 +2,13 @@
 // part, scaled per head and whose values are normalised; and the small kernels of blocks that combine two mixers
 // or gate their heads.
 //
-//   qkv_prepare      per token: q heads  -> RMS norm with a weight shared by the heads (optional), rotation of the
-//                    first `rot` entries (pairs i, i + rot/2, or neighbours 2i, 2i + 1), times a number per head (optional) -> q_out, padded
-//                    to the cache's head size; k heads -> norm, rotation -> K page; v heads -> divided by their
-//                    root mean square (optional) -> V page.  Key and value heads may have different sizes: the
-//                    cache's head size is the larger one, the rest of a row is zeros.  With v_share = n, n neighbouring key
-//                    heads read one value head (the product holds Hkv / n of them) and each caches a copy of it.
+//   qkv_prepare      per token (qkv_prepare.h): a bias on q, k and v (optional); q and k heads -> RMS norm (optional, with or
+//                    without a weight, before or after the rotation), rotation of the first `rot` entries (pairs i, i + rot/2,
+//                    or neighbours 2i, 2i + 1; optionally times a constant); q times a number per head (optional) -> q_out,
+//                    padded to the cache's head size; k -> K page; v heads -> divided by their root mean square (optional) -> V
+//                    page.  Key and value heads may have different sizes: the cache's head size is the larger one, the rest
+//                    of a row is zeros.  With v_share = n, n neighbouring key heads read one value head (the product holds
+//                    Hkv / n of them) and each caches a copy of it.
 //   diff_combine     two softmax maps per head over the same values: o = a1 - lambda * a2, o / rms(o) * out_scale
 //   head_gate        y[t, h, :] *= sigmoid(g[t, h])
 //   rms_pair_mean    out = ca * a / rms(a) * wa + cb * b / rms(b) * wb   (two branch outputs, each normalised over the width)
@@ -15,79 +16,87 @@
 //   act_rows         out[t, :] = act(x[t, c0 : c0 + n])  (a slice of a product's rows made dense, tanh or identity)
 // Norm statistics, angles, the rotation and the per-head factors are 32-bit; results are rounded once.
 #include "common.cuh"
+#include "qkv_prepare.h"
 
 constexpr int QP_BLOCK = 256;
 constexpr int QP_WARPS = QP_BLOCK / 32;
-constexpr int QP_UNITS = 16;     // units of one token a CTA takes, two a warp: the token's angles are made once for all of them
+constexpr int QP_UNITS = 16;     // units of one token a CTA takes in steps of few tokens: the token's angles are made once for all of them
 constexpr int QP_MAX_D = 512;
 
-// A CTA per (token, group of QP_UNITS units), a warp per unit; units: Hq query heads, then Hkv key heads, then Hkv value
-// heads; PER entries of a head a lane (the cache's head size is at most 32 * PER).
-// proj: [T, ld] with columns [q: Hq*D | k: Hkv*D | v: Hkv*Dv | ...].  inv_freq: [rot/2] float32 (angle = pos * inv_freq[i]).
+// cos and sin of a pair's angle at a position.  The angle is made in turns, pos * turns with turns = hi + lo: the product with
+// hi is exact as a float and its rounding error, whole turns leave exactly, so what reaches sincospif is right to 32-bit at any
+// position (pos * angle rounded to a float would lose a digit per decade of positions).
+__device__ __forceinline__ void rotation_angle(float pos, float hi, float lo, float mult, float* sn, float* cs) {
+    const float whole = pos * hi, err = fmaf(pos, hi, -whole);
+    sincospif(2.f * ((whole - rintf(whole)) + fmaf(pos, lo, err)), sn, cs);
+    *sn *= mult;
+    *cs *= mult;
+}
+
+// A CTA per (token, group of units), a warp per unit; units: Hq query heads, then Hkv key heads, then Hkv value heads; PER
+// entries of a head a lane (the cache's head size is at most 32 * PER).
 template <typename TA, int PER>
-__global__ void __launch_bounds__(QP_BLOCK) qkv_prepare_kernel(
-    const TA* __restrict__ proj, int64_t ld, int n_tokens, int Hq, int Hkv, int D, int Dv, int Dc, const float* __restrict__ q_norm_w,
-    const float* __restrict__ k_norm_w, float eps, int v_norm, const float* __restrict__ inv_freq, int rot, int pairing, int v_share,
-    const float* __restrict__ head_mult, const int* __restrict__ positions, const int* __restrict__ seq_of_token,
-    const int* __restrict__ block_table, int bt_stride, int n_seqs, TA* __restrict__ q_out, int64_t q_ld, TA* __restrict__ k_cache,
-    TA* __restrict__ v_cache, int page_size, int num_pages, int* status) {
+__global__ void __launch_bounds__(QP_BLOCK) qkv_prepare_kernel(const ImpQkvPrepare p, int units_per_cta, int* status) {
     pdl_wait();
     pdl_launch_dependents();
     __shared__ float rot_s[QP_WARPS][32 * PER];
     __shared__ float cos_s[16 * PER], sin_s[16 * PER];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int Hq = p.Hq, Hkv = p.Hkv, D = p.D, Dc = p.Dc, rot = p.rot;
     const int units = Hq + 2 * Hkv;
     const int64_t t = blockIdx.x;
-    const int seq = seq_of_token[t], pos = positions[t];
-    if (seq < 0 || seq >= n_seqs || pos < 0 || pos / page_size >= bt_stride) {
-        if (threadIdx.x == 0 && blockIdx.y == 0) imp_report(status, seq < 0 || seq >= n_seqs ? IMP_BAD_SEQUENCE : IMP_BAD_POSITION);
+    const int seq = p.seq_of_token[t], pos = p.positions[t];
+    if (seq < 0 || seq >= p.n_seqs || pos < 0 || pos / p.page_size >= p.bt_stride) {
+        if (threadIdx.x == 0 && blockIdx.y == 0) imp_report(status, seq < 0 || seq >= p.n_seqs ? IMP_BAD_SEQUENCE : IMP_BAD_POSITION);
         return;
     }
     const int half = rot / 2;
-    const int u_begin = blockIdx.y * QP_UNITS, u_end = min(units, u_begin + QP_UNITS);
+    const int u_begin = blockIdx.y * units_per_cta, u_end = min(units, u_begin + units_per_cta);
     if (rot > 0 && u_begin < Hq + Hkv) {     // a group of value heads rotates nothing
-        for (int i = threadIdx.x; i < half; i += QP_BLOCK) sincosf((float)pos * inv_freq[i], &sin_s[i], &cos_s[i]);
+        for (int i = threadIdx.x; i < half; i += QP_BLOCK) rotation_angle((float)pos, p.turns[i], p.turns[half + i], p.rot_mult, &sin_s[i], &cos_s[i]);
     }
     __syncthreads();
-    const int page = block_table[(int64_t)seq * bt_stride + pos / page_size];
+    const int page = p.block_table[(int64_t)seq * p.bt_stride + pos / p.page_size];
     for (int unit = u_begin + warp; unit < u_end; unit += QP_WARPS) {
         const bool is_q = unit < Hq, is_v = unit >= Hq + Hkv;
         const int head = is_q ? unit : is_v ? unit - Hq - Hkv : unit - Hq;
-        const int n = is_v ? Dv : D;
-        const TA* src = proj + t * ld + (is_q ? (int64_t)head * D : is_v ? (int64_t)Hq * D + (int64_t)Hkv * D + (int64_t)(head / v_share) * Dv
-                                                                         : (int64_t)Hq * D + (int64_t)head * D);
+        const int n = is_v ? p.Dv : D;
+        const int64_t col = is_q ? (int64_t)head * D : is_v ? (int64_t)(Hq + Hkv) * D + (int64_t)(head / p.v_share) * p.Dv : (int64_t)(Hq + head) * D;
+        const TA* src = (const TA*)p.proj + t * p.ld + col;
         TA* dst;
         if (is_q) {
-            dst = q_out + t * q_ld + (int64_t)head * Dc;
+            dst = (TA*)p.q_out + t * p.q_ld + (int64_t)head * Dc;
         } else {
-            if (page < 0 || page >= num_pages) {
+            if (page < 0 || page >= p.num_pages) {
                 if (lane == 0) imp_report(status, IMP_BAD_PAGE);
                 continue;
             }
-            TA* cache = is_v ? v_cache : k_cache;
+            TA* cache = (TA*)(is_v ? p.v_cache : p.k_cache);
             if (!cache) continue;
-            dst = cache + (((int64_t)page * Hkv + head) * page_size + pos % page_size) * Dc;   // pages are [page][kv head][slot][entry]
+            dst = cache + (((int64_t)page * Hkv + head) * p.page_size + pos % p.page_size) * Dc;   // pages are [page][kv head][slot][entry]
         }
-        float x[PER], ss = 0.f;
+        float x[PER];
 #pragma unroll
         for (int i = 0; i < PER; ++i) {
             const int d = lane + i * 32;
-            x[i] = d < n ? to_float(src[d]) : 0.f;
-            ss = fmaf(x[i], x[i], ss);
+            x[i] = d < n ? to_float(src[d]) + (p.bias ? p.bias[col + d] : 0.f) : 0.f;
         }
-        const float* nw = is_q ? q_norm_w : is_v ? nullptr : k_norm_w;
-        const bool normed = is_v ? v_norm != 0 : nw != nullptr;
-        if (normed) {
+        const float* nw = is_q ? p.q_norm_w : is_v ? nullptr : p.k_norm_w;
+        auto norm = [&] {
+            float ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < PER; ++i) ss = fmaf(x[i], x[i], ss);     // entries beyond the head are zero
             ss = warp_sum(ss);
-            const float r = rsqrtf(ss / (float)n + eps);
+            const float r = rsqrtf(ss / (float)n + p.eps);
 #pragma unroll
             for (int i = 0; i < PER; ++i) {
                 const int d = lane + i * 32;
                 if (d < n) x[i] = x[i] * r * (nw ? nw[d] : 1.f);
             }
-        }
-        if (!is_v && rot > 0 && pairing == 1) {
-            // neighbours: entry 2i pairs with 2i + 1, which the next lane holds, at angle pos * inv_freq[i]
+        };
+        if (is_v ? p.v_norm != 0 : p.qk_norm == QK_NORM_BEFORE_ROTATION) norm();
+        if (!is_v && rot > 0 && p.pairing == 1) {
+            // neighbours: entry 2i pairs with 2i + 1, which the next lane holds
 #pragma unroll
             for (int i = 0; i < PER; ++i) {
                 const int d = lane + i * 32;
@@ -119,12 +128,119 @@ __global__ void __launch_bounds__(QP_BLOCK) qkv_prepare_kernel(
             }
             __syncwarp();     // the row is written again for the warp's next unit
         }
-        const float mult = (is_q && head_mult) ? head_mult[head] : 1.f;
+        if (!is_v && p.qk_norm == QK_NORM_AFTER_ROTATION) norm();
+        const float mult = (is_q && p.head_mult) ? p.head_mult[head] : 1.f;
 #pragma unroll
         for (int i = 0; i < PER; ++i) {
             const int d = lane + i * 32;
             if (d < Dc) dst[d] = from_float<TA>(d < n ? x[i] * mult : 0.f);
         }
+    }
+}
+
+// The same for 16-bit activations with eight neighbouring entries a lane (16-byte loads and stores; a rotated pair of
+// neighbours is in one lane): LPH lanes a head, 32 / LPH heads a warp at once.  Head sizes that are multiples of 8 up to
+// 8 * LPH, rows that start on 16 bytes, no rotation of halves.
+template <int LPH>
+__global__ void __launch_bounds__(QP_BLOCK) qkv_prepare_vec_kernel(const ImpQkvPrepare p, int units_per_cta, int* status) {
+    pdl_wait();
+    pdl_launch_dependents();
+    using TA = __nv_bfloat16;
+    constexpr int UPW = 32 / LPH;
+    __shared__ __align__(16) float cos_s[4 * LPH], sin_s[4 * LPH];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int sub = lane / LPH, d0 = (lane % LPH) * 8;
+    const int Hq = p.Hq, Hkv = p.Hkv, D = p.D, Dc = p.Dc, rot = p.rot;
+    const int units = Hq + 2 * Hkv;
+    const int64_t t = blockIdx.x;
+    const int seq = p.seq_of_token[t], pos = p.positions[t];
+    if (seq < 0 || seq >= p.n_seqs || pos < 0 || pos / p.page_size >= p.bt_stride) {
+        if (threadIdx.x == 0 && blockIdx.y == 0) imp_report(status, seq < 0 || seq >= p.n_seqs ? IMP_BAD_SEQUENCE : IMP_BAD_POSITION);
+        return;
+    }
+    const int half = rot / 2;
+    const int u_begin = blockIdx.y * units_per_cta, u_end = min(units, u_begin + units_per_cta);
+    if (u_begin < Hq + Hkv) {
+        for (int i = threadIdx.x; i < half; i += QP_BLOCK) rotation_angle((float)pos, p.turns[i], p.turns[half + i], p.rot_mult, &sin_s[i], &cos_s[i]);
+    }
+    __syncthreads();
+    const int page = p.block_table[(int64_t)seq * p.bt_stride + pos / p.page_size];
+    const bool page_ok = page >= 0 && page < p.num_pages;
+    if (!page_ok && threadIdx.x == 0 && u_end > Hq) imp_report(status, IMP_BAD_PAGE);
+    for (int base = u_begin + warp * UPW; base < u_end; base += QP_WARPS * UPW) {   // the same for every lane of a warp
+        const int unit = base + sub;
+        const bool there = unit < u_end;
+        const bool is_q = unit < Hq, is_v = unit >= Hq + Hkv;
+        const int head = is_q ? unit : is_v ? unit - Hq - Hkv : unit - Hq;
+        const int n = is_v ? p.Dv : D;
+        const int64_t col = is_q ? (int64_t)head * D : is_v ? (int64_t)(Hq + Hkv) * D + (int64_t)(head / p.v_share) * p.Dv : (int64_t)(Hq + head) * D;
+        const bool mine = there && d0 < n;
+        float x[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) x[i] = 0.f;
+        if (mine) {
+            const uint4 raw = *reinterpret_cast<const uint4*>((const TA*)p.proj + t * p.ld + col + d0);
+            const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i]));
+                x[2 * i] = f.x, x[2 * i + 1] = f.y;
+            }
+            if (p.bias) {
+                const float4 b0 = *reinterpret_cast<const float4*>(p.bias + col + d0), b1 = *reinterpret_cast<const float4*>(p.bias + col + d0 + 4);
+                x[0] += b0.x, x[1] += b0.y, x[2] += b0.z, x[3] += b0.w;
+                x[4] += b1.x, x[5] += b1.y, x[6] += b1.z, x[7] += b1.w;
+            }
+        }
+        const float* nw = is_q ? p.q_norm_w : is_v ? nullptr : p.k_norm_w;
+        // every lane of the warp takes part in the sums, whichever norms its unit has
+        auto norm = [&](bool wanted) {
+            float ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) ss = fmaf(x[i], x[i], ss);
+#pragma unroll
+            for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            if (!wanted || !mine) return;
+            const float r = rsqrtf(ss / (float)n + p.eps);
+            if (nw) {
+                const float4 a = *reinterpret_cast<const float4*>(nw + d0), b = *reinterpret_cast<const float4*>(nw + d0 + 4);
+                x[0] *= r * a.x, x[1] *= r * a.y, x[2] *= r * a.z, x[3] *= r * a.w;
+                x[4] *= r * b.x, x[5] *= r * b.y, x[6] *= r * b.z, x[7] *= r * b.w;
+            } else {
+#pragma unroll
+                for (int i = 0; i < 8; ++i) x[i] *= r;
+            }
+        };
+        if (p.qk_norm == QK_NORM_BEFORE_ROTATION || p.v_norm) norm(is_v ? p.v_norm != 0 : p.qk_norm == QK_NORM_BEFORE_ROTATION);
+        if (mine && !is_v && d0 < rot) {
+            const float4 cs4 = *reinterpret_cast<const float4*>(&cos_s[d0 >> 1]), sn4 = *reinterpret_cast<const float4*>(&sin_s[d0 >> 1]);
+            const float cs[4] = {cs4.x, cs4.y, cs4.z, cs4.w}, sn[4] = {sn4.x, sn4.y, sn4.z, sn4.w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+                if (d0 + 2 * i < rot) {
+                    const float u = x[2 * i], v = x[2 * i + 1];
+                    x[2 * i] = u * cs[i] - v * sn[i];
+                    x[2 * i + 1] = v * cs[i] + u * sn[i];
+                }
+        }
+        if (p.qk_norm == QK_NORM_AFTER_ROTATION) norm(!is_v);
+        if (!there || d0 >= Dc) continue;
+        TA* dst;
+        if (is_q) {
+            dst = (TA*)p.q_out + t * p.q_ld + (int64_t)head * Dc;
+        } else {
+            TA* cache = (TA*)(is_v ? p.v_cache : p.k_cache);
+            if (!cache || !page_ok) continue;
+            dst = cache + (((int64_t)page * Hkv + head) * p.page_size + pos % p.page_size) * Dc;
+        }
+        const float mult = (is_q && p.head_mult) ? p.head_mult[head] : 1.f;
+        uint32_t o[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const __nv_bfloat162 v = __floats2bfloat162_rn(x[2 * i] * mult, x[2 * i + 1] * mult);
+            o[i] = *reinterpret_cast<const uint32_t*>(&v);
+        }
+        *reinterpret_cast<uint4*>(dst + d0) = make_uint4(o[0], o[1], o[2], o[3]);
     }
 }
 
@@ -165,7 +281,8 @@ __global__ void __launch_bounds__(256) rms_pair_mean_kernel(TA* __restrict__ out
     for (int i = threadIdx.x; i < d; i += blockDim.x) o[i] = from_float<TA>(fmaf(to_float(ar[i]) * ra, wa[i], to_float(br[i]) * rb * wb[i]));
 }
 
-// out[t, f] = the gated activation (GateAct, kinds 0 to 2) over rows [gate | up] (block == 0) or runs of `block` gate entries followed by their up entries.
+// out[t, f] = the gated activation (GateAct, kinds 0 to 2, with its bias in the rows' own order) over rows [gate | up] (block == 0) or
+// runs of `block` gate entries followed by their up entries.
 template <typename T>
 __global__ void gated_act_kernel(T* __restrict__ out, const T* __restrict__ gu, int64_t n_tokens, int F, int block, GateAct act) {
     pdl_wait();
@@ -176,8 +293,8 @@ __global__ void gated_act_kernel(T* __restrict__ out, const T* __restrict__ gu, 
         const int f = (int)(i - t * F);
         const int gi = block ? (f / block) * 2 * block + f % block : f;
         const int ui = block ? gi + block : F + f;
-        const float g = to_float(gu[t * 2 * F + gi]);
-        const float u = to_float(gu[t * 2 * F + ui]);
+        const float g = to_float(gu[t * 2 * F + gi]) + (act.bias ? act.bias[gi] : 0.f);
+        const float u = to_float(gu[t * 2 * F + ui]) + (act.bias ? act.bias[ui] : 0.f);
         out[i] = from_float<T>(gated_f(g, u, act));
     }
 }
@@ -282,48 +399,49 @@ __global__ void diff_combine_vec_kernel(TA* __restrict__ y, const TA* __restrict
     }
 }
 
-IMP_API int imp_qkv_prepare_ex(const void* proj, int64_t ld, int n_tokens, int Hq, int Hkv, int D, int Dv, int Dc, const float* q_norm_w,
-                               const float* k_norm_w, float eps, int v_norm, const float* inv_freq, int rot, int pairing, int v_share,
-                               const float* head_mult, const int* positions, const int* seq_of_token, const int* block_table, int bt_stride,
-                               int n_seqs, void* q_out, int64_t q_ld, void* k_cache, void* v_cache, int page_size, int num_pages, int act_dtype,
-                               int* status, void* stream) {
-    if (n_tokens == 0) return 0;
-    IMP_CHECK_ARG(proj && positions && seq_of_token && block_table && q_out, "imp_qkv_prepare: null pointer");
-    IMP_CHECK_ARG(Hq > 0 && Hkv > 0 && D > 0 && Dv > 0 && Dc >= D && Dc >= Dv && Dc <= QP_MAX_D,
-                  "imp_qkv_prepare: head sizes %d / %d must fit the cache's %d (at most %d)", D, Dv, Dc, QP_MAX_D);
-    IMP_CHECK_ARG(rot >= 0 && rot % 2 == 0 && rot <= D && (rot == 0 || inv_freq), "imp_qkv_prepare: the rotated part must be even and within the head");
-    IMP_CHECK_ARG((q_norm_w == nullptr) == (k_norm_w == nullptr), "imp_qkv_prepare: q and k are normalised together or not at all");
-    IMP_CHECK_ARG((pairing == 0 || pairing == 1) && v_share > 0 && Hkv % v_share == 0, "imp_qkv_prepare: pairing is 0 (halves) or 1 (neighbours); v_share divides the key heads");
-    IMP_CHECK_ARG(ld >= (int64_t)(Hq + Hkv) * D + (int64_t)(Hkv / v_share) * Dv && q_ld >= (int64_t)Hq * Dc, "imp_qkv_prepare: rows too short");
-    IMP_CHECK_ARG(page_size > 0 && num_pages > 0, "imp_qkv_prepare: bad cache geometry");
+IMP_API int imp_qkv_prepare(const ImpQkvPrepare* args, int* status, void* stream) {
+    IMP_CHECK_ARG(args, "imp_qkv_prepare: null pointer");
+    const ImpQkvPrepare& p = *args;
+    if (p.n_tokens == 0) return 0;
+    IMP_CHECK_ARG(p.proj && p.positions && p.seq_of_token && p.block_table && p.q_out, "imp_qkv_prepare: null pointer");
+    IMP_CHECK_ARG(p.Hq > 0 && p.Hkv > 0 && p.D > 0 && p.Dv > 0 && p.Dc >= p.D && p.Dc >= p.Dv && p.Dc <= QP_MAX_D,
+                  "imp_qkv_prepare: head sizes %d / %d must fit the cache's %d (at most %d)", p.D, p.Dv, p.Dc, QP_MAX_D);
+    IMP_CHECK_ARG(p.rot >= 0 && p.rot % 2 == 0 && p.rot <= p.D && (p.rot == 0 || p.turns), "imp_qkv_prepare: the rotated part must be even and within the head");
+    IMP_CHECK_ARG(p.qk_norm >= QK_NORM_NONE && p.qk_norm <= QK_NORM_AFTER_ROTATION && (p.q_norm_w == nullptr) == (p.k_norm_w == nullptr),
+                  "imp_qkv_prepare: q and k are normalised alike");
+    IMP_CHECK_ARG((p.pairing == 0 || p.pairing == 1) && p.v_share > 0 && p.Hkv % p.v_share == 0,
+                  "imp_qkv_prepare: pairing is 0 (halves) or 1 (neighbours); v_share divides the key heads");
+    IMP_CHECK_ARG(p.ld >= (int64_t)(p.Hq + p.Hkv) * p.D + (int64_t)(p.Hkv / p.v_share) * p.Dv && p.q_ld >= (int64_t)p.Hq * p.Dc, "imp_qkv_prepare: rows too short");
+    IMP_CHECK_ARG(p.page_size > 0 && p.num_pages > 0, "imp_qkv_prepare: bad cache geometry");
     cudaStream_t s = (cudaStream_t)stream;
-    const dim3 grid((unsigned)n_tokens, (unsigned)((Hq + 2 * Hkv + QP_UNITS - 1) / QP_UNITS));
-#define QP_LAUNCH(TA, PER)                                                                                                                    \
-    imp_launch(qkv_prepare_kernel<TA, PER>, grid, dim3(QP_BLOCK), 0, s, (const TA*)proj, ld, n_tokens, Hq, Hkv, D, Dv, Dc, q_norm_w, k_norm_w, eps, \
-               v_norm, inv_freq, rot, pairing, v_share, head_mult, positions, seq_of_token, block_table, bt_stride, n_seqs, (TA*)q_out, q_ld, (TA*)k_cache,     \
-               (TA*)v_cache, page_size, num_pages, status)
-#define QP_LAUNCH_PER(TA)                       \
-    do {                                        \
-        if (Dc <= 64) QP_LAUNCH(TA, 2);         \
-        else if (Dc <= 128) QP_LAUNCH(TA, 4);   \
-        else if (Dc <= 256) QP_LAUNCH(TA, 8);   \
-        else QP_LAUNCH(TA, 16);                 \
+    const int units = p.Hq + 2 * p.Hkv;
+    bool vec = p.act_dtype != IMP_F32 && p.D % 8 == 0 && p.Dv % 8 == 0 && p.Dc % 8 == 0 && p.Dc <= 256 && p.ld % 8 == 0 && p.q_ld % 8 == 0 &&
+               (p.rot == 0 || p.pairing == 1);
+    for (const void* q : {p.proj, (const void*)p.bias, (const void*)p.q_norm_w, (const void*)p.k_norm_w, (const void*)p.q_out, (const void*)p.k_cache,
+                          (const void*)p.v_cache})
+        vec = vec && (uintptr_t)q % 16 == 0;
+    // few tokens: a token's units spread over several CTAs; many: one CTA makes the token's angles once for all of them
+    const int per_cta = vec && p.n_tokens >= 2 * imp_sm_count() ? units : QP_UNITS;
+    const dim3 grid((unsigned)p.n_tokens, (unsigned)((units + per_cta - 1) / per_cta));
+    if (vec) {
+        if (p.Dc <= 64) imp_launch(qkv_prepare_vec_kernel<8>, grid, dim3(QP_BLOCK), 0, s, p, per_cta, status);
+        else if (p.Dc <= 128) imp_launch(qkv_prepare_vec_kernel<16>, grid, dim3(QP_BLOCK), 0, s, p, per_cta, status);
+        else imp_launch(qkv_prepare_vec_kernel<32>, grid, dim3(QP_BLOCK), 0, s, p, per_cta, status);
+        IMP_RETURN_LAUNCH();
+    }
+#define QP_LAUNCH(TA, PER) imp_launch(qkv_prepare_kernel<TA, PER>, grid, dim3(QP_BLOCK), 0, s, p, per_cta, status)
+#define QP_LAUNCH_PER(TA)                         \
+    do {                                          \
+        if (p.Dc <= 64) QP_LAUNCH(TA, 2);         \
+        else if (p.Dc <= 128) QP_LAUNCH(TA, 4);   \
+        else if (p.Dc <= 256) QP_LAUNCH(TA, 8);   \
+        else QP_LAUNCH(TA, 16);                   \
     } while (0)
-    if (act_dtype == IMP_F32) QP_LAUNCH_PER(float);
+    if (p.act_dtype == IMP_F32) QP_LAUNCH_PER(float);
     else QP_LAUNCH_PER(__nv_bfloat16);
 #undef QP_LAUNCH_PER
 #undef QP_LAUNCH
     IMP_RETURN_LAUNCH();
-}
-
-IMP_API int imp_qkv_prepare(const void* proj, int64_t ld, int n_tokens, int Hq, int Hkv, int D, int Dv, int Dc, const float* q_norm_w,
-                            const float* k_norm_w, float eps, int v_norm, const float* inv_freq, int rot, const float* head_mult,
-                            const int* positions, const int* seq_of_token, const int* block_table, int bt_stride, int n_seqs, void* q_out,
-                            int64_t q_ld, void* k_cache, void* v_cache, int page_size, int num_pages, int act_dtype, int* status,
-                            void* stream) {
-    return imp_qkv_prepare_ex(proj, ld, n_tokens, Hq, Hkv, D, Dv, Dc, q_norm_w, k_norm_w, eps, v_norm, inv_freq, rot, 0, 1, head_mult, positions,
-                              seq_of_token, block_table, bt_stride, n_seqs, q_out, q_ld, k_cache, v_cache, page_size, num_pages, act_dtype, status,
-                              stream);
 }
 
 // y [T, G * R * Dv] dense; attn rows `ld` apart; lambda: one float32 on the device.
@@ -376,15 +494,16 @@ IMP_API int imp_rms_pair_mean(void* out, const void* a, const float* wa, float c
     IMP_RETURN_LAUNCH();
 }
 
-IMP_API int imp_gated_act(void* out, const void* gate_up, int n_tokens, int F, int block, int act, float limit, int dtype, void* stream) {
+IMP_API int imp_gated_act(void* out, const void* gate_up, int n_tokens, int F, int block, int act, float limit, const float* bias, int dtype,
+                          void* stream) {
     if (n_tokens == 0 || F == 0) return 0;
     IMP_CHECK_ARG(out && gate_up && n_tokens > 0 && F > 0 && block >= 0 && (block == 0 || F % block == 0) && act >= ACT_SILU && act <= ACT_CLIPPED,
                   "imp_gated_act: bad argument");
     cudaStream_t s = (cudaStream_t)stream;
     const int64_t total = (int64_t)n_tokens * F;
     const dim3 grid((unsigned)std::min<int64_t>((total + 255) / 256, 65535));
-    if (dtype == IMP_F32) imp_launch(gated_act_kernel<float>, grid, dim3(256), 0, s, (float*)out, (const float*)gate_up, (int64_t)n_tokens, F, block, GateAct(act, limit));
-    else imp_launch(gated_act_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, (int64_t)n_tokens, F, block, GateAct(act, limit));
+    if (dtype == IMP_F32) imp_launch(gated_act_kernel<float>, grid, dim3(256), 0, s, (float*)out, (const float*)gate_up, (int64_t)n_tokens, F, block, GateAct(act, limit, bias));
+    else imp_launch(gated_act_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, (int64_t)n_tokens, F, block, GateAct(act, limit, bias));
     IMP_RETURN_LAUNCH();
 }
 

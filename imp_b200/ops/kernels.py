@@ -115,16 +115,17 @@ def linear_swiglu(out: torch.Tensor, x: torch.Tensor, w_interleaved: torch.Tenso
 
 
 def linear_gated(out: torch.Tensor, x: torch.Tensor, w_interleaved: torch.Tensor, activation: str = "silu",
-                 limit: float = 0.0) -> torch.Tensor:
+                 limit: float = 0.0, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[M, F] = act(x Wg^T) * (x Wu^T), act "silu" or "gelu_tanh", or "clipped": g sigmoid(1.702 g) (u + 1) with
-    g = min(x Wg^T, limit) and u = x Wu^T held within +-limit; with the activation in the product's epilogue
+    g = min(x Wg^T, limit) and u = x Wu^T held within +-limit; `bias` (float32, one number per row of w_interleaved) is
+    added to the products first; with bias and activation in the product's epilogue
     where the library has such a kernel for the shape (csrc/host/linear.cpp `linear_gated`)."""
     _need_cuda(out, x, w_interleaved)
     if x.shape[0] == 0:
         return out
     act = {"silu": 0, "gelu_tanh": 1, "clipped": 2}[activation]
     o, a, w = _view(out), _view(x), _view(w_interleaved)
-    _op_check(L.load().imp_op_linear_gated(ctypes.byref(o), ctypes.byref(a), ctypes.byref(w), act, float(limit), _stream(), None), "linear_gated")
+    _op_check(L.load().imp_op_linear_gated(ctypes.byref(o), ctypes.byref(a), ctypes.byref(w), act, float(limit), _ptr(bias), _stream(), None), "linear_gated")
     return out
 
 

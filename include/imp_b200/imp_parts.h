@@ -19,7 +19,8 @@
  *   {local name: {"shape": [..], "role": "matrix"|"norm"|"vector"|"int_table",
  *                 "init": "normal"|"one_plus_normal"|"zeros"|"arange_mod", "optional": bool}}
  * Cache spec JSON (what a mixer asks of the cache):
- *   null | {"kind": "paged", "num_kv_heads": int, "head_dim": int, "window": int}
+ *   null | {"kind": "paged", "num_kv_heads": int, "head_dim": int, "window": int}   (window 0: every token, W > 0: the last W
+ *          positions, -C < 0: the chunk of C positions that a query is in)
  *        | {"kind": "state", "tensors": [{"name": str, "shape": [..], "dtype": "float32"|"bfloat16"|"int32"}]}
  * Block slots JSON: [{"name": slot, "category": "mixer"|"feed_forward"|"norm"}, ...] (at most one mixer).
  */

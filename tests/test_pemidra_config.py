@@ -96,7 +96,7 @@ def test_options_that_config_leaves_out_do_not_exist():
 def test_a_pair_owns_a_paged_cache_and_a_state_the_others_a_state():
     plan = plan_for(config_from_dict(CFG))
     left = mixer_cache_spec("gated_head_attention", plan.layers[0].parts["left"].params)
-    assert left == {"kind": "paged", "num_kv_heads": 1, "head_dim": 32, "window": 0}       # keys of 24 and values of 16 in rows of 32
+    assert left == {"kind": "paged", "num_kv_heads": 1, "head_dim": 32, "window": -10}     # keys of 24 and values of 16 in rows of 32, a chunk of 10
     right = mixer_cache_spec("channel_delta_rule", plan.layers[0].parts["right"].params)
     assert [t["name"] for t in right["tensors"]] == ["S", "conv"] and right["tensors"][1]["shape"] == [2, 2 * 24 + 80]
     ret = mixer_cache_spec("retention", plan.layers[1].mixer.params)
