@@ -31,6 +31,7 @@ Other runs, each printing its own JSON line:
     python bench.py --arch pemidra [--layers N] [--batch B]    Pemidra beside Kazedra and Qwen3 at equal sizes
     python bench.py --arch nizorax [--layers N] [--batch B]    Nizorax beside Pemidra, Kuzipel and Qwen3 at equal sizes
     python bench.py --arch nomanex [--layers N] [--batch B]    Nomanex beside Kuzipel, Pemidra and Qwen3 at equal sizes
+    python bench.py --arch ribovik [--layers N] [--batch B]    Ribovik beside Nizorax, Pemidra and Qwen3 at equal sizes
     python bench.py --workload 14b                        8 prompts of 8,192 tokens in 2,048-token portions, 512 tokens at T=0.7
 (`--context` may exceed the configured 4096: the cache and the position table grow with it.)
 """
@@ -790,8 +791,21 @@ def nomanex_config(width, heads, kv_heads, ff, layers, vocab):
             "embedding": {"bigram": {"buckets": 65536, "mul_prev": 40503, "mul_cur": 30011}}, "layers": lays, "max_positions": 8192}
 
 
+def ribovik_config(width, heads, kv_heads, ff, layers, vocab):
+    """Layers cycle through the dense feed-forward of the models beside it, routed experts (16 and two identities, two chosen, a
+    shared one: together the dense inner size, Nizorax's geometry) and the dense one again; attention with heads of 128, the whole of each head
+    rotated with the frequencies of YaRN, chunks of 1,024 positions (Pemidra's geometry)."""
+    attn = {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024},
+            "rot": {"base": 1e6, "dims": 128, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff // 3, "limit": 7.0}, "router": {"experts": 16, "identity": 2, "top": 2},
+           "shared": {"ff": ff // 3, "limit": 7.0}}
+    lays = [{"type": "attention", "mixer": attn, "mlp": moe if i % 3 == 1 else dense} for i in range(layers)]
+    return {"architecture": "Ribovik", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": lays, "max_positions": 8192}
+
+
 def run_arch(args):
-    """Prefill and decode of Kazedra, Kuzipel, Pemidra, Nizorax or Nomanex beside the models the engine already had at equal sizes (random weights): a
+    """Prefill and decode of Kazedra, Kuzipel, Pemidra, Nizorax, Nomanex or Ribovik beside the models the engine already had at equal sizes (random weights): a
     2,048-token prompt whole and in 512-token portions, and decode steps of `--batch` sequences at context 2,048, device
     time between CUDA events."""
     if args.arch == "kuzipel":
@@ -802,6 +816,8 @@ def run_arch(args):
         return run_arch_beside(args, "nizorax", nizorax_config, beside={"pemidra": pemidra_config, "kuzipel": kuzipel_config})
     if args.arch == "nomanex":
         return run_arch_beside(args, "nomanex", nomanex_config, beside={"kuzipel": kuzipel_config, "pemidra": pemidra_config})
+    if args.arch == "ribovik":
+        return run_arch_beside(args, "ribovik", ribovik_config, beside={"nizorax": nizorax_config, "pemidra": pemidra_config})
     peaks, peak_src = read_peaks()
     layers, vocab, B = args.layers or 4, 32768, args.batch
     if args.only in ("prefill", "decode"):
@@ -947,7 +963,7 @@ def main():
     ap.add_argument("--only", default="", choices=["", "decode", "prefill", "timeline", "mixed"],
                     help="run one phase only and print its timing (for profiling small cases)")
     ap.add_argument("--workload", default="", choices=["", "0.6b", "14b"], help="one of the two other workloads of the baseline record")
-    ap.add_argument("--arch", default="", choices=["", "kazedra", "kuzipel", "pemidra", "nizorax", "nomanex"],
+    ap.add_argument("--arch", default="", choices=["", "kazedra", "kuzipel", "pemidra", "nizorax", "nomanex", "ribovik"],
                     help="prefill and decode of this architecture beside the Qwen3 decoder at equal sizes (not the default workload)")
     ap.add_argument("--shape", default="8b", choices=["1b", "8b"], help="with --arch and --only: which of the shapes")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="with --workload: the compute type")

@@ -594,10 +594,11 @@ struct RoutedExperts : FeedForward {
         if (tensor_cores && !st.decode_only() && capturing == cudaStreamCaptureStatusNone && dense_work > 0 &&
             (double)P / (double)R * (double)F * (double)d >= dense_work) {
             std::vector<int> hseg((size_t)E + 1);
-            Tensor xs = rt.empty(P, d);
-            check_launch(imp_gather_rows(xs.data, x.data, x.stride0, row_token, (int)P, (int)d, dt, rt.stream), "gather_rows");
             IMP_CUDA(cudaMemcpyAsync(hseg.data(), seg, hseg.size() * 4, cudaMemcpyDeviceToHost, rt.stream));
             IMP_CUDA(cudaStreamSynchronize(rt.stream));
+            const int64_t listed = hseg[(size_t)E];   // choices that fell on identity experts are not in the list
+            Tensor xs = rt.empty(P, d);
+            check_launch(imp_gather_rows(xs.data, x.data, x.stride0, row_token, (int)listed, (int)d, dt, rt.stream), "gather_rows");
             const size_t el = elem_size(rt.dtype);
             for (int64_t e = 0; e < E; ++e) {
                 const int64_t a0 = hseg[(size_t)e], n = hseg[(size_t)e + 1] - a0;

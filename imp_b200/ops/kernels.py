@@ -216,6 +216,33 @@ def add_normed_layernorm(h: Optional[torch.Tensor], branch: torch.Tensor, branch
     return out
 
 
+class BranchTerm(ctypes.Structure):
+    """One summand of a branch (csrc/branch_terms.h): dense, the unsummed parts of a product, or routed rows."""
+    _fields_ = [("t", ctypes.c_void_p), ("parts", ctypes.c_void_p), ("n_splits", ctypes.c_int), ("y", ctypes.c_void_p),
+                ("pair_row", ctypes.c_void_p), ("wts", ctypes.c_void_p), ("top", ctypes.c_int), ("input", ctypes.c_void_p)]
+
+
+def branch_term(t: Optional[torch.Tensor] = None, parts: Optional[torch.Tensor] = None, y: Optional[torch.Tensor] = None,
+                pair_row: Optional[torch.Tensor] = None, wts: Optional[torch.Tensor] = None,
+                input: Optional[torch.Tensor] = None) -> BranchTerm:
+    """t [T, d]; or parts float32 [splits, T, d]; or y [rows, d] with pair_row int32 and wts float32 [T, top] (a negative
+    place: row t of `input`, or of the stream where input is None); or nothing."""
+    _need_cuda(t, parts, y, pair_row, wts, input)
+    return BranchTerm(_ptr(t), _ptr(parts), parts.shape[0] if parts is not None else 0, _ptr(y), _ptr(pair_row), _ptr(wts),
+                      pair_row.shape[1] if pair_row is not None else 0, _ptr(input))
+
+
+def add_rms_branch(h: torch.Tensor, first: BranchTerm, second: BranchTerm, bias: Optional[torch.Tensor], weight: torch.Tensor,
+                   eps: float, out: torch.Tensor) -> torch.Tensor:
+    """h += rmsnorm(first + second + bias; weight); out = h in its own type."""
+    _need_cuda(h, bias, weight, out)
+    n, d = h.shape
+    assert h.dtype == torch.float32 and h.is_contiguous() and out.is_contiguous() and out.shape == h.shape and weight.numel() == d
+    L.check(L.load().imp_add_rms_branch(_ptr(h), ctypes.addressof(first), ctypes.addressof(second), _ptr(bias), _ptr(weight), _ptr(out), n, d,
+                                        float(eps), _dt(out), _dt(weight), _stream()), "add_rms_branch")
+    return out
+
+
 def rmsnorm_rows(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float,
                  weight_offset: float = 0.0) -> torch.Tensor:
     """Row-wise RMSNorm of a 2-D tensor whose rows may be strided."""

@@ -123,11 +123,30 @@ def test_window_never_frees_what_a_portion_still_reads():
     m.check_invariants()
 
 
+def test_chunk_group_gives_a_chunk_back_when_the_next_begins():
+    m = CacheManager([PagedKVSpec(1, 16, -10)], page_size=4, num_pages=5)      # chunks of 10 positions, pages of 4
+    m.add_request("a")
+    m.reserve("a", 19)
+    m.commit("a", 19)      # the next query, at 19, is in the chunk 10..19: pages 0 and 1 (0..7) are dead, page 2 (8..11) is not
+    assert m.block_table(0, "a")[:2] == [-1, -1] and all(p >= 0 for p in m.block_table(0, "a")[2:])
+    m.reserve("a", 20)
+    m.commit("a", 20)      # the next query begins a chunk: nothing before it is seen again (page 5 starts with it)
+    assert m.block_table(0, "a") == [-1] * 5 and m.free_pages() == 5
+    for n in range(21, 200):
+        m.reserve("a", n)
+        m.commit("a", n)
+        m.check_invariants()
+        first = n - n % 10
+        assert [i for i, p in enumerate(m.block_table(0, "a")) if p >= 0] == list(range(first // 4, (n + 3) // 4))
+    m.release("a")
+    assert m.free_pages() == 5
+
+
 @settings(max_examples=60, deadline=None)
 @given(st.integers(0, 2 ** 31), st.integers(1, 7), st.integers(3, 40))
 def test_random_orders_keep_invariants(seed, page_size, num_pages):
     rng = random.Random(seed)
-    specs = [FULL, PagedKVSpec(2, 16, rng.randint(1, 12)), STATE, FULL]
+    specs = [FULL, PagedKVSpec(2, 16, rng.randint(1, 12)), STATE, FULL, PagedKVSpec(2, 16, -rng.randint(1, 12))]
     m = CacheManager(specs, page_size, num_pages, num_state_slots=3)
     live = {}
     next_id = 0

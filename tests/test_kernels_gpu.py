@@ -229,6 +229,70 @@ def test_linear_gated_fused(K, M, F, K_, activation):
     close(out, a * u, torch.bfloat16)
 
 
+@pytest.mark.parametrize("M", [1, 5, 11, 16, 40, 100, 130, 300, 1100])
+@pytest.mark.parametrize("F,K_", [(8, 64), (200, 96), (1536, 512), (24, 100), (776, 72)])
+@pytest.mark.parametrize("activation", ["silu", "clipped"])
+def test_linear_gated_with_a_bias(K, M, F, K_, activation):
+    """A bias in front of the activation, in the product's epilogue, over the row counts that choose each of its kernels."""
+    x = rnd(M, K_, dtype=torch.bfloat16, seed=33).to(DEV)
+    wg = rnd(F, K_, dtype=torch.bfloat16, seed=34, scale=0.3).to(DEV)
+    wu = rnd(F, K_, dtype=torch.bfloat16, seed=35, scale=0.3).to(DEV)
+    bg, bu = rnd(F, dtype=torch.float32, seed=36, scale=2.0), rnd(F, dtype=torch.float32, seed=37, scale=2.0)
+    w = K.interleave_gate_up(wg, wu)
+    bias = torch.stack([bg.view(-1, 8), bu.view(-1, 8)], dim=1).reshape(-1).to(DEV)
+    out = K.linear_gated(torch.full((M, F), float("nan"), dtype=torch.bfloat16, device=DEV), x, w, activation, limit=1.3, bias=bias)
+    g = x.double().cpu() @ wg.double().cpu().T + bg.double()
+    u = x.double().cpu() @ wu.double().cpu().T + bu.double()
+    if activation == "silu":
+        a = g * torch.sigmoid(g)
+    else:
+        g, u = torch.clamp(g, max=1.3), torch.clamp(u, -1.3, 1.3) + 1
+        a = g * torch.sigmoid(1.702 * g)
+    close(out, a * u, torch.bfloat16)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("n, d", [(1, 72), (3, 5), (9, 70), (8, 1024), (70, 2048), (5, 4096), (200, 4096), (6, 8192), (3, 10000)])
+def test_rms_norm_of_a_branch_in_every_form(K, dtype, n, d):
+    """Dense, in unsummed parts, and as routed rows with identity choices, alone and beside a second summand, with and without a bias."""
+    w = (1 + 0.3 * rnd(d, seed=1)).to(dtype).to(DEV)
+    bias = rnd(d, seed=2).float().to(DEV)
+    dense = rnd(n, d, seed=3).to(dtype).to(DEV)
+    parts = rnd(5, n, d, seed=4).float().to(DEV)
+    rows = rnd(2 * n + 1, d, seed=5).to(dtype).to(DEV)
+    other = rnd(n, d, seed=6).to(dtype).to(DEV)
+    g = torch.Generator().manual_seed(7)
+    place = torch.randint(-1, 2 * n + 1, (n, 3), generator=g).int()
+    place[0, 1] = -1
+    wts = torch.rand(n, 3, generator=g).float()
+    h0 = 2 * rnd(n, d, seed=8).float()
+    D = lambda t: t.double().cpu()
+
+    def routed(own):
+        out = torch.zeros(n, d, dtype=torch.float64)
+        for t in range(n):
+            for k in range(3):
+                r = int(place[t, k])
+                out[t] += wts[t, k].double() * (D(rows)[r] if r >= 0 else own[t])
+        return out
+
+    pr, ww = place.to(DEV), wts.to(DEV)
+    forms = {"dense": (K.branch_term(dense), D(dense)), "parts": (K.branch_term(parts=parts), D(parts).sum(0)),
+             "routed, the stream": (K.branch_term(y=rows, pair_row=pr, wts=ww), routed(h0.double())),
+             "routed, an input": (K.branch_term(y=rows, pair_row=pr, wts=ww, input=other), routed(D(other)))}
+    for name, (term, value) in forms.items():
+        for second, more in ((None, 0.0), (dense, D(dense)), (parts, D(parts).sum(0))):
+            for b in (None, bias):
+                h = h0.clone().to(DEV)
+                out = torch.full((n, d), float("nan"), dtype=dtype, device=DEV)
+                t2 = K.branch_term() if second is None else K.branch_term(parts=second) if second.dim() == 3 else K.branch_term(second)
+                K.add_rms_branch(h, term, t2, b, w, 1e-3, out)
+                v = value + more + (D(bias) if b is not None else 0.0)
+                want = h0.double() + v / torch.sqrt((v * v).mean(-1, keepdim=True) + 1e-3) * D(w)
+                close(h, want, torch.float32)
+                close(out, want, dtype)
+
+
 @pytest.mark.parametrize("M", [1, 5, 16, 40, 100, 130, 300, 1100])
 @pytest.mark.parametrize("N,K_", [(8, 64), (264, 96), (1536, 4096), (24, 100)])
 @pytest.mark.parametrize("dtype", [torch.bfloat16, torch.float32])
