@@ -21,8 +21,9 @@ namespace {
 constexpr int BN_THREADS = 128, BN_MAX_C = 8, BN_ROW_THREADS = 256;
 
 
-// NV float4 a thread; CLUSTER: gridDim.x / C rows, a cluster of C CTAs each; else a CTA a row.
-template <typename TA, typename TW, int NV, bool CLUSTER>
+// NV float4 a thread; CLUSTER: gridDim.x / C rows, a cluster of C CTAs each; else a CTA a row.  DENSE: the branch is one dense
+// tensor (`first.t`), asked for together with the stream.
+template <typename TA, typename TW, int NV, bool CLUSTER, bool DENSE>
 __global__ void __launch_bounds__(CLUSTER ? BN_THREADS : BN_ROW_THREADS)
     add_rms_branch_kernel(float* __restrict__ h, ImpBranchTerm first, ImpBranchTerm second, const float* __restrict__ bias, const TW* __restrict__ w,
                           TA* __restrict__ out, int64_t n_rows, int d, float eps, int C) {
@@ -46,17 +47,25 @@ __global__ void __launch_bounds__(CLUSTER ? BN_THREADS : BN_ROW_THREADS)
         if (c < nv) {
             const float4 v = *reinterpret_cast<const float4*>(hrow + 4 * c);
             x[i][0] = v.x, x[i][1] = v.y, x[i][2] = v.z, x[i][3] = v.w;
+            if (DENSE) {
+                const float4 y = Four<TA>::load((const TA*)first.t + t * d + 4 * c);
+                b[i][0] = y.x, b[i][1] = y.y, b[i][2] = y.z, b[i][3] = y.w;
+            }
             wv[i] = Four<TW>::load(w + 4 * c);
+            if (DENSE && !bias) continue;
             const float4 b0 = bias ? *reinterpret_cast<const float4*>(bias + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
-            b[i][0] = b0.x, b[i][1] = b0.y, b[i][2] = b0.z, b[i][3] = b0.w;
+            if (DENSE) b[i][0] += b0.x, b[i][1] += b0.y, b[i][2] += b0.z, b[i][3] += b0.w;
+            else b[i][0] = b0.x, b[i][1] = b0.y, b[i][2] = b0.z, b[i][3] = b0.w;
         }
     }
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
         const int c = rank * NT + threadIdx.x + i * stride;
         if (c < nv) {
-            add_term<TA, 4>(b[i], first, x[i], t, 4 * c, d, n_rows * d);
-            add_term<TA, 4>(b[i], second, x[i], t, 4 * c, d, n_rows * d);
+            if (!DENSE) {
+                add_term<TA, 4>(b[i], first, x[i], t, 4 * c, d, n_rows * d);
+                add_term<TA, 4>(b[i], second, x[i], t, 4 * c, d, n_rows * d);
+            }
 #pragma unroll
             for (int e = 0; e < 4; ++e) ss = fmaf(b[i][e], b[i][e], ss);
         }
@@ -141,14 +150,17 @@ cudaError_t launch_branch(float* h, const ImpBranchTerm& a, const ImpBranchTerm&
         cfg.attrs = attr;
         cfg.numAttrs = imp_pdl_enabled() ? 2 : 1;
         if (per == 1)
-            return cudaLaunchKernelEx(&cfg, add_rms_branch_kernel<TA, TW, 1, true>, h, a, b, bias, (const TW*)w, (TA*)out, (int64_t)n, d, eps, C);
-        return cudaLaunchKernelEx(&cfg, add_rms_branch_kernel<TA, TW, 2, true>, h, a, b, bias, (const TW*)w, (TA*)out, (int64_t)n, d, eps, C);
+            return cudaLaunchKernelEx(&cfg, add_rms_branch_kernel<TA, TW, 1, true, false>, h, a, b, bias, (const TW*)w, (TA*)out, (int64_t)n, d, eps, C);
+        return cudaLaunchKernelEx(&cfg, add_rms_branch_kernel<TA, TW, 2, true, false>, h, a, b, bias, (const TW*)w, (TA*)out, (int64_t)n, d, eps, C);
     }
     const int per = (nv + BN_ROW_THREADS - 1) / BN_ROW_THREADS;
-#define BN_ROW(NV) \
-    imp_launch(add_rms_branch_kernel<TA, TW, NV, false>, dim3(n), dim3(BN_ROW_THREADS), 0, s, h, a, b, bias, (const TW*)w, (TA*)out, (int64_t)n, d, eps, 1)
+    const bool dense = a.t && !a.parts && !a.y && !b.t && !b.parts && !b.y;
+#define BN_ROW(NV) (dense ? BN_ROW_FORM(NV, true) : BN_ROW_FORM(NV, false))
+#define BN_ROW_FORM(NV, DENSE) \
+    imp_launch(add_rms_branch_kernel<TA, TW, NV, false, DENSE>, dim3(n), dim3(BN_ROW_THREADS), 0, s, h, a, b, bias, (const TW*)w, (TA*)out, (int64_t)n, d, eps, 1)
     return per <= 1 ? BN_ROW(1) : per <= 2 ? BN_ROW(2) : per <= 4 ? BN_ROW(4) : BN_ROW(8);
 #undef BN_ROW
+#undef BN_ROW_FORM
 }
 
 // A CTA per token; four columns a thread where the rows allow it (vec), else one.

@@ -11,7 +11,9 @@
 #include <dlfcn.h>
 #include <sys/stat.h>
 
+#include <algorithm>
 #include <cmath>
+#include <cstdlib>
 #include <map>
 #include <mutex>
 
@@ -245,12 +247,17 @@ static void check_cache(const LayerCache& c, const AttentionGeometry& g) {
     need(c.view.kv_heads == g.hkv && c.view.head_dim == g.dh, "the cache's geometry is not the attention's");
 }
 
+// The sequences' typical number of keys a query sees: their length, or what the window or chunk leaves of it.
+static int visible_context(const Step& st, const AttentionGeometry& g) {
+    return g.window != 0 && st.context > 0 ? std::min(st.context, std::abs(g.window)) : st.context;
+}
+
 static void decode_attention(Step& st, Tensor out, const Tensor& q, const AttentionGeometry& g, const LayerCache& cache) {
     Runtime& rt = *st.rt;
     MmaVariant& lib = mma_variant(g.dh);
     const ImpCacheView& c = cache.view;
     const int T = (int)rows(q);
-    const int n_splits = decode_splits(T, g.hkv, g.hq / g.hkv, c.page_size, rt.sm_count, st.context);
+    const int n_splits = decode_splits(T, g.hkv, g.hq / g.hkv, c.page_size, rt.sm_count, visible_context(st, g));
     const int64_t n_floats = lib.scratch_floats(T, g.hq, n_splits);
     float* scratch = n_floats ? (float*)rt.arena->alloc((size_t)n_floats * 4) : nullptr;
     check_variant(rt,
@@ -270,7 +277,7 @@ bool decode_attention_fused(Step& st, Tensor out, const Tensor& qkv, const Atten
          "fused decode attention: bfloat16 rows of q | k | v and a rotation over the whole head");
     MmaVariant& lib = mma_variant(g.dh);
     const int T = (int)rows(qkv);
-    const int n_splits = decode_splits(T, g.hkv, g.hq / g.hkv, c.page_size, rt.sm_count, st.context);
+    const int n_splits = decode_splits(T, g.hkv, g.hq / g.hkv, c.page_size, rt.sm_count, visible_context(st, g));
     const int64_t n_floats = lib.scratch_floats(T, g.hq, n_splits);
     float* scratch = n_floats ? (float*)rt.arena->alloc((size_t)n_floats * 4) : nullptr;
     const int rc = lib.decode_fused(out.data, out.stride0, qkv.data, qkv.stride0, c.k_pages, c.v_pages, c.block_table, c.bt_stride,
@@ -319,9 +326,11 @@ static bool bias_attention_mma(Step& st, Tensor out, const Tensor& q, const Atte
     auto decode = [&](Tensor o, const Tensor& qq) {
         const int T = (int)rows(qq), G = g.hq / g.hkv;
         // splits until every SM holds about three CTAs, none shorter than 64 keys of the typical context
-        const int base = std::max(1, T * g.hkv * ((G + 15) / 16));
+        const int base = std::max(1, T * g.hkv * ((G + 15) / 16)), context = visible_context(st, g);
         int n_splits = std::max(1, std::min(DECODE_MAX_SPLITS, rt.sm_count * 3 / base));
-        if (st.context > 0) n_splits = std::max(1, std::min(n_splits, st.context / 64));
+        if (context > 0) n_splits = std::max(1, std::min(n_splits, context / 64));
+        // a sink alone, pages of whole 16-key steps: the bulk-copy kernel, split as for plain attention
+        if (!ex.bias && c.page_size % 16 == 0) n_splits = decode_splits(T, g.hkv, G, c.page_size, rt.sm_count, context);
         const int64_t n_floats = lib.scratch_floats(T, g.hq, n_splits);
         float* scratch = n_floats ? (float*)rt.arena->alloc((size_t)n_floats * 4) : nullptr;
         check_variant(rt,

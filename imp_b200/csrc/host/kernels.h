@@ -222,6 +222,10 @@ int imp_moe_route(const void* x, int64_t ldx, int n_tokens, int d, const float* 
 int imp_moe_route_ex(const void* x, int64_t ldx, int n_tokens, int d, const float* wr, const float* br, int E, int top, const float* wg,
                      int* idx, float* wts, float* gate, int score_mode, int n_groups, int keep, int group_top, float weight_scale,
                      const float* choice_bias, int renormalise, int act_dtype, void* stream);
+int imp_moe_choose_sorts(int n_tokens, int R, int E, int top, int n_groups, int biased);
+int imp_moe_choose(const float* z, int64_t ldz, int n_splits, int64_t part_stride, int n_tokens, const float* br, int R, int E, int top,
+                   int* idx, float* wts, float* gate, int score_mode, int n_groups, int keep, int group_top, float weight_scale,
+                   const float* choice_bias, int renormalise, int* seg, int* row_token, int* pair_row, void* stream);
 int imp_moe_sort(const int* idx, int n_tokens, int top, int E, int* seg, int* row_token, int* pair_row, void* stream);
 int imp_gather_rows(void* dst, const void* src, int64_t ld, const int* idx, int n_rows, int d, int dtype, void* stream);
 int imp_moe_combine(void* out, const void* y, const int* pair_row, const float* wts, int n_tokens, int top, const void* shared,

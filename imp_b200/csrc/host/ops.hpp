@@ -72,10 +72,12 @@ struct AttentionGeometry {
     int hq, hkv, dh, window;
     float scale;
 };
-// The part of imp_qkv_prepare's arguments that the step, the cache and the geometry give; D and Dv are the caller's.
-inline ImpQkvPrepare qkv_prepare_args(const Step& st, const ImpCacheView& cv, const AttentionGeometry& g, const Tensor& proj, const Tensor& q) {
+// The part of imp_qkv_prepare's arguments that the step, the cache, the geometry and the product (unsummed, maybe) give; D and
+// Dv are the caller's.
+inline ImpQkvPrepare qkv_prepare_args(const Step& st, const ImpCacheView& cv, const AttentionGeometry& g, const Branch& proj, const Tensor& q) {
     ImpQkvPrepare p;
-    p.proj = proj.data, p.ld = proj.stride0, p.n_tokens = (int)rows(proj);
+    p.proj = proj.t.data, p.ld = proj.t.stride0, p.n_tokens = (int)rows(proj.t);
+    if (proj.split()) p.parts = proj.parts, p.n_splits = proj.n_splits, p.ld = cols(proj.t);
     p.Hq = g.hq, p.Hkv = g.hkv, p.Dc = g.dh;
     p.positions = st.view.positions, p.seq_of_token = st.view.seq_of_token;
     p.block_table = cv.block_table, p.bt_stride = cv.bt_stride, p.n_seqs = st.B();

@@ -617,10 +617,10 @@ struct GatedHeadAttention : Mixer {
         const int64_t T = rows(x);
         const ImpCacheView& cv = cache->view;
         Tensor proj = rt.empty(T, rows(w_in));
-        linear(rt, proj, x, w_in);
+        const Branch qkv = linear(rt, proj, x, w_in, !has_gate);   // unsummed parts go to qkv_prepare as they are
         Tensor q = rt.empty(T, (int64_t)g.hq * g.dh);
         ++rt.launches;
-        ImpQkvPrepare pr = qkv_prepare_args(st, cv, g, proj, q);
+        ImpQkvPrepare pr = qkv_prepare_args(st, cv, g, qkv, q);
         pr.bias = (const float*)qkv_bias.data;
         pr.D = D, pr.Dv = Dv;
         pr.qk_norm = qk_norm, pr.q_norm_w = (const float*)q_norm.data, pr.k_norm_w = (const float*)k_norm.data;

@@ -441,6 +441,15 @@ struct RoutedExperts : FeedForward {
     Tensor w_gate, w_up, w_down;       // [E * F, d], [E * F, d], [E * d, F]; or w_gate [E * 2F, d], gate and up rows alternating in runs of 8
     bool interleaved = false;
     Tensor router, router_bias, sg;    // float32
+    Tensor w_route{};                  // bfloat16 router rows (and the shared expert's mixing row behind them), padded to a multiple of 16: the
+                                       // logits by the tensor-core product
+    cudaStream_t side = nullptr;       // steps of single tokens: the shared expert beside the routed ones
+    cudaEvent_t fork = nullptr, join = nullptr;
+    ~RoutedExperts() override {
+        if (side) cudaStreamDestroy(side);
+        if (fork) cudaEventDestroy(fork);
+        if (join) cudaEventDestroy(join);
+    }
     Tensor s_gu, s_down;               // the shared expert
     bool s_interleaved = false;
 
@@ -538,6 +547,27 @@ struct RoutedExperts : FeedForward {
         }
         w_down = cat_rows(rt, *a.store, ds);
         router = to_float32(rt, *a.store, a.tensor("router"));
+        if (!rt.is_f32() && a.tensor("router").dtype == BF16 && d % 8 == 0 && (!(Fs > 0 && has_sgate) || a.tensor("shared_mix").dtype == BF16)) {
+            std::vector<Tensor> in = {a.tensor("router")};
+            if (Fs > 0 && has_sgate) in.push_back(a.tensor("shared_mix"));
+            int64_t n = 0;
+            for (const Tensor& t : in) n += rows(t);
+            const int64_t pad = (16 - n % 16) % 16;
+            Tensor zeros{};
+            if (pad) {
+                zeros = a.store->alloc(BF16, {pad, d});
+                IMP_CUDA(cudaMemsetAsync(zeros.data, 0, (size_t)numel(zeros) * 2, rt.stream));
+                in.push_back(zeros);
+            }
+            w_route = cat_rows(rt, *a.store, in);
+            IMP_CUDA(cudaStreamSynchronize(rt.stream));
+            if (pad) a.store->release(zeros.data);
+        }
+        if (Fs > 0 && env_flag("IMP_B200_PARALLEL_STREAMS", true)) {
+            IMP_CUDA(cudaStreamCreateWithFlags(&side, cudaStreamNonBlocking));
+            IMP_CUDA(cudaEventCreateWithFlags(&fork, cudaEventDisableTiming));
+            IMP_CUDA(cudaEventCreateWithFlags(&join, cudaEventDisableTiming));
+        }
         if (has_bias) router_bias = to_float32(rt, *a.store, a.tensor("router_bias"));
         if (a.params.get_bool("choice_bias", false)) choice_bias = to_float32(rt, *a.store, a.tensor("choice_bias"));
         if (Fs > 0) {
@@ -563,6 +593,19 @@ struct RoutedExperts : FeedForward {
         }
     }
 
+    Branch shared_expert(Runtime& rt, const Tensor& x, bool may_defer) {
+        const int64_t T = rows(x);
+        Tensor sa = rt.empty(T, Fs);
+        if (s_interleaved) {
+            linear_gated(rt, sa, x, s_gu, shared_act);
+        } else {
+            Tensor gu = rt.empty(T, 2 * Fs);
+            linear(rt, gu, x, s_gu);
+            gated_act(rt, sa, gu, 0, shared_act);
+        }
+        return linear(rt, rt.empty(T, d), sa, s_down, may_defer);
+    }
+
     Branch forward(Step& st, Tensor x) override {
         Runtime& rt = *st.rt;
         const int64_t T = rows(x), P = T * top;
@@ -573,13 +616,44 @@ struct RoutedExperts : FeedForward {
         int* seg = rt.arena->take<int>((size_t)E + 1);
         int* row_token = rt.arena->take<int>((size_t)P);
         int* pair_row = rt.arena->take<int>((size_t)P);
-        rt.launches += 5;
         const bool gated = Fs > 0 && has_sgate;
-        check_launch(imp_moe_route_ex(x.data, x.stride0, (int)T, (int)d, (const float*)router.data, has_bias ? (const float*)router_bias.data : nullptr, (int)R,
-                                      (int)top, gated ? (const float*)sg.data : nullptr, idx, wts, gate, score_mode, n_groups, keep_groups, group_top,
-                                      weight_scale, (const float*)choice_bias.data, renormalise ? 1 : 0, dt, rt.stream),
-                     "moe_route");
-        check_launch(imp_moe_sort(idx, (int)T, (int)top, (int)E, seg, row_token, pair_row, rt.stream), "moe_sort");
+        const bool hand_on = defer_rows && (Fs == 0 || (defer_terms && !gated));
+        // the shared expert needs the input alone: in a step of single tokens it runs on a stream of its own beside the rest
+        Branch shared{};
+        const bool forked = side && st.decode_only() && !st.diag;
+        if (forked) {
+            const cudaStream_t main = rt.stream;
+            IMP_CUDA(cudaEventRecord(fork, main));
+            IMP_CUDA(cudaStreamWaitEvent(side, fork, 0));
+            rt.stream = side;
+            try {
+                shared = shared_expert(rt, x, hand_on && defer_out);
+            } catch (...) {
+                rt.stream = main;
+                throw;
+            }
+            rt.stream = main;
+            IMP_CUDA(cudaEventRecord(join, side));
+        }
+        rt.launches += 5;
+        if (w_route.data && contiguous(x)) {
+            const int64_t N = rows(w_route);
+            Tensor zl = rt.empty(T, N, F32);
+            const Branch z = linear(rt, zl, x, w_route, true);
+            const int sorts = imp_moe_choose_sorts((int)T, (int)R, (int)E, (int)top, n_groups, choice_bias.data != nullptr);
+            rt.launches -= sorts;
+            check_launch(imp_moe_choose(z.split() ? z.parts : (const float*)zl.data, N, z.split() ? z.n_splits : 0, T * N, (int)T,
+                                        has_bias ? (const float*)router_bias.data : nullptr, (int)R, (int)E, (int)top, idx, wts, gated ? gate : nullptr,
+                                        score_mode, n_groups, keep_groups, group_top, weight_scale, (const float*)choice_bias.data, renormalise ? 1 : 0, seg,
+                                        row_token, pair_row, rt.stream),
+                         "moe_choose");
+        } else {
+            check_launch(imp_moe_route_ex(x.data, x.stride0, (int)T, (int)d, (const float*)router.data, has_bias ? (const float*)router_bias.data : nullptr, (int)R,
+                                          (int)top, gated ? (const float*)sg.data : nullptr, idx, wts, gate, score_mode, n_groups, keep_groups, group_top,
+                                          weight_scale, (const float*)choice_bias.data, renormalise ? 1 : 0, dt, rt.stream),
+                         "moe_route");
+            check_launch(imp_moe_sort(idx, (int)T, (int)top, (int)E, seg, row_token, pair_row, rt.stream), "moe_sort");
+        }
         Tensor hid = rt.empty(P, F);
         Tensor y = rt.empty(P, d);
         // Portions of prompts with much work an expert (rows x F x d of 2^31 and more on average): the list's offsets come to
@@ -627,19 +701,8 @@ struct RoutedExperts : FeedForward {
                                           dt, rt.stream),
                          "grouped_gemm (experts, down)");
         }
-        const bool hand_on = defer_rows && (Fs == 0 || (defer_terms && !gated));
-        Branch shared{};
-        if (Fs > 0) {
-            Tensor sa = rt.empty(T, Fs);
-            if (s_interleaved) {
-                linear_gated(rt, sa, x, s_gu, shared_act);
-            } else {
-                Tensor gu = rt.empty(T, 2 * Fs);
-                linear(rt, gu, x, s_gu);
-                gated_act(rt, sa, gu, 0, shared_act);
-            }
-            shared = linear(rt, rt.empty(T, d), sa, s_down, hand_on && defer_out);
-        }
+        if (forked) IMP_CUDA(cudaStreamWaitEvent(rt.stream, join, 0));
+        else if (Fs > 0) shared = shared_expert(rt, x, hand_on && defer_out);
         Tensor out = rt.empty(T, d);
         if (hand_on) {
             --rt.launches;

@@ -196,10 +196,10 @@ struct DifferentialAttention : Mixer {
         const int64_t T = rows(x);
         const ImpCacheView& cv = cache->view;
         Tensor proj = rt.empty(T, rows(w_in));
-        linear(rt, proj, x, w_in);
+        const Branch qkv = linear(rt, proj, x, w_in, true);   // unsummed parts go to qkv_prepare as they are
         Tensor q = rt.empty(T, (int64_t)g.hq * g.dh);
         rt.launches += 2;
-        ImpQkvPrepare pr = qkv_prepare_args(st, cv, g, proj, q);
+        ImpQkvPrepare pr = qkv_prepare_args(st, cv, g, qkv, q);
         pr.D = D, pr.Dv = Dv, pr.v_share = 2;
         pr.turns = (const float*)turns.data, pr.rot = rot, pr.pairing = pairing, pr.rot_mult = rot_mult;
         check_launch(imp_qkv_prepare(&pr, rt.status, rt.stream), "qkv_prepare");

@@ -13,6 +13,9 @@
 // Router outputs beyond the experts that have matrices are identity experts: they are chosen and weighed like the others, take no
 // part in the list (place -1), and give the input itself, y = x[t].
 //
+// Where the router's weights are 16-bit the logits come from the tensor-core product (16-bit operands, 32-bit sums and results: what
+// the 32-bit product of the same numbers gives up to the order of its sum) and moe_choose makes the choice; otherwise moe_route does both.
+//
 // The expert products run over a list of (token, choice) pairs sorted by expert (see grouped_gemm.cu); moe_sort makes
 // that list on the device: seg [E + 1], the token of every list row, and the row of every pair.  Nothing comes back
 // to the host, so the launches of a step depend on its sizes alone.
@@ -42,6 +45,111 @@ template <> struct Vec4<__nv_bfloat16> {
 };
 
 constexpr int ROUTE_BLOCK = 256, ROUTE_MAX_E = 1024, ROUTE_MAX_TOP = 32;
+
+// The choice of one token, made by one warp: `top` rounds of arg-max over what is left (the lower index wins a tie), and the
+// weights.  zt [E] in shared memory: the logits, or with score_mode 1 the sigmoid scores; gt [n_groups] and cs [E] (with
+// choice_bias): room for the groups' and the biased scores.  idx, wts [top].
+struct RouteRule {
+    int E, top, score_mode, n_groups, keep, group_top;
+    float weight_scale;
+    const float* choice_bias;
+    int renormalise;
+};
+__device__ __forceinline__ void choose_experts(const RouteRule& p, float* zt, float* gt, float* cs, int lane, int* __restrict__ idx, float* __restrict__ wts) {
+    const int E = p.E, top = p.top;
+    const float* zl = zt;            // the logits, where the choice scores are others
+    float chosen[ROUTE_MAX_TOP];
+    // softmax scores: the choice runs on the logits (same order); the weights need the largest and the sum over all experts
+    float z_max = 0.f, z_sum = 1.f;
+    if (p.score_mode == 2) {
+        float m = -INFINITY;
+        for (int e = lane; e < E; e += 32) m = fmaxf(m, zt[e]);
+        z_max = warp_max(m);
+        float sum = 0.f;
+        for (int e = lane; e < E; e += 32) sum += expf(zt[e] - z_max);
+        z_sum = warp_sum(sum);
+        if (p.choice_bias) {
+            zt = cs;
+            for (int e = lane; e < E; e += 32) zt[e] = expf(zl[e] - z_max) / z_sum + p.choice_bias[e];
+        }
+        __syncwarp();
+    }
+    if (p.n_groups > 0) {
+        // a group's score: the sum of its two largest scores (of its one score where a group is one expert),
+        // or with group_top 1 its largest one; then `keep`
+        // rounds of arg-max over the groups, the lower index winning a tie; the experts of the other groups leave
+        const int per = E / p.n_groups;
+        for (int g = lane; g < p.n_groups; g += 32) {
+            float a = -INFINITY, b = -INFINITY;
+            for (int e = g * per; e < (g + 1) * per; ++e) {
+                const float v = zt[e];
+                if (v > a) b = a, a = v;
+                else if (v > b) b = v;
+            }
+            gt[g] = per > 1 && p.group_top == 2 ? a + b : a;
+        }
+        __syncwarp();
+        for (int k = 0; k < p.keep; ++k) {
+            float best = -INFINITY;
+            int at = 0x7fffffff;
+            for (int g = lane; g < p.n_groups; g += 32) {
+                const float v = gt[g];
+                if (v > best) best = v, at = g;
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+                const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+                if (ov > best || (ov == best && oa < at)) best = ov, at = oa;
+            }
+            if (lane == 0 && at < p.n_groups) gt[at] = -INFINITY;   // kept
+            __syncwarp();
+        }
+        for (int e = lane; e < E; e += 32)
+            if (gt[e / per] != -INFINITY) zt[e] = -INFINITY;
+        __syncwarp();
+    }
+    for (int k = 0; k < top; ++k) {
+        float best = -INFINITY;
+        int at = 0x7fffffff;
+        for (int e = lane; e < E; e += 32) {
+            const float v = zt[e];
+            if (v > best) best = v, at = e;     // ascending e: the first of equal values stays
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+            if (ov > best || (ov == best && oa < at)) best = ov, at = oa;
+        }
+        if (at >= E) at = 0;     // nothing compares above -inf: the row holds NaNs
+        chosen[k] = p.score_mode == 2 && p.choice_bias ? zl[at] : best;
+        if (lane == 0) {
+            idx[k] = at;
+            zt[at] = -INFINITY;
+        }
+        __syncwarp();
+    }
+    if (lane == 0 && p.score_mode == 1) {
+        for (int k = 0; k < top; ++k) wts[k] = chosen[k] * p.weight_scale;   // the scores themselves, not renormalised
+    } else if (lane == 0 && p.score_mode == 2) {
+        float total = 0.f;
+        for (int k = 0; k < top; ++k) {
+            chosen[k] = expf(chosen[k] - z_max) / z_sum;
+            total += chosen[k];
+        }
+        const float f = p.renormalise ? p.weight_scale / (total + 1e-20f) : p.weight_scale;
+        for (int k = 0; k < top; ++k) wts[k] = chosen[k] * f;
+    } else if (lane == 0) {
+        const float largest = chosen[0];   // the first chosen is the largest
+        float sum = 0.f;
+        for (int k = 0; k < top; ++k) {
+            chosen[k] = expf(chosen[k] - largest);
+            sum += chosen[k];
+        }
+        for (int k = 0; k < top; ++k) wts[k] = chosen[k] / sum;
+    }
+}
 
 // A CTA routes TPB tokens: their rows wait in shared memory as 32-bit values while each warp walks the router's rows (and
 // the shared expert's mixing row), one row at a time against all TPB tokens, so a row of the router is read once per CTA.
@@ -107,150 +215,123 @@ __global__ void __launch_bounds__(ROUTE_BLOCK) moe_route_kernel(const TA* __rest
         }
     }
     __syncthreads();
-    // `top` rounds of arg-max over the logits that are left, a warp per token; the lower index wins a tie
-    for (int tk = warp; tk < nt; tk += ROUTE_BLOCK / 32) {
-        float* zt = z + tk * E;          // what is chosen from
-        const float* zl = z + tk * E;    // the logits, where the choice scores are others
-        const int64_t t = t0 + tk;
-        float chosen[ROUTE_MAX_TOP];
-        // softmax scores: the choice runs on the logits (same order); the weights need the largest and the sum over all experts
-        float z_max = 0.f, z_sum = 1.f;
-        if (score_mode == 2) {
-            float m = -INFINITY;
-            for (int e = lane; e < E; e += 32) m = fmaxf(m, zt[e]);
-            z_max = warp_max(m);
-            float sum = 0.f;
-            for (int e = lane; e < E; e += 32) sum += expf(zt[e] - z_max);
-            z_sum = warp_sum(sum);
-            if (choice_bias) {
-                zt = csc + tk * E;
-                for (int e = lane; e < E; e += 32) zt[e] = expf(zl[e] - z_max) / z_sum + choice_bias[e];
-            }
-            __syncwarp();
+    // a warp per token
+    const RouteRule rule{E, top, score_mode, n_groups, keep, group_top, weight_scale, choice_bias, renormalise};
+    for (int tk = warp; tk < nt; tk += ROUTE_BLOCK / 32)
+        choose_experts(rule, z + tk * E, gsc + tk * n_groups, csc + tk * E, lane, idx + (int64_t)(t0 + tk) * top, wts + (int64_t)(t0 + tk) * top);
+}
+
+constexpr int SORT_BLOCK = 1024, SORT_WARPS = SORT_BLOCK / 32;
+
+// By one CTA of SORT_BLOCK threads.  seg[e] .. seg[e + 1]: expert e's rows of the list; row_token[r]: the token of row r;
+// pair_row[p]: the row of pair p = t * top + k, -1 for a choice beyond the E experts.  Within an expert the rows follow the pair
+// index, so the list is the same for the same routing.  A warp owns a run of consecutive pairs: it counts its experts, the counts
+// become every warp's first row of every expert, and it walks its pairs again.  cnt: SORT_WARPS * E + SORT_WARPS ints in shared memory.
+__device__ __forceinline__ void sort_pairs(const int* idx, int n_pairs, int top, int E, int* cnt, int* __restrict__ seg, int* __restrict__ row_token,
+                                           int* __restrict__ pair_row) {
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    int* mine = cnt + warp * E;
+    int* warp_total = cnt + SORT_WARPS * E;
+    for (int e = tid; e < SORT_WARPS * E; e += SORT_BLOCK) cnt[e] = 0;
+    __syncthreads();
+    const int run = ((n_pairs + SORT_WARPS - 1) / SORT_WARPS + 31) & ~31;
+    const int p_begin = min(n_pairs, warp * run), p_end = min(n_pairs, p_begin + run);
+    for (int p0 = p_begin; p0 < p_end; p0 += 32) {
+        const int p = p0 + lane;
+        const int e = p < p_end ? idx[p] : -1;
+        const bool listed = e >= 0 && e < E;
+        const unsigned same = __match_any_sync(0xffffffffu, listed ? e : -1);
+        if (listed && lane == __ffs(same) - 1) mine[e] += __popc(same);
+        __syncwarp();
+    }
+    __syncthreads();
+    // thread e: the warps' counts of expert e become offsets within it, then a scan over the experts
+    int total = 0;
+    if (tid < E)
+        for (int w = 0; w < SORT_WARPS; ++w) {
+            const int c = cnt[w * E + tid];
+            cnt[w * E + tid] = total;
+            total += c;
         }
-        if (n_groups > 0) {
-            // a group's score: the sum of its two largest scores (of its one score where a group is one expert),
-            // or with group_top 1 its largest one; then `keep`
-            // rounds of arg-max over the groups, the lower index winning a tie; the experts of the other groups leave
-            float* gt = gsc + tk * n_groups;
-            const int per = E / n_groups;
-            for (int g = lane; g < n_groups; g += 32) {
-                float a = -INFINITY, b = -INFINITY;
-                for (int e = g * per; e < (g + 1) * per; ++e) {
-                    const float v = zt[e];
-                    if (v > a) b = a, a = v;
-                    else if (v > b) b = v;
-                }
-                gt[g] = per > 1 && group_top == 2 ? a + b : a;
-            }
-            __syncwarp();
-            for (int k = 0; k < keep; ++k) {
-                float best = -INFINITY;
-                int at = 0x7fffffff;
-                for (int g = lane; g < n_groups; g += 32) {
-                    const float v = gt[g];
-                    if (v > best) best = v, at = g;
-                }
+    int incl = total;
 #pragma unroll
-                for (int o = 16; o > 0; o >>= 1) {
-                    const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-                    const int oa = __shfl_xor_sync(0xffffffffu, at, o);
-                    if (ov > best || (ov == best && oa < at)) best = ov, at = oa;
-                }
-                if (lane == 0 && at < n_groups) gt[at] = -INFINITY;   // kept
-                __syncwarp();
-            }
-            for (int e = lane; e < E; e += 32)
-                if (gt[e / per] != -INFINITY) zt[e] = -INFINITY;
-            __syncwarp();
+    for (int o = 1; o < 32; o <<= 1) {
+        const int v = __shfl_up_sync(0xffffffffu, incl, o);
+        if (lane >= o) incl += v;
+    }
+    if (lane == 31) warp_total[warp] = incl;
+    __syncthreads();
+    int before = 0;
+    for (int w = 0; w < warp; ++w) before += warp_total[w];
+    const int first = before + incl - total;
+    if (tid < E) {
+        seg[tid] = first;
+        if (tid == E - 1) seg[E] = first + total;
+        for (int w = 0; w < SORT_WARPS; ++w) cnt[w * E + tid] += first;
+    }
+    __syncthreads();
+    for (int p0 = p_begin; p0 < p_end; p0 += 32) {
+        const int p = p0 + lane;
+        const int e = p < p_end ? idx[p] : -1;
+        const bool listed = e >= 0 && e < E;
+        const unsigned same = __match_any_sync(0xffffffffu, listed ? e : -1);
+        if (listed) {
+            const int r = mine[e] + __popc(same & ((1u << lane) - 1u));
+            row_token[r] = p / top;
+            pair_row[p] = r;
+        } else if (p < p_end) {
+            pair_row[p] = -1;     // an identity expert: no row of the list
         }
-        for (int k = 0; k < top; ++k) {
-            float best = -INFINITY;
-            int at = 0x7fffffff;
-            for (int e = lane; e < E; e += 32) {
-                const float v = zt[e];
-                if (v > best) best = v, at = e;     // ascending e: the first of equal values stays
-            }
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1) {
-                const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-                const int oa = __shfl_xor_sync(0xffffffffu, at, o);
-                if (ov > best || (ov == best && oa < at)) best = ov, at = oa;
-            }
-            if (at >= E) at = 0;     // nothing compares above -inf: the row holds NaNs
-            chosen[k] = score_mode == 2 && choice_bias ? zl[at] : best;
-            if (lane == 0) {
-                idx[t * top + k] = at;
-                zt[at] = -INFINITY;
-            }
-            __syncwarp();
-        }
-        if (lane == 0 && score_mode == 1) {
-            for (int k = 0; k < top; ++k) wts[t * top + k] = chosen[k] * weight_scale;   // the scores themselves, not renormalised
-        } else if (lane == 0 && score_mode == 2) {
-            float total = 0.f;
-            for (int k = 0; k < top; ++k) {
-                chosen[k] = expf(chosen[k] - z_max) / z_sum;
-                total += chosen[k];
-            }
-            const float f = renormalise ? weight_scale / (total + 1e-20f) : weight_scale;
-            for (int k = 0; k < top; ++k) wts[t * top + k] = chosen[k] * f;
-        } else if (lane == 0) {
-            const float largest = chosen[0];   // the first chosen is the largest
-            float sum = 0.f;
-            for (int k = 0; k < top; ++k) {
-                chosen[k] = expf(chosen[k] - largest);
-                sum += chosen[k];
-            }
-            for (int k = 0; k < top; ++k) wts[t * top + k] = chosen[k] / sum;
-        }
+        __syncwarp();
+        if (listed && lane == __ffs(same) - 1) mine[e] += __popc(same);
+        __syncwarp();
     }
 }
 
-// One CTA.  seg[e] .. seg[e + 1]: expert e's rows of the list; row_token[r]: the token of row r; pair_row[p]: the row of
-// pair p = t * top + k.  Within an expert the rows follow the pair index, so the list is the same for the same routing.
-__global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ idx, int n_pairs, int top, int E, int* __restrict__ seg,
-                                                        int* __restrict__ row_token, int* __restrict__ pair_row) {
+__global__ void __launch_bounds__(SORT_BLOCK) moe_sort_kernel(const int* __restrict__ idx, int n_pairs, int top, int E, int* __restrict__ seg,
+                                                              int* __restrict__ row_token, int* __restrict__ pair_row) {
     pdl_wait();
     pdl_launch_dependents();
-    extern __shared__ int cnt[];   // [E + 1]
-    const int tid = threadIdx.x;
-    for (int e = tid; e <= E; e += blockDim.x) cnt[e] = 0;
-    __syncthreads();
-    for (int p = tid; p < n_pairs; p += blockDim.x) {
-        const int e = idx[p];
-        if (e >= 0 && e < E) atomicAdd(&cnt[e], 1);
-    }
-    __syncthreads();
-    if (tid == 0) {
-        int run = 0;
-        for (int e = 0; e < E; ++e) {
-            const int c = cnt[e];
-            cnt[e] = run;
-            seg[e] = run;
-            run += c;
+    extern __shared__ int cnt[];
+    sort_pairs(idx, n_pairs, top, E, cnt, seg, row_token, pair_row);
+}
+
+// The choice from logits that a product has made: row t of z (rows ldz apart) holds the router's R logits and, with `gate`, the
+// shared expert's mixing logit behind them; with n_splits > 0 z is the product's unsummed parts, part_stride floats apart, added in
+// order.  A warp per token; br: the router's bias or null.  SORT: one CTA for all tokens, which then makes the list (few tokens).
+template <bool SORT>
+__global__ void __launch_bounds__(SORT ? SORT_BLOCK : 256) moe_choose_kernel(const float* __restrict__ z, int64_t ldz, int n_splits, int64_t part_stride,
+                                                                            int n_tokens, const float* __restrict__ br, const RouteRule rule,
+                                                                            int* __restrict__ idx, float* __restrict__ wts, float* __restrict__ gate, int E,
+                                                                            int* __restrict__ seg, int* __restrict__ row_token, int* __restrict__ pair_row) {
+    pdl_wait();
+    pdl_launch_dependents();
+    extern __shared__ __align__(16) float sm[];   // a warp's logits [R], groups [n_groups] and biased scores [R]; with SORT idx and counts behind
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+    const int R = rule.E, per = R * (rule.choice_bias ? 2 : 1) + rule.n_groups;
+    float* zt = sm + (size_t)warp * per;
+    float* gt = zt + R;
+    float* cs = gt + rule.n_groups;
+    int* sidx = reinterpret_cast<int*>(sm + (size_t)n_warps * per);
+    auto logit = [&](int t, int e) {
+        const float* p = z + (int64_t)t * ldz + e;
+        float v = *p;
+        for (int s = 1; s < n_splits; ++s) v += p[(int64_t)s * part_stride];
+        return v;
+    };
+    for (int t = SORT ? warp : blockIdx.x * n_warps + warp; t < (SORT ? n_tokens : min(n_tokens, (int)(blockIdx.x + 1) * n_warps)); t += n_warps) {
+        for (int e = lane; e < R; e += 32) {
+            const float v = logit(t, e) + (br ? br[e] : 0.f);
+            zt[e] = rule.score_mode == 1 ? 1.f / (1.f + expf(-v)) : v;
         }
-        cnt[E] = run;
-        seg[E] = run;
+        if (gate && lane == 0) gate[t] = 1.f / (1.f + expf(-logit(t, R)));
+        __syncwarp();
+        choose_experts(rule, zt, gt, cs, lane, SORT ? sidx + t * rule.top : idx + (int64_t)t * rule.top, wts + (int64_t)t * rule.top);
+        __syncwarp();
     }
-    __syncthreads();
-    for (int p = tid; p < n_pairs; p += blockDim.x)
-        if (idx[p] >= E) pair_row[p] = -1;   // an identity expert: no row of the list
-    // every expert's rows in pair order: a warp walks the pairs of one expert at a time
-    const int lane = tid & 31, warp = tid >> 5, n_warps = blockDim.x >> 5;
-    for (int e = warp; e < E; e += n_warps) {
-        int at = cnt[e];
-        for (int p0 = 0; p0 < n_pairs; p0 += 32) {
-            const int p = p0 + lane;
-            const bool mine = p < n_pairs && idx[p] == e;
-            const unsigned m = __ballot_sync(0xffffffffu, mine);
-            if (mine) {
-                const int r = at + __popc(m & ((1u << lane) - 1u));
-                row_token[r] = p / top;
-                pair_row[p] = r;
-            }
-            at += __popc(m);
-        }
+    if (SORT) {
+        __syncthreads();
+        sort_pairs(sidx, n_tokens * rule.top, rule.top, E, sidx + n_tokens * rule.top, seg, row_token, pair_row);
     }
 }
 
@@ -393,13 +474,58 @@ IMP_API int imp_moe_route(const void* x, int64_t ldx, int n_tokens, int d, const
 IMP_API int imp_moe_sort(const int* idx, int n_tokens, int top, int E, int* seg, int* row_token, int* pair_row, void* stream) {
     if (n_tokens == 0) return 0;
     IMP_CHECK_ARG(idx && seg && row_token && pair_row && top > 0 && E > 0 && E <= ROUTE_MAX_E, "imp_moe_sort: bad argument");
-    cudaError_t e = imp_launch(moe_sort_kernel, dim3(1), dim3(1024), (size_t)(E + 1) * 4, (cudaStream_t)stream, idx, n_tokens * top, top, E, seg,
-                               row_token, pair_row);
+    const size_t smem = (size_t)(SORT_WARPS * E + SORT_WARPS) * 4;
+    cudaError_t e = cudaSuccess;
+    if (smem > 48 * 1024) e = cudaFuncSetAttribute(moe_sort_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e == cudaSuccess)
+        e = imp_launch(moe_sort_kernel, dim3(1), dim3(SORT_BLOCK), smem, (cudaStream_t)stream, idx, n_tokens * top, top, E, seg, row_token, pair_row);
     if (e != cudaSuccess) {
         imp_set_error("imp_moe_sort: %s", cudaGetErrorString(e));
         return (int)e;
     }
     return 0;
+}
+
+// The choice of T tokens from a product's float32 logits (see moe_choose_kernel; the rule as for imp_moe_route_ex, R router outputs of
+// which the first E have matrices), and the list of imp_moe_sort.  gate float32 [T] or null.  sorts: whether one kernel does both.
+IMP_API int imp_moe_choose_sorts(int n_tokens, int R, int E, int top, int n_groups, int biased) {
+    if (n_tokens <= 0 || n_tokens > 128) return 0;
+    return ((size_t)SORT_WARPS * (R * (biased ? 2 : 1) + n_groups) + (size_t)n_tokens * top + (size_t)SORT_WARPS * (E + 1)) * 4 <= 200 * 1024 ? 1 : 0;
+}
+IMP_API int imp_moe_choose(const float* z, int64_t ldz, int n_splits, int64_t part_stride, int n_tokens, const float* br, int R, int E, int top, int* idx,
+                           float* wts, float* gate, int score_mode, int n_groups, int keep, int group_top, float weight_scale, const float* choice_bias,
+                           int renormalise, int* seg, int* row_token, int* pair_row, void* stream) {
+    if (n_tokens == 0) return 0;
+    IMP_CHECK_ARG(z && idx && wts && seg && row_token && pair_row && n_splits >= 0, "imp_moe_choose: bad argument");
+    IMP_CHECK_ARG(R > 0 && R <= ROUTE_MAX_E && E > 0 && E <= R && top > 0 && top <= R && top <= ROUTE_MAX_TOP && ldz >= R + (gate ? 1 : 0),
+                  "imp_moe_choose: %d router outputs (at most %d), %d chosen (at most %d)", R, ROUTE_MAX_E, top, ROUTE_MAX_TOP);
+    IMP_CHECK_ARG(n_groups == 0 || (R % n_groups == 0 && keep > 0 && keep <= n_groups && top <= keep * (R / n_groups)), "imp_moe_choose: bad groups");
+    cudaStream_t s = (cudaStream_t)stream;
+    const RouteRule rule{R, top, score_mode, n_groups, keep, group_top, weight_scale, choice_bias, renormalise};
+    const size_t per = ((size_t)R * (choice_bias ? 2 : 1) + n_groups) * 4;
+    cudaError_t e = cudaSuccess;
+    if (imp_moe_choose_sorts(n_tokens, R, E, top, n_groups, choice_bias != nullptr)) {
+        const size_t smem = SORT_WARPS * per + ((size_t)n_tokens * top + (size_t)SORT_WARPS * (E + 1)) * 4;
+        if (smem > 48 * 1024) e = cudaFuncSetAttribute(moe_choose_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e == cudaSuccess)
+            e = imp_launch(moe_choose_kernel<true>, dim3(1), dim3(SORT_BLOCK), smem, s, z, ldz, n_splits, part_stride, n_tokens, br, rule, idx, wts, gate, E, seg,
+                           row_token, pair_row);
+        if (e != cudaSuccess) {
+            imp_set_error("imp_moe_choose: %s", cudaGetErrorString(e));
+            return (int)e;
+        }
+        return 0;
+    }
+    const size_t smem = 8 * per;
+    if (smem > 48 * 1024) e = cudaFuncSetAttribute(moe_choose_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e == cudaSuccess)
+        e = imp_launch(moe_choose_kernel<false>, dim3((n_tokens + 7) / 8), dim3(256), smem, s, z, ldz, n_splits, part_stride, n_tokens, br, rule, idx, wts,
+                       gate, E, seg, row_token, pair_row);
+    if (e != cudaSuccess) {
+        imp_set_error("imp_moe_choose: %s", cudaGetErrorString(e));
+        return (int)e;
+    }
+    return imp_moe_sort(idx, n_tokens, top, E, seg, row_token, pair_row, stream);
 }
 
 // out [T, d] = sum_k wts[t, k] * y[pair_row[t * top + k]] (+ gate[t] * shared[t]); y [T * top, d], all dense.  A negative place

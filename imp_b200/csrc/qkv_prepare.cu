@@ -62,7 +62,7 @@ __global__ void __launch_bounds__(QP_BLOCK) qkv_prepare_kernel(const ImpQkvPrepa
         const int head = is_q ? unit : is_v ? unit - Hq - Hkv : unit - Hq;
         const int n = is_v ? p.Dv : D;
         const int64_t col = is_q ? (int64_t)head * D : is_v ? (int64_t)(Hq + Hkv) * D + (int64_t)(head / p.v_share) * p.Dv : (int64_t)(Hq + head) * D;
-        const TA* src = (const TA*)p.proj + t * p.ld + col;
+        const TA* src = p.parts ? nullptr : (const TA*)p.proj + t * p.ld + col;
         TA* dst;
         if (is_q) {
             dst = (TA*)p.q_out + t * p.q_ld + (int64_t)head * Dc;
@@ -79,7 +79,17 @@ __global__ void __launch_bounds__(QP_BLOCK) qkv_prepare_kernel(const ImpQkvPrepa
 #pragma unroll
         for (int i = 0; i < PER; ++i) {
             const int d = lane + i * 32;
-            x[i] = d < n ? to_float(src[d]) + (p.bias ? p.bias[col + d] : 0.f) : 0.f;
+            x[i] = 0.f;
+            if (d < n) {
+                if (src) {
+                    x[i] = to_float(src[d]);
+                } else {
+                    float acc = 0.f;
+                    for (int s = 0; s < p.n_splits; ++s) acc += p.parts[((int64_t)s * p.n_tokens + t) * p.ld + col + d];
+                    x[i] = to_float(from_float<TA>(acc));
+                }
+                if (p.bias) x[i] += p.bias[col + d];
+            }
         }
         const float* nw = is_q ? p.q_norm_w : is_v ? nullptr : p.k_norm_w;
         auto norm = [&] {
@@ -178,7 +188,17 @@ __global__ void __launch_bounds__(QP_BLOCK) qkv_prepare_vec_kernel(const ImpQkvP
         float x[8];
 #pragma unroll
         for (int i = 0; i < 8; ++i) x[i] = 0.f;
-        if (mine) {
+        if (mine && p.parts) {
+            const float* src = p.parts + t * p.ld + col + d0;
+#pragma unroll 4
+            for (int s = 0; s < p.n_splits; ++s, src += (int64_t)p.n_tokens * p.ld) {
+                const float4 a = *reinterpret_cast<const float4*>(src), b = *reinterpret_cast<const float4*>(src + 4);
+                x[0] += a.x, x[1] += a.y, x[2] += a.z, x[3] += a.w;
+                x[4] += b.x, x[5] += b.y, x[6] += b.z, x[7] += b.w;
+            }
+#pragma unroll
+            for (int i = 0; i < 8; ++i) x[i] = to_float(from_float<TA>(x[i]));
+        } else if (mine) {
             const uint4 raw = *reinterpret_cast<const uint4*>((const TA*)p.proj + t * p.ld + col + d0);
             const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
 #pragma unroll
@@ -186,6 +206,8 @@ __global__ void __launch_bounds__(QP_BLOCK) qkv_prepare_vec_kernel(const ImpQkvP
                 const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i]));
                 x[2 * i] = f.x, x[2 * i + 1] = f.y;
             }
+        }
+        if (mine) {
             if (p.bias) {
                 const float4 b0 = *reinterpret_cast<const float4*>(p.bias + col + d0), b1 = *reinterpret_cast<const float4*>(p.bias + col + d0 + 4);
                 x[0] += b0.x, x[1] += b0.y, x[2] += b0.z, x[3] += b0.w;
@@ -403,7 +425,7 @@ IMP_API int imp_qkv_prepare(const ImpQkvPrepare* args, int* status, void* stream
     IMP_CHECK_ARG(args, "imp_qkv_prepare: null pointer");
     const ImpQkvPrepare& p = *args;
     if (p.n_tokens == 0) return 0;
-    IMP_CHECK_ARG(p.proj && p.positions && p.seq_of_token && p.block_table && p.q_out, "imp_qkv_prepare: null pointer");
+    IMP_CHECK_ARG((p.proj || p.parts) && p.positions && p.seq_of_token && p.block_table && p.q_out, "imp_qkv_prepare: null pointer");
     IMP_CHECK_ARG(p.Hq > 0 && p.Hkv > 0 && p.D > 0 && p.Dv > 0 && p.Dc >= p.D && p.Dc >= p.Dv && p.Dc <= QP_MAX_D,
                   "imp_qkv_prepare: head sizes %d / %d must fit the cache's %d (at most %d)", p.D, p.Dv, p.Dc, QP_MAX_D);
     IMP_CHECK_ARG(p.rot >= 0 && p.rot % 2 == 0 && p.rot <= p.D && (p.rot == 0 || p.turns), "imp_qkv_prepare: the rotated part must be even and within the head");
@@ -417,7 +439,7 @@ IMP_API int imp_qkv_prepare(const ImpQkvPrepare* args, int* status, void* stream
     const int units = p.Hq + 2 * p.Hkv;
     bool vec = p.act_dtype != IMP_F32 && p.D % 8 == 0 && p.Dv % 8 == 0 && p.Dc % 8 == 0 && p.Dc <= 256 && p.ld % 8 == 0 && p.q_ld % 8 == 0 &&
                (p.rot == 0 || p.pairing == 1);
-    for (const void* q : {p.proj, (const void*)p.bias, (const void*)p.q_norm_w, (const void*)p.k_norm_w, (const void*)p.q_out, (const void*)p.k_cache,
+    for (const void* q : {p.parts ? (const void*)p.parts : p.proj, (const void*)p.bias, (const void*)p.q_norm_w, (const void*)p.k_norm_w, (const void*)p.q_out, (const void*)p.k_cache,
                           (const void*)p.v_cache})
         vec = vec && (uintptr_t)q % 16 == 0;
     // few tokens: a token's units spread over several CTAs; many: one CTA makes the token's angles once for all of them

@@ -8,6 +8,8 @@ enum { QK_NORM_NONE = 0, QK_NORM_BEFORE_ROTATION = 1, QK_NORM_AFTER_ROTATION = 2
 struct ImpQkvPrepare {
     const void* proj = nullptr;        // [n_tokens, ld] in act_dtype, columns [q: Hq * D | k: Hkv * D | v: (Hkv / v_share) * Dv | ...]
     int64_t ld = 0;
+    const float* parts = nullptr;      // instead of proj: the unsummed float32 parts [n_splits][n_tokens, ld] of the product, added
+    int n_splits = 0;                  // in order and rounded to act_dtype as the summing kernel would have stored them
     const float* bias = nullptr;       // one number per column of q, k and v, added first; or null
     int n_tokens = 0, Hq = 0, Hkv = 0, D = 0, Dv = 0;
     int Dc = 0;                        // the cache's head size (at least D and Dv): the rest of a row is zeros

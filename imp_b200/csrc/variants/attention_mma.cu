@@ -1032,13 +1032,14 @@ __device__ __forceinline__ void dec_patch_own_key(const OwnKey& own, unsigned ch
     __syncwarp();
 }
 
-template <int NR>
+// SINK: 2^sink_l2[head] joins every head's softmax denominator (a key without a value); the first split takes it into its state.
+template <int NR, bool SINK = false>
 __global__ void __launch_bounds__((DT_CONSUMERS + 1) * 32) attn_decode_tma_kernel(
     __nv_bfloat16* __restrict__ out, int64_t out_stride, const __nv_bfloat16* __restrict__ q, int64_t q_stride,
     const __nv_bfloat16* __restrict__ kc, const __nv_bfloat16* __restrict__ vc, const int* __restrict__ block_table,
     int bt_stride, const int* __restrict__ seq_of_token, const int* __restrict__ positions, int n_seqs, int Hq,
     int Hkv, int P, int num_pages, float scale_log2, int window, int n_splits, float* __restrict__ part_o,
-    float* __restrict__ part_ml, int* status, const DecFused fz, int cluster_merge) {
+    float* __restrict__ part_ml, int* status, const DecFused fz, int cluster_merge, const float* __restrict__ sink_l2) {
     // cluster_merge: the CTAs of the key splits of one (token, kv head) form a cluster (grid.x == cluster size) and
     // merge their results in the first CTA's shared memory: no partial results in global memory, no merge kernel.
     // pdl_wait() comes later: the batch arrays and the keys before this step's position do not depend on the
@@ -1251,6 +1252,20 @@ __global__ void __launch_bounds__((DT_CONSUMERS + 1) * 32) attn_decode_tma_kerne
             }
         }
     }
+    if (SINK && warp == 0 && split == 0) {
+#pragma unroll
+        for (int r = 0; r < NR; ++r) {
+            const int hr = row0 + g + 8 * r;
+            if (hr >= G) continue;
+            const float sk = sink_l2[hk * G + hr];
+            const float m_new = fmaxf(st.m[r], sk);
+            const float c = exp2f(st.m[r] - m_new);                // st.m = -inf -> 0
+            st.l[r] = st.l[r] * c + exp2f(sk - m_new);
+            st.m[r] = m_new;
+#pragma unroll
+            for (int i = 0; i < NTILES; ++i) { st.o[i][2 * r] *= c; st.o[i][2 * r + 1] *= c; }
+        }
+    }
     if (cluster_merge) {
         // Every CTA of the cluster is past its ring (first barrier; it also says that all of them run), then the
         // splits 1.. store their state into the first CTA's shared memory behind its own merge buffer (second
@@ -1338,16 +1353,16 @@ __global__ void __launch_bounds__((DT_CONSUMERS + 1) * 32) attn_decode_tma_kerne
 constexpr int DT_CLUSTER_MAX = IMP_DT_CLUSTER_MAX;
 
 // *merged is set when the key splits merged inside the kernel (a cluster per (token, kv head)): no merge kernel then.
-template <int NR>
+template <int NR, bool SINK = false>
 static int launch_decode_tma(dim3 grid, cudaStream_t s, void* out, int64_t out_stride, const void* q, int64_t q_stride,
                              const void* kc, const void* vc, const int* block_table, int bt_stride, const int* seq_of_token,
                              const int* positions, int n_seqs, int Hq, int Hkv, int P, int num_pages, float scale_log2,
                              int window, int n_splits, float* part_o, float* part_ml, int* status, const DecFused& fz,
-                             bool* merged) {
+                             bool* merged, const float* sink_l2 = nullptr) {
     constexpr int SLOT = (NTILES * 2 * NR + 2 * NR) * 32 * (int)sizeof(float);      // one warp's (or split's) state
     constexpr int MERGE = (DT_CONSUMERS - 1 + DT_CLUSTER_MAX - 1) * SLOT;           // the warps' merge, then the splits'
     constexpr int SMEM = DT_STAGES * DT_STAGE_BYTES > MERGE ? DT_STAGES * DT_STAGE_BYTES : MERGE;
-    auto kernel = attn_decode_tma_kernel<NR>;
+    auto kernel = attn_decode_tma_kernel<NR, SINK>;
     static bool attr_set = false;
     if (!attr_set) {   // always: the kernel's static barriers come on top of the ring
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
@@ -1400,7 +1415,7 @@ static int launch_decode_tma(dim3 grid, cudaStream_t s, void* out, int64_t out_s
     cudaError_t e = cudaLaunchKernelEx(&cfg, kernel, (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)q, q_stride,
                                        (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, block_table, bt_stride, seq_of_token,
                                        positions, n_seqs, Hq, Hkv, P, num_pages, scale_log2, window, n_splits, part_o, part_ml,
-                                       status, fz, cluster_merge);
+                                       status, fz, cluster_merge, sink_l2);
     if (e != cudaSuccess) { imp_set_error("imp_attn_decode: %s", cudaGetErrorString(e)); return (int)e; }
     *merged = cluster_merge != 0;
     return 0;
@@ -1479,8 +1494,9 @@ IMP_API int imp_attn_decode(void* out, int64_t out_stride, const void* q, int64_
                             n_seqs, Hq, Hkv, P, num_pages, scale, window, n_splits, scratch, status, stream, DecFused{});
 }
 
-// Decode with a score bias by distance and a sink (see ScoreExtras; either table may be null): the kernel that reads
-// keys straight from the pages, at any page size.  The splits' merge adds the sink's term.
+// Decode with a score bias by distance and a sink (see ScoreExtras; either table may be null).  A sink alone, with pages of whole
+// 16-key steps, runs on the bulk-copy kernel; everything else on the kernel that reads keys straight from the pages, where the
+// splits' merge adds the sink's term.
 IMP_API int imp_attn_decode_bias(void* out, int64_t out_stride, const void* q, int64_t q_stride, const void* kc,
                                  const void* vc, const int* block_table, int bt_stride, const int* seq_of_token,
                                  const int* positions, int n_tokens, int n_seqs, int Hq, int Hkv, int P, int num_pages,
@@ -1498,6 +1514,18 @@ IMP_API int imp_attn_decode_bias(void* out, int64_t out_stride, const void* q, i
     float* part_ml = scratch ? scratch + (int64_t)n_tokens * Hq * n_splits * DH : nullptr;
     const ScoreExtras ex{bias_l2, n_dist, sink_l2};
     dim3 grid(n_splits, Hkv * ((G + 15) / 16), n_tokens);
+    if (!bias_l2 && sink_l2 && P % 16 == 0 && getenv("IMP_B200_ATTN_DIRECT") == nullptr) {
+        bool merged = false;
+        const DecFused fz{};
+#define DEC_ARGS grid, s, out, out_stride, q, q_stride, kc, vc, block_table, bt_stride, seq_of_token, positions, n_seqs, Hq, Hkv, P, \
+                 num_pages, scale * 1.4426950408889634f, window, n_splits, part_o, part_ml, status, fz, &merged, sink_l2
+        if (int rc = (G <= 8) ? launch_decode_tma<1, true>(DEC_ARGS) : launch_decode_tma<2, true>(DEC_ARGS)) return rc;
+#undef DEC_ARGS
+        if (n_splits > 1 && !merged)
+            imp_launch(attn_merge_kernel, dim3(n_tokens * Hq), dim3(128), 0, s, (__nv_bfloat16*)out, out_stride, (const float*)part_o,
+                       (const float*)part_ml, Hq, n_splits, (const float*)nullptr);      // the first split's state holds the sink
+        IMP_RETURN_LAUNCH();
+    }
 #define DEC_ARGS grid, s, out, out_stride, q, q_stride, kc, vc, block_table, bt_stride, seq_of_token, positions, n_seqs, Hq, Hkv, P, \
                  num_pages, scale * 1.4426950408889634f, window, n_splits, part_o, part_ml, status, ex
     if (int rc = (G <= 8) ? launch_decode<1, true>(DEC_ARGS) : launch_decode<2, true>(DEC_ARGS)) return rc;
