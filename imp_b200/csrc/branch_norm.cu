@@ -21,12 +21,14 @@ namespace {
 constexpr int BN_THREADS = 128, BN_MAX_C = 8, BN_ROW_THREADS = 256;
 
 
-// NV float4 a thread; CLUSTER: gridDim.x / C rows, a cluster of C CTAs each; else a CTA a row.  DENSE: the branch is one dense
-// tensor (`first.t`), asked for together with the stream.
-template <typename TA, typename TW, int NV, bool CLUSTER, bool DENSE>
+// NV float4 a thread; CLUSTER: gridDim.x / C rows, a cluster of C CTAs each; else a CTA a row.  FORM: what the branch is, so that the usual
+// cases of long portions need few registers: any, one dense tensor (asked for together with the stream), or no unsummed parts.
+enum : int { BN_ANY = 0, BN_DENSE = 1, BN_NO_PARTS = 2 };
+template <typename TA, typename TW, int NV, bool CLUSTER, int FORM>
 __global__ void __launch_bounds__(CLUSTER ? BN_THREADS : BN_ROW_THREADS)
     add_rms_branch_kernel(float* __restrict__ h, ImpBranchTerm first, ImpBranchTerm second, const float* __restrict__ bias, const TW* __restrict__ w,
                           TA* __restrict__ out, int64_t n_rows, int d, float eps, int C) {
+    constexpr bool DENSE = FORM == BN_DENSE;
     constexpr int NT = CLUSTER ? BN_THREADS : BN_ROW_THREADS;
     __shared__ float scratch[33];
     __shared__ float slots[BN_MAX_C];
@@ -58,14 +60,15 @@ __global__ void __launch_bounds__(CLUSTER ? BN_THREADS : BN_ROW_THREADS)
             else b[i][0] = b0.x, b[i][1] = b0.y, b[i][2] = b0.z, b[i][3] = b0.w;
         }
     }
+    if (!DENSE) {
+        const int c0 = 4 * (rank * NT + (int)threadIdx.x);
+        add_term_pieces<TA, NV, FORM == BN_ANY>(b, first, x, t, c0, 4 * stride, d, n_rows * d);
+        add_term_pieces<TA, NV, FORM == BN_ANY>(b, second, x, t, c0, 4 * stride, d, n_rows * d);
+    }
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
         const int c = rank * NT + threadIdx.x + i * stride;
         if (c < nv) {
-            if (!DENSE) {
-                add_term<TA, 4>(b[i], first, x[i], t, 4 * c, d, n_rows * d);
-                add_term<TA, 4>(b[i], second, x[i], t, 4 * c, d, n_rows * d);
-            }
 #pragma unroll
             for (int e = 0; e < 4; ++e) ss = fmaf(b[i][e], b[i][e], ss);
         }
@@ -150,14 +153,14 @@ cudaError_t launch_branch(float* h, const ImpBranchTerm& a, const ImpBranchTerm&
         cfg.attrs = attr;
         cfg.numAttrs = imp_pdl_enabled() ? 2 : 1;
         if (per == 1)
-            return cudaLaunchKernelEx(&cfg, add_rms_branch_kernel<TA, TW, 1, true, false>, h, a, b, bias, (const TW*)w, (TA*)out, (int64_t)n, d, eps, C);
-        return cudaLaunchKernelEx(&cfg, add_rms_branch_kernel<TA, TW, 2, true, false>, h, a, b, bias, (const TW*)w, (TA*)out, (int64_t)n, d, eps, C);
+            return cudaLaunchKernelEx(&cfg, add_rms_branch_kernel<TA, TW, 1, true, BN_ANY>, h, a, b, bias, (const TW*)w, (TA*)out, (int64_t)n, d, eps, C);
+        return cudaLaunchKernelEx(&cfg, add_rms_branch_kernel<TA, TW, 2, true, BN_ANY>, h, a, b, bias, (const TW*)w, (TA*)out, (int64_t)n, d, eps, C);
     }
     const int per = (nv + BN_ROW_THREADS - 1) / BN_ROW_THREADS;
-    const bool dense = a.t && !a.parts && !a.y && !b.t && !b.parts && !b.y;
-#define BN_ROW(NV) (dense ? BN_ROW_FORM(NV, true) : BN_ROW_FORM(NV, false))
-#define BN_ROW_FORM(NV, DENSE) \
-    imp_launch(add_rms_branch_kernel<TA, TW, NV, false, DENSE>, dim3(n), dim3(BN_ROW_THREADS), 0, s, h, a, b, bias, (const TW*)w, (TA*)out, (int64_t)n, d, eps, 1)
+    const int form = a.parts || b.parts ? BN_ANY : a.t && !b.t && !b.y ? BN_DENSE : BN_NO_PARTS;
+#define BN_ROW(NV) (form == BN_DENSE ? BN_ROW_FORM(NV, BN_DENSE) : form == BN_NO_PARTS ? BN_ROW_FORM(NV, BN_NO_PARTS) : BN_ROW_FORM(NV, BN_ANY))
+#define BN_ROW_FORM(NV, FORM) \
+    imp_launch(add_rms_branch_kernel<TA, TW, NV, false, FORM>, dim3(n), dim3(BN_ROW_THREADS), 0, s, h, a, b, bias, (const TW*)w, (TA*)out, (int64_t)n, d, eps, 1)
     return per <= 1 ? BN_ROW(1) : per <= 2 ? BN_ROW(2) : per <= 4 ? BN_ROW(4) : BN_ROW(8);
 #undef BN_ROW
 #undef BN_ROW_FORM

@@ -65,6 +65,59 @@ __device__ __forceinline__ void add_term(float (&acc)[VEC], const ImpBranchTerm&
     }
 }
 
+// The same for a thread that holds NV pieces of four columns, piece i from column first + i * step on while that is below d: what a
+// thread needs of all its pieces is asked for together, parts of a product several at a time, and added in the same order.
+// PARTS: the summand may be a product's parts.
+template <typename TA, int NV, bool PARTS>
+__device__ __forceinline__ void add_term_pieces(float (&acc)[NV][4], const ImpBranchTerm& s, const float (&self)[NV][4], int64_t t, int first, int step, int d,
+                                                int64_t n) {
+    auto fma4 = [](float (&a)[4], float f, const float4& v) {
+        a[0] = fmaf(f, v.x, a[0]), a[1] = fmaf(f, v.y, a[1]), a[2] = fmaf(f, v.z, a[2]), a[3] = fmaf(f, v.w, a[3]);
+    };
+    if (PARTS && s.parts) {
+        constexpr int NB = NV == 1 ? 12 : NV == 2 ? 6 : 2;
+        const float* p = s.parts + t * d;
+        for (int s0 = 0; s0 < s.n_splits; s0 += NB) {
+            float4 v[NB][NV];
+#pragma unroll
+            for (int j = 0; j < NB; ++j)
+#pragma unroll
+                for (int i = 0; i < NV; ++i)
+                    if (s0 + j < s.n_splits && first + i * step < d) v[j][i] = *reinterpret_cast<const float4*>(p + (s0 + j) * n + first + i * step);
+#pragma unroll
+            for (int j = 0; j < NB; ++j)
+#pragma unroll
+                for (int i = 0; i < NV; ++i)
+                    if (s0 + j < s.n_splits && first + i * step < d) acc[i][0] += v[j][i].x, acc[i][1] += v[j][i].y, acc[i][2] += v[j][i].z, acc[i][3] += v[j][i].w;
+        }
+    } else if (s.y) {
+        for (int k = 0; k < s.top; ++k) {
+            const int row = s.pair_row[t * s.top + k];
+            const float f = s.wts[t * s.top + k];
+            const TA* src = row >= 0 ? (const TA*)s.y + (int64_t)row * d : s.input ? (const TA*)s.input + t * d : nullptr;
+            if (src) {
+                float4 v[NV];
+#pragma unroll
+                for (int i = 0; i < NV; ++i)
+                    if (first + i * step < d) v[i] = Four<TA>::load(src + first + i * step);
+#pragma unroll
+                for (int i = 0; i < NV; ++i)
+                    if (first + i * step < d) fma4(acc[i], f, v[i]);
+            } else {
+#pragma unroll
+                for (int i = 0; i < NV; ++i)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) acc[i][e] = fmaf(f, self[i][e], acc[i][e]);
+            }
+        }
+    } else if (s.t) {
+        const TA* src = (const TA*)s.t + t * d;
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+            if (first + i * step < d) fma4(acc[i], 1.f, Four<TA>::load(src + first + i * step));
+    }
+}
+
 // Every pointer of a summand starts on 16 bytes (what four columns at a time need, with d a multiple of 4).
 inline bool term_aligned(const ImpBranchTerm& s) {
     for (const void* p : {s.t, (const void*)s.parts, s.y, s.input})

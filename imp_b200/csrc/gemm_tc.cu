@@ -1222,9 +1222,18 @@ IMP_API int imp_gemm_bf16_tc_splits(int M, int N, int K) {
     const int pairs = imp_sm_count() / 2;
     const int k_blocks = (K + TC_BK - 1) / TC_BK;
     int splits = pairs / (tiles2 > 0 ? tiles2 : 1);
-    if (splits > k_blocks / TC2_MIN_KB_PER_SPLIT) splits = k_blocks / TC2_MIN_KB_PER_SPLIT;
-    if (splits > TC2_MAX_SPLITS) splits = TC2_MAX_SPLITS;
-    return splits < 1 ? 1 : splits;
+    // one column of tiles (a router, a low-rank product): the parts are small, so a part may be short
+    const int min_kb = N <= TC2_BN ? 8 : TC2_MIN_KB_PER_SPLIT, max_splits = N <= TC2_BN ? 16 : TC2_MAX_SPLITS;
+    if (splits > k_blocks / min_kb) splits = k_blocks / min_kb;
+    if (splits > max_splits) splits = max_splits;
+    if (splits < 1) return 1;
+    // no part is empty: as many as parts of equal length (the last one shorter) make
+    for (int before = 0; before != splits;) {
+        before = splits;
+        const int kb = (k_blocks + splits - 1) / splits;
+        splits = (k_blocks + kb - 1) / kb;
+    }
+    return splits;
 }
 
 // scratch[s][M, N] (32-bit, M * N floats apart) for s < imp_gemm_bf16_tc_splits(M, N, K): the parts of A W^T.

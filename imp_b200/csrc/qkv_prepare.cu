@@ -150,8 +150,8 @@ __global__ void __launch_bounds__(QP_BLOCK) qkv_prepare_kernel(const ImpQkvPrepa
 
 // The same for 16-bit activations with eight neighbouring entries a lane (16-byte loads and stores; a rotated pair of
 // neighbours is in one lane): LPH lanes a head, 32 / LPH heads a warp at once.  Head sizes that are multiples of 8 up to
-// 8 * LPH, rows that start on 16 bytes, no rotation of halves.
-template <int LPH>
+// 8 * LPH, rows that start on 16 bytes, no rotation of halves.  PARTS: from the product's unsummed parts.
+template <int LPH, bool PARTS>
 __global__ void __launch_bounds__(QP_BLOCK) qkv_prepare_vec_kernel(const ImpQkvPrepare p, int units_per_cta, int* status) {
     pdl_wait();
     pdl_launch_dependents();
@@ -188,7 +188,7 @@ __global__ void __launch_bounds__(QP_BLOCK) qkv_prepare_vec_kernel(const ImpQkvP
         float x[8];
 #pragma unroll
         for (int i = 0; i < 8; ++i) x[i] = 0.f;
-        if (mine && p.parts) {
+        if (PARTS && mine) {
             const float* src = p.parts + t * p.ld + col + d0;
 #pragma unroll 4
             for (int s = 0; s < p.n_splits; ++s, src += (int64_t)p.n_tokens * p.ld) {
@@ -198,7 +198,7 @@ __global__ void __launch_bounds__(QP_BLOCK) qkv_prepare_vec_kernel(const ImpQkvP
             }
 #pragma unroll
             for (int i = 0; i < 8; ++i) x[i] = to_float(from_float<TA>(x[i]));
-        } else if (mine) {
+        } else if (!PARTS && mine) {
             const uint4 raw = *reinterpret_cast<const uint4*>((const TA*)p.proj + t * p.ld + col + d0);
             const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
 #pragma unroll
@@ -446,9 +446,15 @@ IMP_API int imp_qkv_prepare(const ImpQkvPrepare* args, int* status, void* stream
     const int per_cta = vec && p.n_tokens >= 2 * imp_sm_count() ? units : QP_UNITS;
     const dim3 grid((unsigned)p.n_tokens, (unsigned)((units + per_cta - 1) / per_cta));
     if (vec) {
-        if (p.Dc <= 64) imp_launch(qkv_prepare_vec_kernel<8>, grid, dim3(QP_BLOCK), 0, s, p, per_cta, status);
-        else if (p.Dc <= 128) imp_launch(qkv_prepare_vec_kernel<16>, grid, dim3(QP_BLOCK), 0, s, p, per_cta, status);
-        else imp_launch(qkv_prepare_vec_kernel<32>, grid, dim3(QP_BLOCK), 0, s, p, per_cta, status);
+#define QP_VEC(LPH)                                                                                                       \
+    do {                                                                                                                  \
+        if (p.parts) imp_launch(qkv_prepare_vec_kernel<LPH, true>, grid, dim3(QP_BLOCK), 0, s, p, per_cta, status);       \
+        else imp_launch(qkv_prepare_vec_kernel<LPH, false>, grid, dim3(QP_BLOCK), 0, s, p, per_cta, status);              \
+    } while (0)
+        if (p.Dc <= 64) QP_VEC(8);
+        else if (p.Dc <= 128) QP_VEC(16);
+        else QP_VEC(32);
+#undef QP_VEC
         IMP_RETURN_LAUNCH();
     }
 #define QP_LAUNCH(TA, PER) imp_launch(qkv_prepare_kernel<TA, PER>, grid, dim3(QP_BLOCK), 0, s, p, per_cta, status)
